@@ -87,7 +87,14 @@ const char* lumi_last_error(void);
  * attn_rope_base) and binds the model to a device. */
 int32_t lumi_model_create(const char* config_json, int32_t device_id, lumi_model** out);
 
-/* One call per safetensors entry, name including the `item.` prefix.  dtype F32 or BF16; rank-2
+/* Designs with an "architecture" key in their config.json (Zozonex: gated delta-rule and windowed attention layers listed one
+ * by one) bring their own reader and tensor names; a config without it is the Mamba-3 / attention hybrid above.
+ *
+ * Model options, set before the first tensor: "widen_weights" = 1 keeps every bf16 tensor as fp32 on the device, which makes
+ * the whole model run in fp32 (products, cache, states). */
+int32_t lumi_model_set_option(lumi_model* m, const char* name, int64_t value);
+
+/* One call per safetensors entry, name including the `item.` prefix (designs with a reader of their own: their own names).  dtype F32 or BF16; rank-2
  * tensors keep their stored width on the device, rank-1 tensors become fp32.  `ssm.h_init` may be
  * rank 2 [n_heads, d_state] or rank 1 [n_heads * d_state]. */
 int32_t lumi_model_load_tensor(lumi_model* m, const char* name, int32_t dtype, const int64_t* shape,
@@ -158,6 +165,13 @@ int32_t lumi_prefill(lumi_session* s, const uint32_t* tokens, int32_t batch, int
 int32_t lumi_prefill_ragged(lumi_session* s, const uint32_t* tokens, const int32_t* lengths, int32_t batch, int32_t T_max,
                             float* last_logits);
 
+/* Feeds the next T tokens of the sequence in `slot`, from the state that earlier calls left (a fresh or reset slot starts at
+ * position 0), and returns the logits of the places want[n_want] (ascending, 0 <= want < T) as logits_out[n_want][vocab].
+ * Prompts may be cut into calls anywhere; the logits do not depend on the cuts beyond rounding.  The hybrid takes slot 0 only
+ * and runs token by token. */
+int32_t lumi_extend(lumi_session* s, int32_t slot, const uint32_t* tokens, int32_t T, const int32_t* want, int32_t n_want,
+                    float* logits_out);
+
 /* One forward_step for each of `batch` sequences: consumes in_tokens[batch], writes the sampled /
  * argmax next token to out_tokens[batch] (may be NULL) and, if logits_out != NULL, the logits
  * [batch][vocab].  `step` indexes the Philox counter. */
@@ -189,7 +203,8 @@ int32_t lumi_session_read_state(lumi_session* s, int32_t slot, int32_t layer, fl
                                 float* b_prev, float* cum_angle);
 
 /* Runs block `layer` alone on a caller-supplied residual stream x[batch][d_model] (host, in/out),
- * using and updating the session state — for per-layer parity tests. */
+ * using and updating the session state — for per-layer parity tests.  Designs that list their layers advance the position
+ * with the last layer only: run the layers of a token in order. */
 int32_t lumi_debug_run_block(lumi_session* s, int32_t layer, float* x, int32_t batch);
 
 /* Teacher-forced scoring for the reference's `evaluate` command (inference/src/eval.rs:39-139: perplexity and

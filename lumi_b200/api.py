@@ -23,7 +23,7 @@ _lib = None
 EXPORTS = [
     "lumi_last_error", "lumi_model_create", "lumi_model_load_tensor", "lumi_model_load_safetensors",
     "lumi_model_finalize", "lumi_model_free", "lumi_model_info", "lumi_session_create", "lumi_session_reset",
-    "lumi_session_free", "lumi_session_set_option", "lumi_prefill", "lumi_prefill_ragged", "lumi_decode_step", "lumi_generate",
+    "lumi_session_free", "lumi_session_set_option", "lumi_prefill", "lumi_prefill_ragged", "lumi_extend", "lumi_model_set_option", "lumi_decode_step", "lumi_generate",
     "lumi_decode_loop_device", "lumi_profile_step", "lumi_score", "lumi_session_read_state", "lumi_session_state_bytes", "lumi_session_save_state", "lumi_session_load_state", "lumi_debug_run_block", "lumi_k_gemm_bf16_tcgen05",
     "lumi_k_gemv", "lumi_debug_gemm_wait_timeout", "lumi_debug_gemm_plan", "lumi_k_ssm_step", "lumi_k_ssd_prefill", "lumi_mamba_block_static",
 ]
@@ -70,6 +70,8 @@ def lib():
         L.lumi_session_set_option.argtypes = [vp, C.c_char_p, i64]
         L.lumi_prefill.argtypes = [vp, vp, i32, i32, vp]
         L.lumi_prefill_ragged.argtypes = [vp, vp, vp, i32, i32, vp]
+        L.lumi_model_set_option.argtypes = [vp, C.c_char_p, i64]
+        L.lumi_extend.argtypes = [vp, i32, vp, i32, vp, i32, vp]
         L.lumi_decode_step.argtypes = [vp, vp, i32, C.POINTER(Sampling), i32, vp, vp]
         L.lumi_generate.argtypes = [vp, vp, i32, i32, i32, C.POINTER(Sampling), vp, vp, vp, C.POINTER(Stats)]
         L.lumi_decode_loop_device.argtypes = [vp, i32, i32, C.POINTER(C.c_float), C.POINTER(i64)]
@@ -114,22 +116,28 @@ class NmModel:
         return h
 
     @classmethod
-    def load(cls, model_path: str, config_path: str, device: int = 0) -> "NmModel":
-        """`load_model` of inference/src/main.rs:72-89: config.json + one safetensors file."""
+    def load(cls, model_path: str, config_path: str, device: int = 0, widen_weights: bool = False) -> "NmModel":
+        """`load_model` of inference/src/main.rs:72-89: config.json + one safetensors file.  The design is chosen by the
+        config; widen_weights keeps bf16 tensors as fp32, so that everything runs in fp32."""
         with open(config_path) as f:
             text = f.read()
         h = cls._create(text, device)
-        m = cls(h, synth.ModelConfig.from_json(text))
+        m = cls(h, synth.config_from_json(text))
+        if widen_weights:
+            check(lib().lumi_model_set_option(h, b"widen_weights", 1))
         check(lib().lumi_model_load_safetensors(h, model_path.encode()))
         check(lib().lumi_model_finalize(h))
         return m
 
     @classmethod
-    def from_tensors(cls, cfg: synth.ModelConfig, tensors: Iterable[Tuple[str, int, np.ndarray]], device: int = 0) -> "NmModel":
+    def from_tensors(cls, cfg: synth.ModelConfig, tensors: Iterable[Tuple[str, int, np.ndarray]], device: int = 0,
+                     widen_weights: bool = False) -> "NmModel":
         """Loads from in-memory (name, dtype code, array) entries — the per-tensor entry point a host
         that does its own safetensors parsing would call."""
         h = cls._create(cfg.to_json(), device)
         m = cls(h, cfg)
+        if widen_weights:
+            check(lib().lumi_model_set_option(h, b"widen_weights", 1))
         for name, dt, arr in tensors:
             m.load_tensor(name, dt, arr)
         check(lib().lumi_model_finalize(h))
@@ -224,6 +232,14 @@ class Session:
         logits = np.empty((B, self.model.config.vocab_size), dtype=np.float32) if want_logits else None
         check(lib().lumi_prefill_ragged(self._h, _ptr(prompts), _ptr(lengths), B, T, _ptr(logits)))
         return logits
+
+    def extend(self, tokens, want=(), slot: int = 0) -> np.ndarray:
+        """The next tokens of the sequence in `slot`; returns the logits of the places `want` among them, [len(want), vocab]."""
+        tokens = np.ascontiguousarray(tokens, dtype=np.uint32)
+        want = np.ascontiguousarray(want, dtype=np.int32)
+        out = np.empty((len(want), self.model.config.vocab_size), dtype=np.float32)
+        check(lib().lumi_extend(self._h, slot, _ptr(tokens), len(tokens), _ptr(want), len(want), _ptr(out)))
+        return out
 
     def score(self, tokens) -> np.ndarray:
         """log p(tokens[b][t+1] | tokens[b][:t+1]) for every position (inference/src/eval.rs:39-139); [batch, T-1]."""

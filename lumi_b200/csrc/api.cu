@@ -4,6 +4,7 @@
 #include "internal.h"
 #include "json_min.h"
 
+#include <cmath>
 #include <cstdarg>
 #include <cstdio>
 #include <cstdlib>
@@ -72,6 +73,12 @@ int32_t parse_config(const char* json, Config& c) {
     std::string err;
     JsonParser p(json, strlen(json));
     if (!p.parse(root, err) || root.kind != JsonValue::Object) return fail(LUMI_E_CONFIG, "config.json: %s", err.empty() ? "not a JSON object" : err.c_str());
+    if (const JsonValue* v = root.find("architecture")) {               // a registered design with a reader of its own
+        if (v->kind != JsonValue::String) return fail(LUMI_E_CONFIG, "config.json: key 'architecture' must be a string");
+        c.arch = find_architecture(v->str.c_str());
+        if (c.arch == nullptr) return fail(LUMI_E_CONFIG, "config.json: architecture '%s' is not known", v->str.c_str());
+        return c.arch->parse(root, c);
+    }
     bool ok = get_int(root, "d_model", true, c.d_model, err) && get_int(root, "n_layers", true, c.n_layers, err) &&
               get_int(root, "d_state", true, c.d_state, err) && get_int(root, "expand", true, c.expand, err) &&
               get_int(root, "n_heads", true, c.n_heads, err) && get_int(root, "n_groups", true, c.n_groups, err) &&
@@ -126,7 +133,7 @@ extern "C" int32_t lumi_model_create(const char* config_json, int32_t device_id,
     int ndev = 0;
     LUMI_CUDA(cudaGetDeviceCount(&ndev));
     if (device_id < 0 || device_id >= ndev) return fail(LUMI_E_INVALID, "device %d not available (%d CUDA devices)", device_id, ndev);
-    if (!ssm_shape_supported(c.head_dim(), c.d_state) && c.n_attn_layers() < c.n_layers)
+    if (!c.stacked() && !ssm_shape_supported(c.head_dim(), c.d_state) && c.n_attn_layers() < c.n_layers)
         return fail(LUMI_E_UNSUPPORTED, "head_dim %d / d_state %d: kernels exist for head_dim in {16,32,64} and d_state in {16,32,64,128}", c.head_dim(), c.d_state);
     lumi_model* m = new lumi_model();
     m->cfg = c;
@@ -135,9 +142,19 @@ extern "C" int32_t lumi_model_create(const char* config_json, int32_t device_id,
     return LUMI_OK;
 }
 
-// Expected shape of a tensor by its name (without the "item." prefix); rank 0 = not a tensor of this model.
-static int expected_shape(const lumi_model* m, const std::string& name, int64_t shp[2]) {
+extern "C" int32_t lumi_model_set_option(lumi_model* m, const char* name, int64_t value) {
+    if (!m || !name) return fail(LUMI_E_INVALID, "null argument to lumi_model_set_option");
+    if (m->finalized || !m->tensors.empty()) return fail(LUMI_E_INVALID, "model options come before the first tensor");
+    if (strcmp(name, "widen_weights") == 0) m->widen = value != 0;
+    else return fail(LUMI_E_INVALID, "unknown model option '%s'", name);
+    return LUMI_OK;
+}
+
+// Expected shape of a tensor by its name (without the design's prefix); rank 0 = not a tensor of this model.
+static int expected_shape(const lumi_model* m, const std::string& name, int64_t shp[2], bool& wide) {
     const Config& c = m->cfg;
+    wide = false;
+    if (c.arch != nullptr) return c.arch->expected_shape(c, name, shp, wide);
     if (name == "embedding.weight") { shp[0] = c.vocab; shp[1] = c.d_model; return 2; }
     if (name == "final_norm.gamma") { shp[0] = c.d_model; return 1; }
     if (name.rfind("blocks.", 0) != 0) return 0;
@@ -171,10 +188,12 @@ extern "C" int32_t lumi_model_load_tensor(lumi_model* m, const char* name, int32
     if (m->finalized) return fail(LUMI_E_INVALID, "model already finalized");
     if (dtype != LUMI_DTYPE_F32 && dtype != LUMI_DTYPE_BF16) return fail(LUMI_E_TENSOR, "tensor '%s': dtype code %d not supported (F32, BF16)", name, dtype);
     std::string n(name);
-    if (n.rfind("item.", 0) != 0) return LUMI_OK;         // the reference only reads names under "item." (main.rs:86)
-    n = n.substr(5);
+    const std::string prefix = m->cfg.arch != nullptr ? m->cfg.arch->tensor_prefix : "item.";
+    if (n.rfind(prefix, 0) != 0) return LUMI_OK;          // the reference only reads names under "item." (main.rs:86)
+    n = n.substr(prefix.size());
     int64_t exp[2] = {0, 0};
-    const int erank = expected_shape(m, n, exp);
+    bool wide = false;
+    const int erank = expected_shape(m, n, exp, wide);
     if (erank == 0) return LUMI_OK;                       // tensors the model never asks for are ignored, as VarBuilder does
     if (m->tensors.count(n)) return fail(LUMI_E_TENSOR, "tensor '%s' loaded twice", name);
     int64_t count = 1;
@@ -193,8 +212,8 @@ extern "C" int32_t lumi_model_load_tensor(lumi_model* m, const char* name, int32
     if ((uint64_t)count * esz != nbytes) return fail(LUMI_E_TENSOR, "tensor '%s': %llu bytes given, shape needs %llu", name, (unsigned long long)nbytes, (unsigned long long)(count * esz));
     LUMI_CUDA(cudaSetDevice(m->device));
     DevTensor t;
-    const bool keep_width = (erank == 2) && !is_hinit;
-    if (keep_width) {
+    const bool keep_width = (erank == 2) && !is_hinit && !wide;
+    if (keep_width && !(m->widen && dtype == LUMI_DTYPE_BF16)) {
         if (m->wdtype >= 0 && m->wdtype != dtype) return fail(LUMI_E_TENSOR, "tensor '%s': rank-2 tensors mix F32 and BF16", name);
         m->wdtype = dtype;
         t.dtype = dtype;
@@ -211,8 +230,12 @@ extern "C" int32_t lumi_model_load_tensor(lumi_model* m, const char* name, int32
             for (int64_t i = 0; i < count; ++i) tmp[i] = bf16_to_f32(b[i]);
             src = tmp.data();
         }
+        if (keep_width) {                                 // a bf16 matrix widened to fp32
+            if (m->wdtype >= 0 && m->wdtype != LUMI_DTYPE_F32) return fail(LUMI_E_TENSOR, "tensor '%s': rank-2 tensors mix F32 and BF16", name);
+            m->wdtype = LUMI_DTYPE_F32;
+        }
         t.dtype = LUMI_DTYPE_F32;
-        t.rows = 1; t.cols = count;
+        t.rows = keep_width ? exp[0] : 1; t.cols = keep_width ? exp[1] : count;
         t.bytes = (size_t)count * 4;
         LUMI_CUDA(cudaMalloc(&t.p, t.bytes));
         LUMI_CUDA(cudaMemcpy(t.p, src, t.bytes, cudaMemcpyHostToDevice));
@@ -223,7 +246,7 @@ extern "C" int32_t lumi_model_load_tensor(lumi_model* m, const char* name, int32
 
 static int32_t need(lumi_model* m, const std::string& n, DevTensor& out) {
     auto it = m->tensors.find(n);
-    if (it == m->tensors.end()) return fail(LUMI_E_TENSOR, "tensor 'item.%s' is missing", n.c_str());
+    if (it == m->tensors.end()) return fail(LUMI_E_TENSOR, "tensor '%s%s' is missing", m->cfg.arch != nullptr ? m->cfg.arch->tensor_prefix : "item.", n.c_str());
     out = it->second;
     return LUMI_OK;
 }
@@ -265,11 +288,114 @@ static int32_t concat_rows(lumi_model* m, const std::vector<std::string>& names,
     return LUMI_OK;
 }
 
+// ---- listed layers: their weights in the padded layout the products take -----------------------------------
+static int64_t up64(int64_t n) { return (n + 63) / 64 * 64; }
+
+// [rows][cols] matrices stacked by rows, every part starting on a multiple of 8 rows, the total and the columns padded to
+// multiples of 64 with zeros.  offs (may be null) receives the first row of every part.  The parts are released.
+static int32_t stack_padded(lumi_model* m, const std::vector<std::string>& names, DevTensor& out, std::vector<int>* offs) {
+    std::vector<DevTensor> parts(names.size());
+    int64_t rows = 0;
+    std::vector<int64_t> at;
+    for (size_t i = 0; i < names.size(); ++i) {
+        LUMI_TRY(need(m, names[i], parts[i]));
+        at.push_back(rows);
+        if (offs) offs->push_back((int)rows);
+        rows += (parts[i].rows + 7) / 8 * 8;
+    }
+    out = parts[0];
+    const size_t esz = out.dtype == LUMI_DTYPE_BF16 ? 2 : 4;
+    const int64_t cols = up64(out.cols);
+    out.rows = up64(rows); out.cols = cols; out.bytes = (size_t)out.rows * cols * esz;
+    LUMI_CUDA(cudaMalloc(&out.p, out.bytes));
+    m->owned.push_back(out.p);
+    LUMI_CUDA(cudaMemset(out.p, 0, out.bytes));
+    for (size_t i = 0; i < names.size(); ++i) {
+        LUMI_CUDA(cudaMemcpy2D((char*)out.p + (size_t)at[i] * cols * esz, cols * esz, parts[i].p, parts[i].cols * esz, parts[i].cols * esz,
+                               parts[i].rows, cudaMemcpyDeviceToDevice));
+        LUMI_CUDA(cudaFree(parts[i].p));
+        m->tensors[names[i]].p = nullptr;
+    }
+    return LUMI_OK;
+}
+// The factor of a norm whose stored weight is an offset from one, padded with zeros.
+static int32_t norm_factor(lumi_model* m, const std::string& n, const float*& out) {
+    DevTensor t;
+    LUMI_TRY(need(m, n, t));
+    std::vector<float> w(up64(t.cols), 0.f);
+    LUMI_CUDA(cudaMemcpy(w.data(), t.p, (size_t)t.cols * 4, cudaMemcpyDeviceToHost));
+    for (int64_t i = 0; i < t.cols; ++i) w[i] = 1.0f + w[i];
+    void* p = nullptr;
+    LUMI_CUDA(cudaMalloc(&p, w.size() * 4));
+    m->owned.push_back(p);
+    LUMI_CUDA(cudaMemcpy(p, w.data(), w.size() * 4, cudaMemcpyHostToDevice));
+    out = (const float*)p;
+    return LUMI_OK;
+}
+
+static int32_t finalize_stacked(lumi_model* m) {
+    const Config& c = m->cfg;
+    for (auto& kv : m->tensors) m->weight_bytes += (int64_t)kv.second.bytes;
+    {
+        // the embedding keeps its row count (the vocabulary), its columns are padded
+        DevTensor t;
+        LUMI_TRY(need(m, "embed", t));
+        m->embedding = t;
+        if (t.cols != up64(t.cols)) {
+            const size_t esz = t.dtype == LUMI_DTYPE_BF16 ? 2 : 4;
+            m->embedding.cols = up64(t.cols);
+            m->embedding.bytes = (size_t)t.rows * m->embedding.cols * esz;
+            LUMI_CUDA(cudaMalloc(&m->embedding.p, m->embedding.bytes));
+            m->owned.push_back(m->embedding.p);
+            LUMI_CUDA(cudaMemset(m->embedding.p, 0, m->embedding.bytes));
+            LUMI_CUDA(cudaMemcpy2D(m->embedding.p, m->embedding.cols * esz, t.p, t.cols * esz, t.cols * esz, t.rows, cudaMemcpyDeviceToDevice));
+        }
+    }
+    LUMI_TRY(norm_factor(m, "final.norm", m->final_norm_g));
+    m->layers.assign(c.n_layers, Layer());
+    for (int i = 0; i < c.n_layers; ++i) {
+        Layer& L = m->layers[i];
+        const MixerSpec& mx = c.specs[i].mixer;
+        const std::string p = "l" + std::to_string(i) + ".", q = p + "mix.";
+        L.spec = &c.specs[i];
+        LUMI_TRY(norm_factor(m, p + "norm1", L.s.norm1));
+        std::vector<int> off;
+        if (mx.kind == MIXER_DELTA) {
+            L.kind_idx = m->n_delta++;
+            LUMI_TRY(stack_padded(m, {q + "q", q + "k", q + "v", q + "b", q + "a", q + "g"}, L.s.in, &off));
+            L.s.off_b = off[3]; L.s.off_a = off[4]; L.s.off_g = off[5];
+            LUMI_TRY(need_f(m, q + "q.conv", L.s.conv_q));
+            LUMI_TRY(need_f(m, q + "k.conv", L.s.conv_k));
+            LUMI_TRY(need_f(m, q + "v.conv", L.s.conv_v));
+            LUMI_TRY(need_f(m, q + "A_log", L.s.a_log));
+            LUMI_TRY(need_f(m, q + "dt_bias", L.s.dt_bias));
+            LUMI_TRY(need_f(m, q + "norm", L.s.o_norm));
+        } else {
+            L.kind_idx = m->n_wattn++;
+            L.window = mx.window;
+            std::vector<std::string> names = {q + "q"};
+            if (mx.kv_from < 0) { names.push_back(q + "k"); names.push_back(q + "v"); }
+            LUMI_TRY(stack_padded(m, names, L.s.in, &off));
+        }
+        if (off.size() > 1) { L.s.off_k = off[1]; L.s.off_v = off[2]; }
+        LUMI_TRY(stack_padded(m, {q + "o"}, L.s.out, nullptr));
+        if (L.spec->ff > 0) {
+            LUMI_TRY(norm_factor(m, p + "norm2", L.s.norm2));
+            LUMI_TRY(stack_padded(m, {p + "mlp.up"}, L.s.up, nullptr));
+            LUMI_TRY(stack_padded(m, {p + "mlp.down"}, L.s.down, nullptr));
+        }
+    }
+    if (m->wdtype < 0) m->wdtype = LUMI_DTYPE_F32;
+    m->finalized = true;
+    return LUMI_OK;
+}
+
 extern "C" int32_t lumi_model_finalize(lumi_model* m) {
     if (!m) return fail(LUMI_E_INVALID, "model is null");
     if (m->finalized) return LUMI_OK;
     LUMI_CUDA(cudaSetDevice(m->device));
     const Config& c = m->cfg;
+    if (c.stacked()) return finalize_stacked(m);
     LUMI_TRY(need(m, "embedding.weight", m->embedding));
     LUMI_TRY(need_f(m, "final_norm.gamma", m->final_norm_g));
     m->weight_bytes = 0;
@@ -324,12 +450,124 @@ extern "C" int32_t lumi_model_info(const lumi_model* m, int64_t* o) {
     if (!m || !o) return fail(LUMI_E_INVALID, "null argument to lumi_model_info");
     const Config& c = m->cfg;
     o[0] = c.d_model; o[1] = c.n_layers; o[2] = c.d_state; o[3] = c.n_heads; o[4] = c.head_dim(); o[5] = c.n_groups;
-    o[6] = c.vocab; o[7] = m->n_mamba; o[8] = m->n_attn; o[9] = c.in_proj_out(); o[10] = m->wdtype; o[11] = m->weight_bytes;
+    o[6] = c.vocab; o[7] = m->n_mamba + m->n_delta; o[8] = m->n_attn + m->n_wattn; o[9] = c.in_proj_out(); o[10] = m->wdtype; o[11] = m->weight_bytes;
     return LUMI_OK;
 }
 
 // ---- sessions ---------------------------------------------------------------------------------------
 static size_t state_h_per_seq(const Config& c) { return (size_t)c.n_heads * c.head_dim() * c.d_state; }
+
+static void free_rows(RowBufs& b) {
+    void* all[] = {b.x, b.proj, b.mix, b.qkv, b.gates, b.y32, b.xh, b.xl, b.ah, b.al};
+    for (void* p : all) if (p) cudaFree(p);
+    b = RowBufs();
+}
+
+// Widest rows of the passes over listed layers.
+struct RowWidths { size_t proj = 0, act = 0, mix = 0, qkv = 0, gates = 0; };
+static RowWidths row_widths(const lumi_model* m) {
+    RowWidths w;
+    w.mix = (size_t)m->cfg.x_ld();
+    for (const Layer& L : m->layers) {
+        const MixerSpec& x = L.spec->mixer;
+        w.proj = std::max(w.proj, (size_t)L.s.in.rows);
+        w.act = std::max({w.act, (size_t)L.s.out.cols, L.spec->ff > 0 ? (size_t)L.s.up.rows : 0});
+        if (x.kind == MIXER_DELTA) {
+            const size_t dk4 = (x.dim + 3) / 4 * 4, dvp = (x.vdim + 3) / 4 * 4;
+            w.mix = std::max(w.mix, x.heads * dvp);
+            w.qkv = std::max(w.qkv, 2 * x.kv_heads * dk4 + x.heads * dvp);
+            w.gates = std::max(w.gates, (size_t)2 * x.heads);
+        }
+    }
+    return w;
+}
+// slices: the buffers of the chunked recurrence are needed as well.  Everything starts as zeros, so that padding stays finite.
+static int32_t alloc_rows(lumi_session* s, RowBufs& b, size_t rows, bool slices) {
+    const RowWidths w = row_widths(s->m);
+    const bool half = s->m->wdtype == LUMI_DTYPE_BF16;
+    const size_t rp = (rows + 127) / 128 * 128, ldx = s->m->cfg.x_ld();
+    auto get = [&](auto*& p, size_t n) -> int32_t {
+        LUMI_CUDA(cudaMalloc(&p, n * sizeof(*p)));
+        LUMI_CUDA(cudaMemsetAsync(p, 0, n * sizeof(*p), s->stream));
+        return LUMI_OK;
+    };
+    if (b.x == nullptr) LUMI_TRY(get(b.x, rp * ldx));
+    LUMI_TRY(get(b.proj, rp * w.proj));
+    LUMI_TRY(get(b.mix, rp * w.mix));
+    LUMI_TRY(get(b.y32, (half && s->opt_gemm != 1 ? std::min<size_t>(rp, 8) : rp) * std::max(w.act, ldx)));
+    if (half) {
+        LUMI_TRY(get(b.xh, rp * ldx));
+        LUMI_TRY(get(b.xl, rp * ldx));
+        LUMI_TRY(get(b.ah, rp * w.act));
+        LUMI_TRY(get(b.al, rp * w.act));
+    }
+    if (slices && w.qkv > 0) {
+        LUMI_TRY(get(b.qkv, rp * w.qkv));
+        LUMI_TRY(get(b.gates, rp * w.gates));
+    }
+    b.rows = rows;
+    return LUMI_OK;
+}
+
+// State of the listed layers: per slot the matrix states and convolution rings of the delta-rule layers, and for attention
+// layers with keys and values of their own a ring of pages.  One ring length serves all of them: the widest window plus the
+// longest slice a pass may append before it attends (without a window: the whole capacity).
+static int32_t alloc_stacked(lumi_session* s) {
+    const Config& c = s->m->cfg;
+    const size_t B = s->max_batch;
+    const size_t esz = s->m->wdtype == LUMI_DTYPE_BF16 ? 2 : 4;
+    s->slice_max = 4096;
+    if (s->m->n_wattn > 0) {
+        if (s->max_tokens_kv <= 0) return fail(LUMI_E_INVALID, "max_tokens_kv must be > 0 for a model with attention layers");
+        const int mw = c.max_window(), cap = s->max_tokens_kv;
+        int ring = cap;
+        if (mw > 0 && cap >= mw) {
+            ring = mw - 1 + std::min(std::max(cap, 64), 1024);
+            s->kv_limit = 0;
+        } else {
+            s->kv_limit = cap;
+        }
+        s->pages_per_seq = (ring + kPageTokens - 1) / kPageTokens;
+        if (s->kv_limit == 0) s->slice_max = s->pages_per_seq * kPageTokens - mw + 1;
+        std::vector<int32_t> pt(B * s->pages_per_seq);
+        for (size_t i = 0; i < pt.size(); ++i) pt[i] = (int32_t)i;       // slot b owns pages [b*pps, (b+1)*pps)
+        LUMI_CUDA(cudaMalloc(&s->page_table, sizeof(int32_t) * pt.size()));
+        LUMI_CUDA(cudaMemcpy(s->page_table, pt.data(), pt.size() * sizeof(int32_t), cudaMemcpyHostToDevice));
+        size_t pw = 0;
+        for (const LayerSpec& L : c.specs) if (L.mixer.kind == MIXER_ATTENTION) pw = std::max(pw, window_attention_part_floats(L.mixer));
+        LUMI_CUDA(cudaMalloc(&s->attn_part, sizeof(float) * kAttnPartUnits * pw));
+        LUMI_CUDA(cudaMalloc(&s->attn_part_count, sizeof(int32_t) * kAttnPartUnits));
+        LUMI_CUDA(cudaMemset(s->attn_part_count, 0, sizeof(int32_t) * kAttnPartUnits));
+    }
+    s->lstate.assign(c.n_layers, LayerState());
+    for (int i = 0; i < c.n_layers; ++i) {
+        const MixerSpec& m = c.specs[i].mixer;
+        LayerState& L = s->lstate[i];
+        if (m.kind == MIXER_DELTA) {
+            L.dvp = (m.vdim + 3) / 4 * 4;
+            L.channels = 2 * m.kv_heads * m.dim + m.heads * m.vdim;
+            L.s_seq = (size_t)m.heads * m.dim * L.dvp;
+            L.conv_seq = (size_t)m.taps * L.channels;
+            LUMI_CUDA(cudaMalloc(&L.S, sizeof(float) * B * L.s_seq));
+            LUMI_CUDA(cudaMalloc(&L.conv, sizeof(float) * B * L.conv_seq));
+            LUMI_CUDA(cudaMemset(L.conv, 0, sizeof(float) * B * L.conv_seq));
+        } else {
+            L.dk_pad = (m.dim + 15) / 16 * 16; L.dv_pad = (m.vdim + 15) / 16 * 16;
+            if (m.kv_from >= 0) continue;
+            L.kv_bytes = B * s->pages_per_seq * (size_t)m.kv_heads * kPageTokens * (L.dk_pad + L.dv_pad) * esz;
+            LUMI_CUDA(cudaMalloc(&L.kv, L.kv_bytes));
+            LUMI_CUDA(cudaMemset(L.kv, 0, L.kv_bytes));
+        }
+    }
+    if (c.embed_positions) {
+        // frequencies in half turns per position: f / pi
+        std::vector<double> f((c.d_model + 1) / 2);
+        for (size_t i = 0; i < f.size(); ++i) f[i] = std::pow(10000.0, -2.0 * (double)i / (double)c.d_model) / 3.14159265358979323846;
+        LUMI_CUDA(cudaMalloc(&s->pos_freq, sizeof(double) * f.size()));
+        LUMI_CUDA(cudaMemcpy(s->pos_freq, f.data(), sizeof(double) * f.size(), cudaMemcpyHostToDevice));
+    }
+    return LUMI_OK;
+}
 
 extern "C" void lumi_session_free(lumi_session* s) {
     if (!s) return;
@@ -341,6 +579,12 @@ extern "C" void lumi_session_free(lumi_session* s) {
                    s->pf_x, s->pf_proj, s->pf_rb, s->pf_rc, s->pf_hi, s->pf_lo, s->slot_buf, s->xn_hi, s->xn_lo, s->ssq, s->attn_part, s->attn_part_count, s->amax_val, s->amax_idx, s->row_len, s->xlast,
                    s->b1_layers, s->b1_grid_ctl, s->b1_amax_val, s->b1_amax_idx, s->b1_timing, s->b1_tagged};
     for (void* p : dev) if (p) cudaFree(p);
+    s->dec.x = nullptr;                                   // the session's x, freed above
+    free_rows(s->dec);
+    free_rows(s->pre);
+    for (LayerState& L : s->lstate) { if (L.kv) cudaFree(L.kv); if (L.S) cudaFree(L.S); if (L.conv) cudaFree(L.conv); }
+    if (s->pos_freq) cudaFree(s->pos_freq);
+    if (s->want_idx) cudaFree(s->want_idx);
     if (s->ctl_host) cudaFreeHost(s->ctl_host);
     if (s->pin_tokens) cudaFreeHost(s->pin_tokens);
     if (s->ev0) cudaEventDestroy(s->ev0);
@@ -406,22 +650,31 @@ static int32_t session_alloc(lumi_session* s) {
     LUMI_CUDA(cudaMalloc(&s->kv_pos, sizeof(int32_t) * B));
     LUMI_CUDA(cudaMalloc(&s->slot_buf, sizeof(int32_t) * B));
     LUMI_CUDA(cudaMalloc(&s->row_len, sizeof(int32_t) * B));
-    LUMI_CUDA(cudaMalloc(&s->xlast, sizeof(float) * B * c.d_model));
+    LUMI_CUDA(cudaMalloc(&s->xlast, sizeof(float) * B * c.x_ld()));
     LUMI_CUDA(cudaMalloc(&s->gemm_counters, sizeof(int32_t) * 2 * kGemmCounters));
     LUMI_CUDA(cudaMemset(s->gemm_counters, 0, sizeof(int32_t) * 2 * kGemmCounters));
     LUMI_CUDA(cudaMalloc(&s->gemm_scratch, sizeof(float) * 2 * kGemmScratchFloats));
+    if (c.stacked()) {
+        LUMI_TRY(alloc_stacked(s));
+        LUMI_CUDA(cudaMalloc(&s->x, sizeof(float) * (B + 127) / 128 * 128 * c.x_ld()));
+        LUMI_CUDA(cudaMemset(s->x, 0, sizeof(float) * (B + 127) / 128 * 128 * c.x_ld()));
+        s->dec.x = s->x;
+        LUMI_TRY(alloc_rows(s, s->dec, B, false));
+    }
     const size_t kmax = std::max<size_t>({(size_t)c.d_model, (size_t)c.d_inner(), na > 0 ? (size_t)c.mlp_dim() : 0});
     const size_t pmax = std::max<size_t>({nm > 0 ? (size_t)c.in_proj_out() : 0, na > 0 ? (size_t)(c.d_model + 2 * c.kv_dim()) : 0,
                                           na > 0 ? (size_t)(2 * c.mlp_dim()) : 0});
-    LUMI_CUDA(cudaMalloc(&s->x, sizeof(float) * B * c.d_model));
-    LUMI_CUDA(cudaMalloc(&s->proj, sizeof(float) * B * pmax));
-    LUMI_CUDA(cudaMalloc(&s->y32, sizeof(float) * B * kmax));
+    if (!c.stacked()) {
+        LUMI_CUDA(cudaMalloc(&s->x, sizeof(float) * B * c.d_model));
+        LUMI_CUDA(cudaMalloc(&s->proj, sizeof(float) * B * pmax));
+        LUMI_CUDA(cudaMalloc(&s->y32, sizeof(float) * B * kmax));
+    }
     LUMI_CUDA(cudaMalloc(&s->logits, sizeof(float) * B * c.vocab));
     // per-CTA argmax partials of the greedy head at batch <= 8 (at most one CTA per vocabulary row)
     s->amax_stride = c.vocab;
     LUMI_CUDA(cudaMalloc(&s->amax_val, sizeof(float) * 8 * (size_t)c.vocab));
     LUMI_CUDA(cudaMalloc(&s->amax_idx, sizeof(int) * 8 * (size_t)c.vocab));
-    if (s->m->wdtype == LUMI_DTYPE_BF16) {
+    if (s->m->wdtype == LUMI_DTYPE_BF16 && !c.stacked()) {
         // rows padded to a whole 128-row tile so TMA boxes never start outside the allocation
         const size_t rows = (B + 127) / 128 * 128;
         s->act_ld = kmax;
@@ -448,7 +701,7 @@ static int32_t session_alloc(lumi_session* s) {
     memset(s->ctl_host, 0, sizeof(StepCtl));
     LUMI_CUDA(cudaMemset(s->tok_cur, 0, sizeof(uint32_t) * B));
     // batch-1 persistent kernel: per-layer pointer table, barrier words, argmax partials
-    s->b1_ok = decode_b1_supported(c, na, s->m->device);
+    s->b1_ok = !c.stacked() && decode_b1_supported(c, na, s->m->device);
     if (s->b1_ok) {
         std::vector<B1Layer> tab;
         for (const Layer& L : s->m->layers) {
@@ -515,8 +768,14 @@ extern "C" int32_t lumi_session_reset(lumi_session* s, const int32_t* slots, int
         LUMI_CUDA(cudaMemcpyAsync(dslots, slots, sizeof(int32_t) * n_slots, cudaMemcpyHostToDevice, s->stream));
         n = n_slots;
     }
+    for (size_t i = 0; i < s->lstate.size(); ++i) {       // listed layers: only the matrix states; rings are read by position
+        const LayerState& L = s->lstate[i];
+        if (L.S == nullptr) continue;
+        if (!slots) LUMI_CUDA(cudaMemsetAsync(L.S, 0, sizeof(float) * B * L.s_seq, s->stream));
+        else for (int j = 0; j < n_slots; ++j) LUMI_CUDA(cudaMemsetAsync(L.S + (size_t)slots[j] * L.s_seq, 0, sizeof(float) * L.s_seq, s->stream));
+    }
     for (auto& L : s->m->layers) {
-        if (L.is_attn) continue;
+        if (!L.is_mamba()) continue;
         const size_t l = L.kind_idx;
         LUMI_CUDA(launch_state_reset(s->h + l * B * state_h_per_seq(c), s->xprev + l * B * c.d_inner(),
                                      s->bprev + l * B * c.n_heads * c.d_state, s->cum + l * B * c.n_heads * (c.d_state / 2),
@@ -534,7 +793,11 @@ extern "C" int32_t lumi_session_reset(lumi_session* s, const int32_t* slots, int
 extern "C" int32_t lumi_session_set_option(lumi_session* s, const char* name, int64_t value) {
     if (!s || !name) return fail(LUMI_E_INVALID, "null argument to lumi_session_set_option");
     const std::string n(name);
-    if (n == "gemm") { if (value < 0 || value > 2) return fail(LUMI_E_INVALID, "option gemm: 0, 1 or 2"); s->opt_gemm = (int)value; }
+    if (n == "gemm") {
+        if (value < 0 || value > 2) return fail(LUMI_E_INVALID, "option gemm: 0, 1 or 2");
+        if (s->m->cfg.stacked() && value == 1) return fail(LUMI_E_UNSUPPORTED, "option gemm: designs that list their layers choose between GEMV and tensor cores by rows");
+        s->opt_gemm = (int)value;
+    }
     else if (n == "split_activations") s->opt_split = value ? 1 : 0;
     else if (n == "graph") s->opt_graph = value ? 1 : 0;
     else if (n == "pdl") s->opt_pdl = value ? 1 : 0;
@@ -584,6 +847,7 @@ void mark(StepPlan& p) {
 bool use_tc(const lumi_session* s, int B) {
     const Config& c = s->m->cfg;
     if (s->m->wdtype != LUMI_DTYPE_BF16 || s->opt_gemm == 1) return false;
+    if (c.stacked()) return s->opt_gemm == 2 || B > 8;                  // padded to whole blocks at load
     if ((c.d_model % 64) || (c.d_inner() % 64) || (s->m->n_attn > 0 && (c.mlp_dim() % 64))) return false;
     return s->opt_gemm == 2 || B > 8;
 }
@@ -742,6 +1006,158 @@ int32_t attention_block(StepPlan& p, const Layer& L) {
     return LUMI_OK;
 }
 
+// ---- listed layers ------------------------------------------------------------------------------------------
+// Rows of one pass: nseq sequences (slots b0 ...) x ts tokens; decode steps have ts == 1.
+struct RowPass {
+    RowBufs* b;
+    int nseq, ts, b0;
+    const int32_t* row_len;      // prompts of different lengths (null otherwise)
+    int t_abs0;                  // first prompt position of a slice; -1 = decode form (the step's prompt position decides)
+    int rows() const { return nseq * ts; }
+};
+
+EmbedPost embed_post_of(const lumi_session* s, const RowBufs& b, int slot0, bool tc) {
+    EmbedPost e;
+    const Config& c = s->m->cfg;
+    if (!c.stacked()) return e;
+    e.scale = c.embed_scale;
+    e.freq = c.embed_positions ? s->pos_freq : nullptr;
+    e.pos = s->kv_pos + slot0;
+    e.width = c.d_model;
+    if (tc) { e.hi = b.xh; e.lo = s->opt_split ? b.xl : nullptr; }
+    return e;
+}
+
+// D = act(A W^T) over `rows` rows: tensor cores from the bf16 halves, or the weight-streaming kernel from fp32 rows.  The result
+// goes to out32, or (tensor cores, out_hi given) as bf16 halves only.
+int32_t product(StepPlan& p, int rows, const DevTensor& W, const float* in32, const __nv_bfloat16* hi, const __nv_bfloat16* lo, float* out32,
+                int ldd, int act, __nv_bfloat16* out_hi = nullptr, __nv_bfloat16* out_lo = nullptr) {
+    lumi_session* s = p.s;
+    const int N = (int)W.rows, K = (int)W.cols;
+    mark(p);
+    if (!p.tc) {
+        GemvArgs g{in32, K, W.p, W.dtype, out32, ldd, nullptr, nullptr, rows, N, K, s->m->cfg.eps, act, &s->ctl->status};
+        const cudaError_t e = launch_gemv(g, p.st_hi);
+        if (e == cudaErrorInvalidValue) return fail(LUMI_E_UNSUPPORTED, "a product over %d inputs is longer than the streaming kernel takes", K);
+        LUMI_CUDA(e);
+        return LUMI_OK;
+    }
+    GemmArgs g{hi, s->opt_split ? lo : nullptr, (const __nv_bfloat16*)W.p, out_hi ? nullptr : out32, ldd, rows, N, K, 0, &s->ctl->status,
+               s->gemm_counters, kGemmCounters, s->gemm_scratch, kGemmScratchFloats};
+    g.nf.act = act;
+    g.nf.out_hi = out_hi;
+    g.nf.out_lo = s->opt_split ? out_lo : nullptr;
+    return launch_gemm_tcgen05(g, p.st_hi);
+}
+
+// The residual stream takes the norm of a sublayer's output; on the tensor-core path its bf16 halves are renewed as well.
+int32_t add_normed(StepPlan& p, RowPass& r, const float* w) {
+    const Config& c = p.s->m->cfg;
+    RowBufs& b = *r.b;
+    RowNormArgs a{b.x, b.mix, w, nullptr, p.tc ? b.xh : nullptr, p.tc && p.s->opt_split ? b.xl : nullptr, nullptr, r.rows(), c.d_model, c.x_ld(), c.eps};
+    const int fam = p.fam;
+    p.fam = FAM_NORM;
+    mark(p);
+    LUMI_CUDA(launch_row_norm(a, p.st_hi));
+    p.fam = fam;
+    return LUMI_OK;
+}
+
+int32_t listed_layer(StepPlan& p, RowPass& r, const Layer& L) {
+    lumi_session* s = p.s;
+    const Config& c = s->m->cfg;
+    const MixerSpec& m = L.spec->mixer;
+    RowBufs& b = *r.b;
+    const int rows = r.rows(), ldx = c.x_ld(), li = (int)(&L - s->m->layers.data());
+    __nv_bfloat16* ah = p.tc ? b.ah : nullptr;
+    __nv_bfloat16* al = p.tc && s->opt_split ? b.al : nullptr;
+    float* y32 = p.tc ? nullptr : b.y32;
+    p.fam = m.kind == MIXER_DELTA ? FAM_IN_PROJ : FAM_ATTN;
+    LUMI_TRY(product(p, rows, L.s.in, b.x, b.xh, b.xl, b.proj, (int)L.s.in.rows, 0));
+    int n = 0;
+    if (m.kind == MIXER_DELTA) {
+        const LayerState& S = s->lstate[li];
+        DeltaArgs a{};
+        a.proj = b.proj; a.ldp = (int)L.s.in.rows;
+        a.off_q = L.s.off_q; a.off_k = L.s.off_k; a.off_v = L.s.off_v; a.off_b = L.s.off_b; a.off_a = L.s.off_a; a.off_g = L.s.off_g;
+        a.conv_q = L.s.conv_q; a.conv_k = L.s.conv_k; a.conv_v = L.s.conv_v;
+        a.a_log = L.s.a_log; a.dt_bias = L.s.dt_bias; a.o_norm = L.s.o_norm;
+        a.S = S.S; a.conv = S.conv;
+        a.H = m.heads; a.G = m.kv_heads; a.dk = m.dim; a.dv = m.vdim; a.dvp = S.dvp; a.taps = m.taps;
+        a.eps = c.eps; a.unit_eps = m.unit_eps;
+        a.pos = s->kv_pos; a.row_len = r.row_len; a.t_abs0 = r.t_abs0; a.ctl = s->ctl;
+        a.nseq = r.nseq; a.ts = r.ts; a.b0 = r.b0;
+        a.y32 = y32; a.yhi = ah; a.ylo = al; a.ldy = (int)L.s.out.cols;
+        a.qkv = b.qkv; a.ldqkv = 2 * m.kv_heads * ((m.dim + 3) / 4 * 4) + m.heads * S.dvp; a.gates = b.gates; a.o32 = b.mix;
+        p.fam = FAM_SSM;
+        mark(p);
+        // short slices and fp32 models go token by token (the chunked form's products are tf32 terms)
+        const bool chunked = r.ts >= 16 && b.qkv != nullptr && s->m->wdtype == LUMI_DTYPE_BF16 && delta_chunk_supported(m.dim, m.vdim);
+        const cudaError_t e = chunked ? launch_delta_chunk(a, p.st_lo, &n) : launch_delta_step(a, p.st_lo, &n);
+        if (e == cudaErrorInvalidValue) return fail(LUMI_E_UNSUPPORTED, "delta-rule heads of %d x %d are not built", m.dim, m.vdim);
+        LUMI_CUDA(e);
+    } else {
+        const LayerState& own = s->lstate[li];
+        const LayerState& src = s->lstate[m.kv_from >= 0 ? m.kv_from : li];
+        WinAttnArgs a{};
+        a.proj = b.proj; a.ldp = (int)L.s.in.rows; a.off_q = L.s.off_q; a.off_k = L.s.off_k; a.off_v = L.s.off_v;
+        a.kv = src.kv; a.kv_is_f32 = s->m->wdtype == LUMI_DTYPE_BF16 ? 0 : 1; a.dk_pad = own.dk_pad; a.dv_pad = own.dv_pad;
+        a.page_table = s->page_table; a.pages_per_seq = s->pages_per_seq; a.pos = s->kv_pos;
+        a.H = m.heads; a.G = m.kv_heads; a.dk = m.dim; a.dv = m.vdim; a.m = m;
+        a.append = m.kv_from < 0 ? 1 : 0;
+        a.eps = c.eps;
+        a.row_len = r.row_len; a.t_abs0 = r.t_abs0; a.ctl = s->ctl;
+        a.nseq = r.nseq; a.ts = r.ts; a.b0 = r.b0; a.limit = s->kv_limit;
+        a.y32 = y32; a.yhi = ah; a.ylo = al; a.ldy = (int)L.s.out.cols;
+        a.part = s->attn_part; a.part_count = s->attn_part_count;
+        mark(p);
+        const cudaError_t e = launch_window_attention(a, p.st_hi, &n);
+        if (e == cudaErrorInvalidValue) return fail(LUMI_E_UNSUPPORTED, "attention heads of %d / %d elements are not built", m.dim, m.vdim);
+        LUMI_CUDA(e);
+    }
+    p.n += n - 1;                                         // mark() counted one
+    p.fam = m.kind == MIXER_DELTA ? FAM_OUT_PROJ : FAM_ATTN;
+    LUMI_TRY(product(p, rows, L.s.out, b.y32, b.ah, b.al, b.mix, ldx, 0));
+    LUMI_TRY(add_normed(p, r, L.s.norm1));
+    if (L.spec->ff > 0) {
+        p.fam = FAM_ATTN;
+        LUMI_TRY(product(p, rows, L.s.up, b.x, b.xh, b.xl, b.y32, (int)L.s.up.rows, 2, ah, b.al));
+        LUMI_TRY(product(p, rows, L.s.down, b.y32, b.ah, b.al, b.mix, ldx, 0));
+        LUMI_TRY(add_normed(p, r, L.s.norm2));
+    }
+    return LUMI_OK;
+}
+
+// Final norm and tied head over `rows` rows of b.x (row_idx, device, picks them; null = the first `rows`).
+int32_t listed_head(StepPlan& p, RowBufs& b, const int32_t* row_idx, int rows, float* out) {
+    lumi_session* s = p.s;
+    const Config& c = s->m->cfg;
+    const bool tc = use_tc(s, rows);
+    RowNormArgs a{b.x, nullptr, s->m->final_norm_g, tc ? nullptr : b.y32, tc ? b.xh : nullptr, tc && s->opt_split ? b.xl : nullptr, row_idx, rows,
+                  c.d_model, c.x_ld(), c.eps};
+    p.fam = FAM_HEAD;
+    mark(p);
+    LUMI_CUDA(launch_row_norm(a, p.st_hi));
+    const bool keep = p.tc;
+    p.tc = tc;
+    const int32_t rc = product(p, rows, s->m->embedding, b.y32, b.xh, b.xl, out, c.vocab, 0);
+    p.tc = keep;
+    return rc;
+}
+
+bool tracks_positions(const lumi_session* s) { return s->m->n_attn > 0 || s->m->cfg.stacked(); }
+
+// Final norm and tied head of the step's rows (s->x) into s->logits.
+int32_t final_head(StepPlan& p) {
+    lumi_session* s = p.s;
+    const Config& c = s->m->cfg;
+    if (c.stacked()) return listed_head(p, s->dec, nullptr, p.B, s->logits);
+    p.fam = FAM_HEAD;
+    if (p.tc) LUMI_TRY(ensure_norm_input(p, s->x, s->m->final_norm_g));
+    p.fam = FAM_HEAD;
+    return linear(p, s->m->embedding, s->x, c.d_model, s->logits, c.vocab, nullptr, s->m->final_norm_g, 0, c.vocab, true);
+}
+
 // embedding -> blocks -> (final norm -> logits -> sample) -> advance
 // Largest batch of the tensor-core path whose CUDA-core kernels are launched with programmatic dependent launch
 // (LUMI_PDL_TC; 0 = never): the state step then becomes resident under the in_proj GEMM and requests its tiles early.
@@ -771,11 +1187,14 @@ int32_t enqueue_step(lumi_session* s, int B, bool with_head, int64_t* launches,
     struct PdlGemmScope { PdlGemmScope(bool on) { set_launch_pdl_gemm(on); } ~PdlGemmScope() { set_launch_pdl_gemm(false); } } pdl_gemm_scope(s->opt_pdl && prof == nullptr && p.tc && B <= pdl_gemm_max());
     p.st_hi = p.st_lo = s->stream;
     mark(p);
-    LUMI_CUDA(launch_embed(s->m->embedding.p, s->m->embedding.dtype, s->tok_cur, s->x, B, c.d_model, c.vocab, s->ctl, s->stream, row_len));
-    const bool two_lanes = p.tc && prof == nullptr && row_len == nullptr && s->opt_overlap > 0 && B >= s->opt_overlap && s->m->n_attn == 0 && B >= 2;
+    LUMI_CUDA(launch_embed(s->m->embedding.p, s->m->embedding.dtype, s->tok_cur, s->x, B, c.x_ld(), c.vocab, s->ctl, s->stream, row_len,
+                           embed_post_of(s, s->dec, 0, p.tc)));
+    const bool two_lanes = !c.stacked() && p.tc && prof == nullptr && row_len == nullptr && s->opt_overlap > 0 && B >= s->opt_overlap && s->m->n_attn == 0 && B >= 2;
     if (!two_lanes) {
+        RowPass rows{&s->dec, B, 1, 0, row_len, -1};
         for (const Layer& L : s->m->layers) {
-            if (L.is_attn) LUMI_TRY(attention_block(p, L));
+            if (L.spec != nullptr) LUMI_TRY(listed_layer(p, rows, L));
+            else if (L.is_attn) LUMI_TRY(attention_block(p, L));
             else LUMI_TRY(mamba_block(p, L));
         }
     } else {
@@ -818,34 +1237,38 @@ int32_t enqueue_step(lumi_session* s, int B, bool with_head, int64_t* launches,
     if (fused) {
         p.fam = FAM_HEAD;
         int nparts = 0;
-        GemvArgs g{s->x, c.d_model, s->m->embedding.p, s->m->embedding.dtype, nullptr, c.vocab, nullptr, s->m->final_norm_g, B, c.vocab,
-                   c.d_model, c.eps, 0, &s->ctl->status};
+        GemvArgs g{s->x, c.x_ld(), s->m->embedding.p, s->m->embedding.dtype, nullptr, c.vocab, nullptr, s->m->final_norm_g, B, c.vocab,
+                   c.x_ld(), c.eps, 0, &s->ctl->status};
+        if (c.x_ld() != c.d_model) {                      // padded rows: the mean runs over the true width, in a kernel of its own
+            RowNormArgs rn{s->x, nullptr, s->m->final_norm_g, s->dec.y32, nullptr, nullptr, nullptr, B, c.d_model, c.x_ld(), c.eps};
+            mark(p);
+            LUMI_CUDA(launch_row_norm(rn, s->stream));
+            g.A = s->dec.y32;
+            g.gamma = nullptr;
+        }
         g.amax_val = s->amax_val; g.amax_idx = s->amax_idx; g.amax_stride = s->amax_stride; g.amax_parts = &nparts;
         mark(p);
         LUMI_CUDA(launch_gemv(g, s->stream));
         p.fam = FAM_SAMPLE;
         mark(p);
         LUMI_CUDA(launch_head_finish(s->amax_val, s->amax_idx, nparts, s->amax_stride, B, s->ctl, s->tok_cur, s->finished, s->out_len,
-                                     s->m->n_attn > 0 ? s->kv_pos : nullptr, s->stream));
+                                     tracks_positions(s) ? s->kv_pos : nullptr, s->stream));
         *launches = p.n;
         return LUMI_OK;
     }
     if (with_head) {
-        p.fam = FAM_HEAD;
-        if (p.tc) LUMI_TRY(ensure_norm_input(p, s->x, s->m->final_norm_g));
-        p.fam = FAM_HEAD;
-        LUMI_TRY(linear(p, s->m->embedding, s->x, c.d_model, s->logits, c.vocab, nullptr, s->m->final_norm_g, 0, c.vocab, true));
+        LUMI_TRY(final_head(p));
         p.fam = FAM_SAMPLE;
         mark(p);
         LUMI_CUDA(launch_sample(s->logits, B, c.vocab, s->ctl, s->tok_cur, s->finished, s->out_len, s->stream));
     }
     if (row_len != nullptr) {                      // ragged prefill: keep the residual of every sequence that is at its last prompt token
         mark(p);
-        LUMI_CUDA(launch_capture_last(s->x, s->xlast, row_len, s->ctl, B, c.d_model, s->stream));
+        LUMI_CUDA(launch_capture_last(s->x, s->xlast, row_len, s->ctl, B, c.x_ld(), s->stream));
     }
     p.fam = FAM_SAMPLE;
     mark(p);
-    LUMI_CUDA(launch_advance_step(s->ctl, s->m->n_attn > 0 ? s->kv_pos : nullptr, B, with_head ? 1 : 0, s->stream, row_len));
+    LUMI_CUDA(launch_advance_step(s->ctl, tracks_positions(s) ? s->kv_pos : nullptr, B, with_head ? 1 : 0, s->stream, row_len));
     if (prof) {   // closing event
         p.fam = FAM_COUNT;
         mark(p);
@@ -992,6 +1415,7 @@ int32_t grow(T*& p, size_t& cap, size_t need_elems) {
 }
 
 bool use_chunked_prefill(const lumi_session* s, int batch, int T) {
+    if (s->m->cfg.stacked()) return s->opt_chunked_prefill > 0 && T >= 2;       // any element type, windows included: the ring holds a slice more
     if (!(s->opt_chunked_prefill > 0 && T >= s->opt_chunked_prefill && s->m->wdtype == LUMI_DTYPE_BF16 && s->opt_gemm != 1 &&
           prefill_ssd_supported(s->m->cfg) && (s->m->cfg.d_model % 64) == 0 && (s->m->cfg.d_inner() % 64) == 0))
         return false;
@@ -1004,14 +1428,97 @@ bool use_chunked_prefill(const lumi_session* s, int batch, int T) {
     return true;
 }
 
+// Head over a slice's rows, a block of rows at a time, then the log-probability of each row's target (shared by the slice loops).
+int score_block_rows(int V) {
+    return (int)std::min<size_t>(4096, std::max<size_t>(128, ((size_t)256 << 20) / ((size_t)V * sizeof(float)) / 128 * 128));
+}
+
+// The slice loop for designs that list their layers: slices of up to slice_max tokens per sequence, each through every layer
+// with the caches and states carried from slice to slice.  Arguments as for prefill_chunked.
+int32_t prefill_listed(lumi_session* s, int batch, int T, bool with_head, float* score_out, const int32_t* lens, int slot0,
+                       const std::vector<int32_t>* want, float* want_out) {
+    const Config& c = s->m->cfg;
+    const int ldx = c.x_ld(), V = c.vocab;
+    const int nb_max = std::min(batch, 2048);
+    int TS = std::max(64, (std::max(64, s->opt_prefill_rows) / nb_max) / 64 * 64);
+    TS = std::min({TS, s->slice_max, T});
+    const size_t rows_max = (size_t)nb_max * TS;
+    if (rows_max > s->pre.rows) {
+        LUMI_CUDA(cudaStreamSynchronize(s->stream));
+        free_rows(s->pre);
+        LUMI_TRY(alloc_rows(s, s->pre, rows_max, true));
+    }
+    RowBufs& b = s->pre;
+    if (want != nullptr && want->size() > s->want_cap) LUMI_TRY(grow(s->want_idx, s->want_cap, want->size()));
+    size_t wanted = 0;
+    std::vector<int32_t> local;                           // outlives the copies below (synchronised before it changes)
+    for (int b0 = 0; b0 < batch; b0 += nb_max) {
+        const int nb = std::min(nb_max, batch - b0);
+        for (int t0 = 0; t0 < T; t0 += TS) {
+            RowPass r{&b, nb, std::min(TS, T - t0), slot0 + b0, lens, t0};
+            const int M = r.rows();
+            StepPlan p{s, M, use_tc(s, M)};
+            p.st_hi = p.st_lo = s->stream;
+            mark(p);
+            LUMI_CUDA(launch_prefill_embed(s->m->embedding.p, s->m->embedding.dtype, s->prompt_dev, b.x, ldx, V, M, r.ts, t0, b0, batch, s->ctl,
+                                           s->stream, lens, embed_post_of(s, b, slot0 + b0, p.tc)));
+            for (const Layer& L : s->m->layers) LUMI_TRY(listed_layer(p, r, L));
+            mark(p);
+            LUMI_CUDA(launch_kv_advance(s->kv_pos, slot0 + b0, nb, r.ts, s->stream, lens, t0));
+            if (score_out != nullptr) {
+                const int SR = score_block_rows(V);
+                LUMI_TRY(grow(s->score_logits, s->score_logits_cap, (size_t)SR * V));
+                for (int r0 = 0; r0 < M; r0 += SR) {
+                    const int nr = std::min(SR, M - r0);
+                    RowBufs part = b;                     // the head works on the block's rows
+                    part.x = b.x + (size_t)r0 * ldx;
+                    LUMI_TRY(listed_head(p, part, nullptr, nr, s->score_logits));
+                    mark(p);
+                    LUMI_CUDA(launch_logprob_rows(s->score_logits, nr, V, s->prompt_dev, batch, T, r.ts, t0, b0, r0, score_out, s->stream));
+                }
+            }
+            if (want != nullptr) {
+                const size_t first = wanted;
+                while (wanted < want->size() && (*want)[wanted] < t0 + r.ts) ++wanted;
+                if (wanted > first) {
+                    local.assign(want->begin() + first, want->begin() + wanted);
+                    for (int32_t& w : local) w -= t0;
+                    const int nw = (int)local.size();
+                    LUMI_CUDA(cudaMemcpyAsync(s->want_idx, local.data(), sizeof(int32_t) * nw, cudaMemcpyHostToDevice, s->stream));
+                    LUMI_CUDA(cudaStreamSynchronize(s->stream));
+                    LUMI_TRY(listed_head(p, b, s->want_idx, nw, want_out + first * V));
+                }
+            }
+            if (t0 + r.ts >= T || lens != nullptr) {      // different lengths: every slice may hold some sequence's last token
+                mark(p);
+                LUMI_CUDA(launch_gather_last(b.x, s->x, ldx, r.ts, nb, b0, s->stream, lens, t0));
+            }
+            s->launches += p.n;
+        }
+    }
+    if (with_head) {
+        StepPlan p{s, batch, use_tc(s, batch)};
+        p.st_hi = p.st_lo = s->stream;
+        LUMI_TRY(final_head(p));
+        LUMI_CUDA(launch_sample(s->logits, batch, V, s->ctl, s->tok_cur, s->finished, s->out_len, s->stream));
+        LUMI_CUDA(launch_advance_step(s->ctl, nullptr, batch, 1, s->stream));          // positions were advanced slice by slice
+        s->launches += p.n + 2;
+    }
+    return LUMI_OK;
+}
+
 // Prompt of T tokens for sequences 0..batch-1 through the chunked SSD scan; tokens come from
 // prompt_dev[T][batch].  Leaves the decode state of every layer as the step-by-step path would, the
 // last position's residual in x, and (with_head) its logits plus the sampled first token.
 // score_out (device, [batch][T-1]) != null: log p(next prompt token) at every position, from the head over all rows.
 // lens (device, [batch]) != null: prompts of different lengths inside the [T][batch] rectangle (T = the longest): every sequence
 // ends in the state after its own last token, x holds the residual at that token, and padding is never looked at.
-int32_t prefill_chunked(lumi_session* s, int batch, int T, bool with_head, float* score_out = nullptr, const int32_t* lens = nullptr) {
+// slot0: slot of the first sequence (designs that list their layers; 0 otherwise).  want (host, ascending prompt positions, one
+// sequence): logits of those positions go to want_out (device, [n_want][vocab]).
+int32_t prefill_chunked(lumi_session* s, int batch, int T, bool with_head, float* score_out = nullptr, const int32_t* lens = nullptr,
+                        int slot0 = 0, const std::vector<int32_t>* want = nullptr, float* want_out = nullptr) {
     const Config& c = s->m->cfg;
+    if (c.stacked()) return prefill_listed(s, batch, T, with_head, score_out, lens, slot0, want, want_out);
     const int D = c.d_model, DI = c.d_inner(), R = c.in_proj_out();
     const bool hybrid = s->m->n_attn > 0;
     const int KVD = hybrid ? c.kv_dim() : 0, Q = D + 2 * KVD, MLP = hybrid ? c.mlp_dim() : 0;
@@ -1116,7 +1623,7 @@ int32_t prefill_chunked(lumi_session* s, int batch, int T, bool with_head, float
             if (score_out != nullptr) {
                 // final norm + tied head over the rows of the slice, a block of rows at a time, then log-softmax at the target
                 const int V = c.vocab;
-                const int SR = (int)std::min<size_t>(4096, std::max<size_t>(128, ((size_t)256 << 20) / ((size_t)V * sizeof(float)) / 128 * 128));
+                const int SR = score_block_rows(V);
                 LUMI_TRY(grow(s->score_logits, s->score_logits_cap, (size_t)SR * V));
                 LUMI_CUDA(launch_norm_split(s->pf_x, s->m->final_norm_g, s->pf_hi, lo, M, D, c.eps, s->stream));
                 for (int r0 = 0; r0 < M; r0 += SR) {
@@ -1269,19 +1776,54 @@ extern "C" int32_t lumi_prefill_ragged(lumi_session* s, const uint32_t* tokens, 
     }
     if (last_logits) {
         // final norm + tied head on each sequence's residual at its own last token
-        if (!chunked) LUMI_CUDA(cudaMemcpyAsync(s->x, s->xlast, sizeof(float) * batch * s->m->cfg.d_model, cudaMemcpyDeviceToDevice, s->stream));
+        if (!chunked) LUMI_CUDA(cudaMemcpyAsync(s->x, s->xlast, sizeof(float) * batch * s->m->cfg.x_ld(), cudaMemcpyDeviceToDevice, s->stream));
         StepPlan p{s, batch, use_tc(s, batch)};
         p.st_hi = p.st_lo = s->stream;
         const Config& c = s->m->cfg;
-        if (p.tc) LUMI_TRY(ensure_norm_input(p, s->x, s->m->final_norm_g));
-        p.fam = FAM_HEAD;
-        LUMI_TRY(linear(p, s->m->embedding, s->x, c.d_model, s->logits, c.vocab, nullptr, s->m->final_norm_g, 0, c.vocab, true));
+        LUMI_TRY(final_head(p));
         s->launches += p.n;
         LUMI_CUDA(cudaMemcpyAsync(last_logits, s->logits, sizeof(float) * batch * c.vocab, cudaMemcpyDeviceToHost, s->stream));
     }
     LUMI_TRY(pull_ctl(s));
     LUMI_CUDA(cudaStreamSynchronize(s->stream));
     return check_status(s);
+}
+
+// The next tokens of ONE sequence, from whatever state it is in, with the logits of chosen places among them.
+extern "C" int32_t lumi_extend(lumi_session* s, int32_t slot, const uint32_t* tokens, int32_t T, const int32_t* want, int32_t n_want,
+                               float* logits_out) {
+    if (!s) return fail(LUMI_E_INVALID, "session is null");
+    if (slot < 0 || slot >= s->max_batch) return fail(LUMI_E_INVALID, "slot %d out of range [0,%d)", slot, s->max_batch);
+    if (!tokens || T <= 0 || n_want < 0 || (n_want > 0 && (!want || !logits_out))) return fail(LUMI_E_INVALID, "extend needs tokens, T > 0 and an output for what is wanted");
+    for (int i = 0; i < n_want; ++i)
+        if (want[i] < 0 || want[i] >= T || (i > 0 && want[i] <= want[i - 1])) return fail(LUMI_E_INVALID, "wanted places must be ascending and inside the tokens");
+    const Config& c = s->m->cfg;
+    const int V = c.vocab;
+    LUMI_CUDA(cudaSetDevice(s->m->device));
+    s->fused_head = false;
+    if (!c.stacked() && slot != 0) return fail(LUMI_E_UNSUPPORTED, "this design extends the sequence in slot 0 only");
+    if (c.stacked() && (T > 1 || slot != 0)) {
+        LUMI_TRY(upload_prompt(s, tokens, 1, T));
+        if (n_want > 0) LUMI_TRY(grow(s->gen_dump, s->gen_dump_cap, (size_t)n_want * V));
+        fill_ctl(s, 1, nullptr);
+        s->ctl_host->prompt = s->prompt_dev;
+        s->ctl_host->prompt_len = s->ctl_host->prompt_pos = T;
+        LUMI_TRY(push_ctl(s));
+        const std::vector<int32_t> places(want, want + n_want);
+        LUMI_TRY(prefill_chunked(s, 1, T, false, nullptr, nullptr, slot, n_want > 0 ? &places : nullptr, s->gen_dump));
+        if (n_want > 0) LUMI_CUDA(cudaMemcpyAsync(logits_out, s->gen_dump, sizeof(float) * (size_t)n_want * V, cudaMemcpyDeviceToHost, s->stream));
+        LUMI_TRY(pull_ctl(s));
+        LUMI_CUDA(cudaStreamSynchronize(s->stream));
+        return check_status(s);
+    }
+    // a single token, or a design without slices of one sequence: the decode step, token by token
+    const lumi_sampling sp{0.f, 0, 0, 0u, 1};
+    for (int t = 0, w = 0; t < T; ++t) {
+        const bool wanted = w < n_want && want[w] == t;
+        if (wanted) LUMI_TRY(lumi_decode_step(s, tokens + t, 1, &sp, t, nullptr, logits_out + (size_t)w++ * V));
+        else LUMI_TRY(lumi_prefill(s, tokens + t, 1, 1, nullptr));
+    }
+    return LUMI_OK;
 }
 
 // Teacher-forced scoring: log p(tokens[b][t+1] | tokens[b][0..t]) for t = 0 .. T-2, the quantity the reference's
@@ -1421,7 +1963,15 @@ extern "C" int32_t lumi_generate(lumi_session* s, const uint32_t* prompts, int32
         const Config& cf = s->m->cfg;
         const int64_t per_seq = (int64_t)s->m->n_mamba * 2 * 4 *
                                 ((int64_t)state_h_per_seq(cf) + cf.d_inner() + cf.n_heads * cf.d_state + cf.n_heads * (cf.d_state / 2));
-        stats->bytes_per_step = s->m->weight_bytes + (int64_t)batch * per_seq;
+        int64_t listed = 0;                               // listed layers: states read and written, the window's keys and values read
+        for (size_t i = 0; i < s->lstate.size(); ++i) {
+            const LayerState& L = s->lstate[i];
+            const MixerSpec& m = cf.specs[i].mixer;
+            const int64_t esz = s->m->wdtype == LUMI_DTYPE_BF16 ? 2 : 4;
+            if (m.kind == MIXER_DELTA) listed += 2 * 4 * (int64_t)L.s_seq + 4 * (int64_t)L.conv_seq;
+            else listed += esz * m.kv_heads * (L.dk_pad + L.dv_pad) * (int64_t)std::min(m.window > 0 ? m.window : T + n_new / 2, T + n_new / 2);
+        }
+        stats->bytes_per_step = s->m->weight_bytes + (int64_t)batch * (per_seq + listed);
         const int64_t steps = std::max(0, n_new - 1);
         stats->achieved_gbps = (steps > 0 && stats->ms_decode > 0.f) ? (float)((double)stats->bytes_per_step * (double)steps / ((double)stats->ms_decode * 1e-3) / 1e9) : 0.f;
         stats->waves = 1;
@@ -1487,7 +2037,7 @@ extern "C" int32_t lumi_session_read_state(lumi_session* s, int32_t slot, int32_
     if (!s) return fail(LUMI_E_INVALID, "session is null");
     const Config& c = s->m->cfg;
     if (slot < 0 || slot >= s->max_batch) return fail(LUMI_E_INVALID, "slot %d out of range", slot);
-    if (layer < 0 || layer >= c.n_layers || s->m->layers[layer].is_attn) return fail(LUMI_E_INVALID, "layer %d is not a Mamba layer", layer);
+    if (layer < 0 || layer >= c.n_layers || !s->m->layers[layer].is_mamba()) return fail(LUMI_E_INVALID, "layer %d is not a Mamba layer", layer);
     LUMI_CUDA(cudaSetDevice(s->m->device));
     const size_t B = s->max_batch, l = s->m->layers[layer].kind_idx;
     const size_t nh = state_h_per_seq(c), nx = c.d_inner(), nb = (size_t)c.n_heads * c.d_state, nc = (size_t)c.n_heads * (c.d_state / 2);
@@ -1520,6 +2070,7 @@ SnapLayout snap_layout(const lumi_session* s) {
     L.nh = state_h_per_seq(c); L.nx = c.d_inner(); L.nb = (size_t)c.n_heads * c.d_state; L.nc = (size_t)c.n_heads * (c.d_state / 2);
     L.kv_seq_bytes = s->m->n_attn > 0 ? s->kv_layer_bytes / (size_t)s->max_batch : 0;
     L.payload = (size_t)s->m->n_mamba * (L.nh + L.nx + L.nb + L.nc) * sizeof(float) + (size_t)s->m->n_attn * L.kv_seq_bytes;
+    for (const LayerState& S : s->lstate) L.payload += (S.s_seq + S.conv_seq) * sizeof(float) + S.kv_bytes / (size_t)s->max_batch;
     return L;
 }
 }  // namespace
@@ -1547,6 +2098,13 @@ static int32_t snap_copy(lumi_session* s, int32_t slot, char* buf, bool save) {
     }
     for (size_t a = 0; a < (size_t)s->m->n_attn; ++a)      // slot b owns pages [b * pages_per_seq, (b + 1) * pages_per_seq)
         LUMI_CUDA(xfer((char*)s->kv_pool + a * s->kv_layer_bytes + (size_t)slot * L.kv_seq_bytes, L.kv_seq_bytes));
+    for (const LayerState& S : s->lstate) {
+        if (S.S != nullptr) {
+            LUMI_CUDA(xfer(S.S + slot * S.s_seq, S.s_seq * sizeof(float)));
+            LUMI_CUDA(xfer(S.conv + slot * S.conv_seq, S.conv_seq * sizeof(float)));
+        }
+        if (S.kv != nullptr) LUMI_CUDA(xfer((char*)S.kv + (size_t)slot * (S.kv_bytes / B), S.kv_bytes / B));
+    }
     return LUMI_OK;
 }
 
@@ -1557,7 +2115,7 @@ extern "C" int32_t lumi_session_save_state(lumi_session* s, int32_t slot, void* 
     if (nbytes < (int64_t)(sizeof(SnapHeader) + L.payload))
         return fail(LUMI_E_INVALID, "snapshot buffer of %lld bytes, %zu needed", (long long)nbytes, sizeof(SnapHeader) + L.payload);
     LUMI_CUDA(cudaSetDevice(s->m->device));
-    SnapHeader hd{kSnapMagic, 1u, (uint32_t)s->m->n_mamba, (uint32_t)s->m->n_attn, (uint64_t)L.payload, 0, 0u};
+    SnapHeader hd{kSnapMagic, 1u, (uint32_t)(s->m->n_mamba + s->m->n_delta), (uint32_t)(s->m->n_attn + s->m->n_wattn), (uint64_t)L.payload, 0, 0u};
     LUMI_CUDA(cudaMemcpyAsync(&hd.kv_pos, s->kv_pos + slot, sizeof(int32_t), cudaMemcpyDeviceToHost, s->stream));
     LUMI_TRY(snap_copy(s, slot, (char*)host_buf + sizeof(SnapHeader), true));
     LUMI_CUDA(cudaStreamSynchronize(s->stream));
@@ -1573,13 +2131,15 @@ extern "C" int32_t lumi_session_load_state(lumi_session* s, int32_t slot, const 
     if (nbytes < (int64_t)sizeof(hd)) return fail(LUMI_E_INVALID, "snapshot shorter than its header");
     memcpy(&hd, host_buf, sizeof(hd));
     if (hd.magic != kSnapMagic || hd.version != 1u) return fail(LUMI_E_INVALID, "not a sequence snapshot");
-    if (hd.n_mamba != (uint32_t)s->m->n_mamba || hd.n_attn != (uint32_t)s->m->n_attn || hd.payload_bytes != (uint64_t)L.payload)
+    if (hd.n_mamba != (uint32_t)(s->m->n_mamba + s->m->n_delta) || hd.n_attn != (uint32_t)(s->m->n_attn + s->m->n_wattn) || hd.payload_bytes != (uint64_t)L.payload)
         return fail(LUMI_E_TENSOR, "snapshot of another model or cache size (%u Mamba + %u attention layers, %llu bytes; this session: %d + %d, %zu)",
-                    hd.n_mamba, hd.n_attn, (unsigned long long)hd.payload_bytes, s->m->n_mamba, s->m->n_attn, L.payload);
+                    hd.n_mamba, hd.n_attn, (unsigned long long)hd.payload_bytes, s->m->n_mamba + s->m->n_delta, s->m->n_attn + s->m->n_wattn, L.payload);
     if (nbytes < (int64_t)(sizeof(hd) + L.payload)) return fail(LUMI_E_INVALID, "snapshot truncated");
     // the position indexes the page table and the cache: a value outside what this session can hold is refused here
     // (with a sliding window on every attention layer positions may run past the capacity: the ring wraps)
     if (hd.kv_pos < 0) return fail(LUMI_E_INVALID, "snapshot with a negative position (%d)", hd.kv_pos);
+    if (s->kv_limit > 0 && hd.kv_pos > s->kv_limit)
+        return fail(LUMI_E_INVALID, "snapshot at position %d, this session's cache holds %d tokens", hd.kv_pos, s->kv_limit);
     if (s->m->n_attn > 0) {
         bool all_windowed = true;
         for (const Layer& Ly : s->m->layers) if (Ly.is_attn && !(Ly.window > 0 && Ly.window <= s->max_tokens_kv)) all_windowed = false;
@@ -1600,17 +2160,25 @@ extern "C" int32_t lumi_debug_run_block(lumi_session* s, int32_t layer, float* x
     LUMI_CUDA(cudaSetDevice(s->m->device));
     fill_ctl(s, batch, nullptr);
     LUMI_TRY(push_ctl(s));
-    LUMI_CUDA(cudaMemcpyAsync(s->x, x, sizeof(float) * batch * c.d_model, cudaMemcpyHostToDevice, s->stream));
+    const size_t row = sizeof(float) * c.d_model, pitch = sizeof(float) * c.x_ld();
+    LUMI_CUDA(cudaMemcpy2DAsync(s->x, pitch, x, row, row, batch, cudaMemcpyHostToDevice, s->stream));
     StepPlan p{s, batch, use_tc(s, batch)};
     p.st_hi = p.st_lo = s->stream;
     const Layer& L = s->m->layers[layer];
-    if (L.is_attn) {
+    if (L.spec != nullptr) {
+        // positions stay where they are: the caller runs one layer after the other for the same token, and the last
+        // layer ends the token
+        if (p.tc) LUMI_CUDA(launch_norm_split(s->x, nullptr, s->dec.xh, s->opt_split ? s->dec.xl : nullptr, batch, c.x_ld(), c.eps, s->stream));
+        RowPass r{&s->dec, batch, 1, 0, nullptr, -1};
+        LUMI_TRY(listed_layer(p, r, L));
+        if (layer == c.n_layers - 1) LUMI_CUDA(launch_advance_step(s->ctl, s->kv_pos, batch, 0, s->stream));
+    } else if (L.is_attn) {
         LUMI_TRY(attention_block(p, L));
         LUMI_CUDA(launch_advance_step(s->ctl, s->kv_pos, batch, 0, s->stream));
     } else {
         LUMI_TRY(mamba_block(p, L));
     }
-    LUMI_CUDA(cudaMemcpyAsync(x, s->x, sizeof(float) * batch * c.d_model, cudaMemcpyDeviceToHost, s->stream));
+    LUMI_CUDA(cudaMemcpy2DAsync(x, row, s->x, pitch, row, batch, cudaMemcpyDeviceToHost, s->stream));
     LUMI_TRY(pull_ctl(s));
     LUMI_CUDA(cudaStreamSynchronize(s->stream));
     return check_status(s);

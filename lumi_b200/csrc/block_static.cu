@@ -54,7 +54,7 @@ extern "C" int32_t lumi_mamba_block_static(lumi_model* m, int32_t layer, uint64_
     if (!m || !x || !h || !x_prev || !b_prev || !cum_angle) return fail(LUMI_E_INVALID, "null argument to lumi_mamba_block_static");
     if (!m->finalized) return fail(LUMI_E_INVALID, "lumi_model_finalize must succeed first");
     const Config& c = m->cfg;
-    if (layer < 0 || layer >= c.n_layers || m->layers[layer].is_attn) return fail(LUMI_E_INVALID, "layer %d is not a Mamba layer", layer);
+    if (layer < 0 || layer >= c.n_layers || !m->layers[layer].is_mamba()) return fail(LUMI_E_INVALID, "layer %d is not a Mamba layer", layer);
     const int R = c.in_proj_out(), DI = c.d_inner(), D = c.d_model;
     if (batch < 1 || batch > kStaticMaxBatch)
         return fail(LUMI_E_UNSUPPORTED, "lumi_mamba_block_static: batch %d outside [1, %d] (fixed scratch; use a session for larger batches)", batch, kStaticMaxBatch);

@@ -263,6 +263,15 @@ __device__ __forceinline__ void mbar_arrive(uint64_t* bar) {
     asm volatile("mbarrier.arrive.shared::cta.b64 _, [%0];" ::"r"(smem_u32(bar)) : "memory");
 }
 
+// activation in the epilogue (NormFuse::act)
+__device__ __forceinline__ float epi_act(float v, int act) {
+    if (act == 2) { v = fmaxf(v, 0.f); v *= v; }
+    return v;
+}
+__device__ __forceinline__ float4 gamma4(const float* gamma, int col) {
+    return gamma != nullptr ? __ldg(reinterpret_cast<const float4*>(gamma + col)) : make_float4(1.f, 1.f, 1.f, 1.f);
+}
+
 template <int BN, bool SPLIT>
 __global__ void __launch_bounds__(192, 1)
 gemm_persistent_kernel(const __grid_constant__ CUtensorMap map_ahi, const __grid_constant__ CUtensorMap map_alo,
@@ -475,19 +484,20 @@ gemm_persistent_kernel(const __grid_constant__ CUtensorMap map_ahi, const __grid
 #pragma unroll
                                     for (int s2 = 1; s2 < kMaxSplits; ++s2)
                                         if (s2 < splits) { sum.x += pv[s2][j].x; sum.y += pv[s2][j].y; sum.z += pv[s2][j].z; sum.w += pv[s2][j].w; }
-                                    v[4 * j] = fmaf(sum.x, rs, o[j].x); v[4 * j + 1] = fmaf(sum.y, rs, o[j].y);
-                                    v[4 * j + 2] = fmaf(sum.z, rs, o[j].z); v[4 * j + 3] = fmaf(sum.w, rs, o[j].w);
+                                    v[4 * j] = epi_act(fmaf(sum.x, rs, o[j].x), nf.act); v[4 * j + 1] = epi_act(fmaf(sum.y, rs, o[j].y), nf.act);
+                                    v[4 * j + 2] = epi_act(fmaf(sum.z, rs, o[j].z), nf.act); v[4 * j + 3] = epi_act(fmaf(sum.w, rs, o[j].w), nf.act);
                                 }
+                                if (D != nullptr)
 #pragma unroll
-                                for (int j = 0; j < 4; ++j) *reinterpret_cast<float4*>(dp + 4 * j) = make_float4(v[4 * j], v[4 * j + 1], v[4 * j + 2], v[4 * j + 3]);
+                                    for (int j = 0; j < 4; ++j) *reinterpret_cast<float4*>(dp + 4 * j) = make_float4(v[4 * j], v[4 * j + 1], v[4 * j + 2], v[4 * j + 3]);
                             } else {
                                 for (int e = 0; e < 16; ++e) {
                                     v[e] = 0.f;
                                     if (col + e < nlim) {
                                         float sum = 0.f;
                                         for (int s2 = 0; s2 < splits; ++s2) sum += __ldcg(scratch + ((size_t)(s2 * ntiles + t) * BM + row_l) * BN + c16 + e);
-                                        v[e] = fmaf(sum, rs, acc_in ? __ldcg(dp + e) : 0.f);
-                                        dp[e] = v[e];
+                                        v[e] = epi_act(fmaf(sum, rs, acc_in ? __ldcg(dp + e) : 0.f), nf.act);
+                                        if (D != nullptr) dp[e] = v[e];
                                     }
                                 }
                             }
@@ -497,8 +507,7 @@ gemm_persistent_kernel(const __grid_constant__ CUtensorMap map_ahi, const __grid
 #pragma unroll
                                 for (int g8 = 0; g8 < 16; g8 += 8) {
                                     if (col + g8 < nlim) {
-                                        const float4 ga = __ldg(reinterpret_cast<const float4*>(nf.gamma_next + col + g8));
-                                        const float4 gb = __ldg(reinterpret_cast<const float4*>(nf.gamma_next + col + g8 + 4));
+                                        const float4 ga = gamma4(nf.gamma_next, col + g8), gb = gamma4(nf.gamma_next, col + g8 + 4);
                                         const float gg[8] = {ga.x, ga.y, ga.z, ga.w, gb.x, gb.y, gb.z, gb.w};
                                         uint32_t hw[4], lw[4];
 #pragma unroll
@@ -517,7 +526,7 @@ gemm_persistent_kernel(const __grid_constant__ CUtensorMap map_ahi, const __grid
                                         if (nf.out_lo != nullptr) *reinterpret_cast<uint4*>(nf.out_lo + oo) = make_uint4(lw[0], lw[1], lw[2], lw[3]);
                                     }
                                 }
-                                if (((col + 16) & 31) == 0 || col + 16 >= nlim) { nf.ssq_out[(size_t)row * nf.ssq_stride + (col >> 5)] = ssq; ssq = 0.f; }
+                                if (nf.ssq_out != nullptr && (((col + 16) & 31) == 0 || col + 16 >= nlim)) { nf.ssq_out[(size_t)row * nf.ssq_stride + (col >> 5)] = ssq; ssq = 0.f; }
                             }
                         }
                     }
@@ -543,15 +552,16 @@ gemm_persistent_kernel(const __grid_constant__ CUtensorMap map_ahi, const __grid
                         float4 v[8];
 #pragma unroll
                         for (int j = 0; j < 8; ++j)
-                            v[j] = make_float4(fmaf(__uint_as_float(r[4 * j]), rs, o[j].x), fmaf(__uint_as_float(r[4 * j + 1]), rs, o[j].y),
-                                               fmaf(__uint_as_float(r[4 * j + 2]), rs, o[j].z), fmaf(__uint_as_float(r[4 * j + 3]), rs, o[j].w));
+                            v[j] = make_float4(epi_act(fmaf(__uint_as_float(r[4 * j]), rs, o[j].x), nf.act), epi_act(fmaf(__uint_as_float(r[4 * j + 1]), rs, o[j].y), nf.act),
+                                               epi_act(fmaf(__uint_as_float(r[4 * j + 2]), rs, o[j].z), nf.act), epi_act(fmaf(__uint_as_float(r[4 * j + 3]), rs, o[j].w), nf.act));
                         if (nf.out_hi != nullptr) {
                             // the next RMSNorm's input for the next product: x * gamma as bf16 hi + lo (16-byte stores), and x^2 summed
                             float4 gm[8];
 #pragma unroll
-                            for (int j = 0; j < 8; ++j) gm[j] = __ldg(reinterpret_cast<const float4*>(nf.gamma_next + col0 + 4 * j));
+                            for (int j = 0; j < 8; ++j) gm[j] = gamma4(nf.gamma_next, col0 + 4 * j);
+                            if (D != nullptr)
 #pragma unroll
-                            for (int j = 0; j < 8; ++j) *reinterpret_cast<float4*>(dp + 4 * j) = v[j];
+                                for (int j = 0; j < 8; ++j) *reinterpret_cast<float4*>(dp + 4 * j) = v[j];
 #pragma unroll
                             for (int jj = 0; jj < 4; ++jj) {
                                 uint32_t hw[4], lw[4];
@@ -580,10 +590,11 @@ gemm_persistent_kernel(const __grid_constant__ CUtensorMap map_ahi, const __grid
                             if (col0 + j < nlim) {
                                 float v = __uint_as_float(r[j]) * rs;
                                 if (acc_in) v += __ldcg(dp + j);
-                                dp[j] = v;
+                                v = epi_act(v, nf.act);
+                                if (D != nullptr) dp[j] = v;
                                 if (nf.out_hi != nullptr) {
                                     ssq = fmaf(v, v, ssq);
-                                    const float w0 = v * nf.gamma_next[col0 + j];
+                                    const float w0 = nf.gamma_next != nullptr ? v * nf.gamma_next[col0 + j] : v;
                                     const __nv_bfloat16 hh = __float2bfloat16_rn(w0);
                                     nf.out_hi[(size_t)row * N + col0 + j] = hh;
                                     if (nf.out_lo != nullptr) nf.out_lo[(size_t)row * N + col0 + j] = __float2bfloat16_rn(w0 - __bfloat162float(hh));
@@ -591,7 +602,7 @@ gemm_persistent_kernel(const __grid_constant__ CUtensorMap map_ahi, const __grid
                             }
                         }
                     }
-                    if (nf.out_hi != nullptr) nf.ssq_out[(size_t)row * nf.ssq_stride + (col0 >> 5)] = ssq;
+                    if (nf.ssq_out != nullptr) nf.ssq_out[(size_t)row * nf.ssq_stride + (col0 >> 5)] = ssq;
                 }
             }
             tc_fence_before();
@@ -779,8 +790,10 @@ int32_t launch_gemm_tcgen05(const GemmArgs& a, cudaStream_t st) {
         return fail(LUMI_E_INVALID, "tcgen05 GEMM operands must be 16-byte aligned");
     LUMI_TRY(gemm_tcgen05_init());
     const bool split = a.a_lo != nullptr;
-    const bool fused = a.nf.ssq_in != nullptr || a.nf.out_hi != nullptr;
-    if (a.nf.out_hi != nullptr && ((a.N & 7) != 0 || a.nf.gamma_next == nullptr || a.nf.ssq_out == nullptr || a.nf.ssq_stride * 32 < a.N))
+    const bool fused = a.nf.ssq_in != nullptr || a.nf.out_hi != nullptr || a.nf.act != 0;
+    if (a.nf.out_hi != nullptr && a.nf.gamma_next == nullptr && a.nf.ssq_out == nullptr) {
+        if ((a.N & 7) != 0) return fail(LUMI_E_INVALID, "a result in bf16 halves needs N %% 8 == 0");
+    } else if (a.nf.out_hi != nullptr && ((a.N & 7) != 0 || a.nf.gamma_next == nullptr || a.nf.ssq_out == nullptr || a.nf.ssq_stride * 32 < a.N))
         return fail(LUMI_E_INVALID, "folded RMSNorm output needs N %% 8 == 0, the next norm's weights and room for N / 32 partial sums per row");
     // LUMI_GEMM_MODE (tuning aid): 0 = default choice, 1 = 128-wide tiles two CTAs per SM, 2 = 128-wide one CTA per SM,
     // 3 = 256-wide one CTA per SM

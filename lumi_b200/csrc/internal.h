@@ -30,6 +30,41 @@ int32_t fail(int32_t code, const char* fmt, ...);
     } while (0)
 
 // ---- configuration (ModelConfig of the reference, inference/src/model.rs:20-86) -----------------
+// One layer of a model whose config lists its layers one by one: a mixer and, behind it, an optional feed-forward, each
+// followed by a norm of its OUTPUT before it joins the residual stream.  Every mixer constant is a field here, so that
+// another design can combine them differently.
+enum MixerKind { MIXER_NONE = 0, MIXER_DELTA, MIXER_ATTENTION };
+struct MixerSpec {
+    MixerKind kind = MIXER_NONE;
+    int heads = 0, kv_heads = 0, dim = 0, vdim = 0;
+    int taps = 1;              // delta rule: length of the short convolutions
+    float unit_eps = 1e-6f;    // delta rule: epsilon inside the root of the unit vectors
+    float scale = 1.f;         // attention: factor of the scores
+    int window = 0;            // attention: tokens a position sees, itself included (0 = all)
+    int kv_from = -1;          // attention: layer whose keys and values are read (-1 = this layer's own)
+    bool qk_norm = false;      // attention: q and k over their root mean square
+    bool sink = false;         // attention: one score of `sink_score` without a value joins the softmax
+    float sink_score = 0.f;
+};
+struct LayerSpec {
+    MixerSpec mixer;
+    int ff = 0;                // width of the squared-ReLU feed-forward (0 = none)
+};
+
+struct Config;
+struct JsonValue;
+// A model design: how its config.json is read and what its tensors are called.  `name` is the config's "architecture";
+// a config without that key is the Mamba-3 / attention hybrid.
+struct Architecture {
+    const char* name;
+    const char* tensor_prefix;                            // names without it are not looked at ("" = every name counts)
+    int32_t (*parse)(const JsonValue& root, Config& out);
+    // shape of a tensor by its name (prefix removed); rank 0 = not a tensor of this model.  `wide` is set for tensors
+    // that are kept in fp32 whatever their rank
+    int (*expected_shape)(const Config& c, const std::string& name, int64_t shp[2], bool& wide);
+};
+const Architecture* find_architecture(const char* name);  // null if there is none of that name
+
 struct Config {
     int d_model = 0, n_layers = 0, d_state = 0, expand = 0, n_heads = 0, n_groups = 0, vocab = 0, max_seq_len = 0;
     int attention_interval = 0, attn_n_heads = 16, attn_kv_heads = 4, attn_mlp_expand = 4;
@@ -38,9 +73,23 @@ struct Config {
     int attn_mlp_dim = 0;        // extension: 0 = attn_mlp_expand * d_model
     float attn_rope_base = 0.f;  // extension: 0 = no rotary embedding in attention
     float eps = 1e-5f;           // the reference hard-codes 1e-5 (model.rs:97) and has no norm_eps key
+    const Architecture* arch = nullptr;
+    std::vector<LayerSpec> specs;          // one entry per layer for designs that list them; empty for the hybrid
+    float embed_scale = 1.f;
+    bool embed_positions = false;          // sinusoidal position vectors are added to the embedding
+
+    bool stacked() const { return !specs.empty(); }
+    // elements per row of the residual stream on the device: rows of listed designs are padded with zeros to whole
+    // 64-element blocks, so that any width goes through the tensor-core products
+    int x_ld() const { return stacked() ? (d_model + 63) / 64 * 64 : d_model; }
+    int max_window() const {               // most tokens an attention layer looks back over; 0 = one of them sees all
+        int w = 1;
+        for (const LayerSpec& l : specs) if (l.mixer.kind == MIXER_ATTENTION) { if (l.mixer.window <= 0) return 0; if (l.mixer.window > w) w = l.mixer.window; }
+        return w;
+    }
 
     int d_inner() const { return expand * d_model; }
-    int head_dim() const { return d_inner() / n_heads; }
+    int head_dim() const { return n_heads > 0 ? d_inner() / n_heads : 0; }
     int bc() const { return n_groups * d_state; }
     int in_proj_out() const { return 2 * d_inner() + 2 * bc() + 3 * n_heads + n_heads * d_state / 2; }
     int attn_head_dim() const { return d_model / attn_n_heads; }
@@ -72,12 +121,24 @@ struct AttnW {
     const float *attn_norm_g = nullptr, *mlp_norm_g = nullptr;
     DevTensor qkv, o, gate_up, down;     // q|k|v and gate|up rows concatenated at finalize
 };
+// Weights of a listed layer.  `in` holds the input projections stacked by rows, each part padded to a multiple of 8 rows;
+// columns (and the stacked total) are padded to multiples of 64 with zeros.  Norm weights are stored as the factor itself.
+struct SubW {
+    DevTensor in, out, up, down;
+    int off_q = 0, off_k = 0, off_v = 0, off_b = 0, off_a = 0, off_g = 0;
+    const float *conv_q = nullptr, *conv_k = nullptr, *conv_v = nullptr;      // [channels][taps]
+    const float *a_log = nullptr, *dt_bias = nullptr, *o_norm = nullptr;
+    const float *norm1 = nullptr, *norm2 = nullptr;                           // [x_ld]
+};
 struct Layer {
     bool is_attn = false;
     int kind_idx = 0;     // index among the Mamba layers, or among the attention layers
     int window = 0;
     MambaW m;
     AttnW a;
+    const LayerSpec* spec = nullptr;      // set for layers of a design that lists them; `s` then holds the weights
+    SubW s;
+    bool is_mamba() const { return !is_attn && spec == nullptr; }
 };
 
 }  // namespace lumi
@@ -87,12 +148,14 @@ struct lumi_model {
     int device = 0;
     bool finalized = false;
     int wdtype = -1;                                  // dtype of rank-2 tensors (all must agree)
+    bool widen = false;                               // bf16 tensors are widened to fp32 when they are loaded
     std::map<std::string, lumi::DevTensor> tensors;   // by name without the "item." prefix
     std::vector<void*> owned;                         // extra device allocations made at finalize
     std::vector<lumi::Layer> layers;
     lumi::DevTensor embedding;
     const float* final_norm_g = nullptr;
     int n_mamba = 0, n_attn = 0;
+    int n_delta = 0, n_wattn = 0;                     // listed layers by mixer
     int64_t weight_bytes = 0;                         // bytes of weights one decode step reads
 };
 
@@ -127,7 +190,26 @@ struct GraphEntry {
 
 }  // namespace lumi
 
-namespace lumi { struct B1Layer; }
+namespace lumi {
+struct B1Layer;
+// Per-sequence state of one listed layer for all slots of a session.
+struct LayerState {
+    void* kv = nullptr;         // attention: page pool [slot pages][kv_head][K rows | V rows of 64 tokens], rows padded to dk_pad / dv_pad
+    size_t kv_bytes = 0;
+    int dk_pad = 0, dv_pad = 0;
+    float* S = nullptr;         // delta rule: [slot][head][dim][dv_pad]
+    float* conv = nullptr;      // delta rule: [slot][taps][channels] raw inputs of the short convolutions, ring over positions
+    int dvp = 0, channels = 0;
+    size_t s_seq = 0, conv_seq = 0;      // floats per sequence
+};
+// Row buffers of a pass over listed layers (one set for decode steps, one for prompt slices).
+struct RowBufs {
+    size_t rows = 0;
+    float *x = nullptr;                              // residual stream [rows][x_ld] (the decode set uses the session's x)
+    float *proj = nullptr, *mix = nullptr, *qkv = nullptr, *gates = nullptr, *y32 = nullptr;
+    __nv_bfloat16 *xh = nullptr, *xl = nullptr, *ah = nullptr, *al = nullptr;
+};
+}
 
 struct lumi_session {
     lumi_model* m = nullptr;
@@ -176,6 +258,13 @@ struct lumi_session {
     int32_t* row_len = nullptr;        // [max_batch] prompt lengths of a ragged prefill
     float* xlast = nullptr;            // [max_batch][d_model] residual rows at each sequence's last prompt token
     int pages_per_seq = 0;
+    // designs that list their layers
+    std::vector<lumi::LayerState> lstate;
+    lumi::RowBufs dec, pre;
+    int kv_limit = 0;                  // positions at or past it are refused (0 = the ring takes any)
+    int slice_max = 0;                 // most tokens of a sequence per pass (what the ring leaves beside the widest window)
+    double* pos_freq = nullptr;        // [d_model / 2] frequencies of the position vectors
+    int32_t* want_idx = nullptr; size_t want_cap = 0;
     // activations
     float *x = nullptr, *proj = nullptr, *y32 = nullptr, *logits = nullptr;
     __nv_bfloat16 *act_hi = nullptr, *act_lo = nullptr;
@@ -215,7 +304,7 @@ struct GemvArgs {
     const float* gamma;              // RMSNorm weight applied to rows of A first, or null
     int M, N, K;
     float eps;
-    int act;                         // 0 none; 1: D = sigmoid(W_gate a) * (W_up a), W = [gate rows | up rows], N = rows of each
+    int act;                         // 0 none; 1: D = sigmoid(W_gate a) * (W_up a), W = [gate rows | up rows], N = rows of each; 2: D = max(0, W a)^2
     int32_t* status = nullptr;       // device word that receives STATUS_TIMEOUT if a bounded wait gives up; may be null
     bool allow_preload = true;       // false: never the single-wave preloading kernel (the only GEMV with a device-side wait)
     // greedy head: per (batch row, CTA) the best (value, row) of the CTA's rows goes to amax_val / amax_idx
@@ -239,8 +328,18 @@ bool launch_pdl_on();
 void set_launch_pdl_gemm(bool on);
 bool launch_pdl_gemm_on();
 
+// What some designs do to an embedding row before it becomes the residual stream: a factor, a sinusoidal position vector
+// (freq: [width / 2], pos: position of each sequence's first row in this pass), and the bf16 halves of the result for the
+// first product.  The defaults leave the row as the table holds it.
+struct EmbedPost {
+    float scale = 1.f;
+    const double* freq = nullptr;
+    const int32_t* pos = nullptr;
+    int width = 0;
+    __nv_bfloat16 *hi = nullptr, *lo = nullptr;
+};
 cudaError_t launch_embed(const void* emb, int dtype, const uint32_t* tok_cur, float* x, int B, int D, int vocab,
-                         StepCtl* ctl, cudaStream_t st, const int32_t* row_len = nullptr);
+                         StepCtl* ctl, cudaStream_t st, const int32_t* row_len = nullptr, const EmbedPost& post = EmbedPost());
 // x[B][D] fp32 -> RMSNorm(gamma) -> bf16 hi (+ lo if lo != null); gamma null = plain split.
 // ssq != null: hi / lo = x * gamma without the per-row scale, ssq[b * ssq_stride] = sum of x^2 (for a GEMM with a folded norm)
 cudaError_t launch_norm_split(const float* x, const float* gamma, __nv_bfloat16* hi, __nv_bfloat16* lo, int B, int D,
@@ -323,6 +422,9 @@ struct NormFuse {
     const float* gamma_next = nullptr;
     __nv_bfloat16 *out_hi = nullptr, *out_lo = nullptr;
     float* ssq_out = nullptr;
+    // activation before the result is stored: 0 none, 2 max(0, v)^2.  With gamma_next null, out_hi / out_lo receive the
+    // result itself (width N) and no sums of squares are written; D may then be null
+    int act = 0;
 };
 
 struct GemmArgs {
@@ -388,9 +490,65 @@ struct PrefillArgs {
 };
 bool prefill_ssd_supported(const Config& c);
 cudaError_t launch_prefill_embed(const void* emb, int dtype, const uint32_t* prompt, float* x, int D, int vocab, int rows, int ts,
-                                 int t_abs0, int b_abs0, int batch_total, StepCtl* ctl, cudaStream_t st, const int32_t* lens = nullptr);
+                                 int t_abs0, int b_abs0, int batch_total, StepCtl* ctl, cudaStream_t st, const int32_t* lens = nullptr,
+                                 const EmbedPost& post = EmbedPost());
 cudaError_t launch_prefill_scan(const PrefillArgs& a, cudaStream_t st);
 cudaError_t launch_gather_last(const float* xr, float* x, int D, int ts, int nb, int b0, cudaStream_t st, const int32_t* lens = nullptr, int t_abs0 = 0);
+
+// ---- listed layers: norm of a sublayer's output into the residual stream (sublayer.cu) --------------------
+// x[r] += o[r] / sqrt(mean(o[r]^2) + eps) * w over `width` elements (rows of ld elements, padding stays zero); with hi set,
+// the new residual also goes out as bf16 halves for the next product.  o == null: rows of x are normalised into y32 and / or
+// hi / lo instead and x is left alone; row_idx (device, may be null) then picks the rows of x.
+struct RowNormArgs {
+    float* x; const float* o; const float* w;
+    float* y32; __nv_bfloat16 *hi, *lo;
+    const int32_t* row_idx;
+    int rows, width, ld;
+    float eps;
+};
+cudaError_t launch_row_norm(const RowNormArgs& a, cudaStream_t st);
+
+// ---- gated delta rule (delta_rule.cu) ----------------------------------------------------------------------
+// Rows of the stacked input projections; row r = sequence b0 + r / ts, token r % ts of this pass.
+struct DeltaArgs {
+    const float* proj; int ldp;
+    int off_q, off_k, off_v, off_b, off_a, off_g;
+    const float *conv_q, *conv_k, *conv_v;           // [channels][taps]; channels of the ring: q | k | v
+    const float *a_log, *dt_bias, *o_norm;
+    float* S; float* conv;                           // this layer's state, slot 0
+    int H, G, dk, dv, dvp, taps;
+    float eps, unit_eps;
+    const int32_t* pos;                              // [slot] position of the pass's first token
+    const int32_t* row_len; int t_abs0;              // prompts of different lengths (null otherwise), as in PrefillArgs
+    const StepCtl* ctl;                              // decode form (ts == 1) with row_len: the step's prompt position decides
+    int nseq, ts, b0;
+    float* y32; __nv_bfloat16 *yhi, *ylo; int ldy;   // gated, normalised output rows
+    // chunked form: prepared q | k | v rows (unit vectors, activations applied), [rows][2 G dk + H dv] padded, and per (row, head)
+    // beta and the logarithm of the decay; the read-out before its norm
+    float* qkv; int ldqkv; float* gates; float* o32;
+};
+cudaError_t launch_delta_step(const DeltaArgs& a, cudaStream_t st, int* launches);
+bool delta_chunk_supported(int dk, int dv);
+cudaError_t launch_delta_chunk(const DeltaArgs& a, cudaStream_t st, int* launches);
+
+// ---- windowed attention with a softmax sink (window_attention.cu) -----------------------------------------
+struct WinAttnArgs {
+    const float* proj; int ldp; int off_q, off_k, off_v;
+    void* kv; int kv_is_f32; int dk_pad, dv_pad;
+    const int32_t* page_table; int pages_per_seq;    // ring of pages_per_seq pages per slot
+    const int32_t* pos;                              // [slot] position of the pass's first token
+    int H, G, dk, dv;
+    MixerSpec m;
+    int append;                                      // 0: the keys and values are another layer's and already in the cache
+    float eps;
+    const int32_t* row_len; int t_abs0; StepCtl* ctl;
+    int nseq, ts, b0;
+    int limit;                                       // positions at or past it are refused (0 = the ring takes any)
+    float* y32; __nv_bfloat16 *yhi, *ylo; int ldy;
+    float* part; int32_t* part_count;                // as in AttnArgs, decode only
+};
+cudaError_t launch_window_attention(const WinAttnArgs& a, cudaStream_t st, int* launches);
+size_t window_attention_part_floats(const MixerSpec& m);      // room for the partial results of one (row, head group)
 
 cudaError_t launch_gate_mul(const float* gu, int ld, float* out32, __nv_bfloat16* hi, __nv_bfloat16* lo, int B, int mlp,
                             cudaStream_t st);

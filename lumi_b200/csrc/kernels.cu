@@ -7,6 +7,7 @@
 // products use FMA with a fixed summation order (per-lane strided partials, xor-shuffle tree), so
 // results are bit-stable from run to run.
 #include "internal.h"
+#include "embed_post.cuh"
 #include <type_traits>
 
 #include <cfloat>
@@ -97,7 +98,7 @@ template <> struct WLoad<__nv_bfloat16> {
 // ---- embedding gather (model.rs:772-773) -----------------------------------------------------------
 template <typename WT>
 __global__ void embed_kernel(const WT* __restrict__ emb, const uint32_t* tok_cur, float* x,
-                             int D, int vocab, StepCtl* ctl, const int32_t* row_len) {
+                             int D, int vocab, StepCtl* ctl, const int32_t* row_len, EmbedPost post) {
     const int b = blockIdx.x;
     pdl_launch_dependents();
     pdl_wait();
@@ -116,8 +117,18 @@ __global__ void embed_kernel(const WT* __restrict__ emb, const uint32_t* tok_cur
     for (int c = threadIdx.x; c < D / E; c += blockDim.x) {
         float w[E];
         WLoad<WT>::load(row + c * E, w);
+        embed_post<E>(post, w, c * E, post.pos != nullptr ? post.pos[b] : 0);
 #pragma unroll
         for (int e = 0; e < E; ++e) x[(size_t)b * D + c * E + e] = w[e];
+        if (post.hi != nullptr) {
+#pragma unroll
+            for (int e = 0; e < E; ++e) {
+                __nv_bfloat16 hh, ll;
+                split_bf16(w[e], hh, ll);
+                post.hi[(size_t)b * D + c * E + e] = hh;
+                if (post.lo != nullptr) post.lo[(size_t)b * D + c * E + e] = ll;
+            }
+        }
     }
 }
 
@@ -311,6 +322,7 @@ __global__ void __launch_bounds__(256) gemv_kernel(const float* A, int lda, cons
                 if (b >= nb) break;
                 float v = acc[r][b];
                 if constexpr (ACT == 1) v = __fmul_rn(sigmoid_ref(v), acc[RPW + r][b]);     // model.rs:550-552
+                if constexpr (ACT == 2) { v = fmaxf(v, 0.f); v = __fmul_rn(v, v); }
                 size_t o = (size_t)(m0 + b) * ldd + row;
                 if (R != nullptr) v = __fadd_rn(v, R[o]);
                 if (D != nullptr) D[o] = v;
@@ -1283,7 +1295,7 @@ static cudaError_t launch_k(void (*kern)(KArgs...), dim3 grid, dim3 block, size_
 }
 
 cudaError_t launch_embed(const void* emb, int dtype, const uint32_t* tok_cur, float* x, int B, int D, int vocab,
-                         StepCtl* ctl, cudaStream_t st, const int32_t* row_len) {
+                         StepCtl* ctl, cudaStream_t st, const int32_t* row_len, const EmbedPost& post) {
     // The first kernel of a step is never launched early: it starts only when the previous step has
     // completely finished, which is what lets later kernels of this step read state ahead of their
     // own dependency wait.
@@ -1291,9 +1303,9 @@ cudaError_t launch_embed(const void* emb, int dtype, const uint32_t* tok_cur, fl
     g_pdl = false;
     cudaError_t e;
     if (dtype == LUMI_DTYPE_BF16)
-        e = launch_k(embed_kernel<__nv_bfloat16>, dim3(B), dim3(128), 0, st, (const __nv_bfloat16*)emb, tok_cur, x, D, vocab, ctl, row_len);
+        e = launch_k(embed_kernel<__nv_bfloat16>, dim3(B), dim3(128), 0, st, (const __nv_bfloat16*)emb, tok_cur, x, D, vocab, ctl, row_len, post);
     else
-        e = launch_k(embed_kernel<float>, dim3(B), dim3(128), 0, st, (const float*)emb, tok_cur, x, D, vocab, ctl, row_len);
+        e = launch_k(embed_kernel<float>, dim3(B), dim3(128), 0, st, (const float*)emb, tok_cur, x, D, vocab, ctl, row_len, post);
     g_pdl = keep;
     return e;
 }
@@ -1335,10 +1347,20 @@ static cudaError_t gemv_dispatch(const GemvArgs& a, cudaStream_t st) {
 
 template <typename WT>
 static cudaError_t gemv_by_batch(const GemvArgs& a, cudaStream_t st) {
+    if (a.M > 1 && (size_t)a.K * sizeof(float) * (a.M > 4 ? 8 : 4) > 200 * 1024) {      // the staged rows have to fit: fewer of them per CTA
+        if (a.act == 1) return gemv_dispatch<WT, 1, 1>(a, st);
+        if (a.act == 2) return gemv_dispatch<WT, 1, 2>(a, st);
+        return gemv_dispatch<WT, 1, 0>(a, st);
+    }
     if (a.act == 1) {
         if (a.M <= 1) return gemv_dispatch<WT, 1, 1>(a, st);
         if (a.M <= 2) return gemv_dispatch<WT, 2, 1>(a, st);
         return gemv_dispatch<WT, 4, 1>(a, st);
+    }
+    if (a.act == 2) {
+        if (a.M <= 1) return gemv_dispatch<WT, 1, 2>(a, st);
+        if (a.M <= 4) return gemv_dispatch<WT, 4, 2>(a, st);
+        return gemv_dispatch<WT, 8, 2>(a, st);
     }
     if (a.M <= 1) return gemv_dispatch<WT, 1, 0>(a, st);
     if (a.M <= 2) return gemv_dispatch<WT, 2, 0>(a, st);

@@ -34,6 +34,7 @@
 //   * The pointwise part (softplus / sigmoid / tanh / SiLU / sin / cos) uses the fast hardware forms here: their
 //     error (~1e-6) is far below the operand split's (1.5e-5) — the decode step keeps the exact forms.
 #include "internal.h"
+#include "embed_post.cuh"
 
 #include <cuda.h>
 
@@ -175,10 +176,15 @@ constexpr uint32_t kChunkTxBytes = 3 * LCH * 32 * 4 + 2 * LCH * 64 * 4;
 // row r = b * ts + t  of the super-chunk; token ids come from prompt[(t_abs) * batch_total + b_abs]
 template <typename WT>
 __global__ void embed_rows_kernel(const WT* __restrict__ emb, const uint32_t* __restrict__ prompt, float* __restrict__ x, int D,
-                                  int vocab, int ts, int t_abs0, int b_abs0, int batch_total, StepCtl* ctl, const int32_t* __restrict__ lens) {
+                                  int vocab, int ts, int t_abs0, int b_abs0, int batch_total, StepCtl* ctl, const int32_t* __restrict__ lens,
+                                  EmbedPost post) {
     const int r = blockIdx.x, b = r / ts, t = r - b * ts;
     if (lens != nullptr && t_abs0 + t >= lens[b_abs0 + b]) {      // padding behind a shorter prompt: never looked at, the row is zero
-        for (int k = threadIdx.x; k < D; k += blockDim.x) x[(size_t)r * D + k] = 0.f;
+        for (int k = threadIdx.x; k < D; k += blockDim.x) {
+            x[(size_t)r * D + k] = 0.f;
+            if (post.hi != nullptr) post.hi[(size_t)r * D + k] = __float2bfloat16_rn(0.f);
+            if (post.lo != nullptr) post.lo[(size_t)r * D + k] = __float2bfloat16_rn(0.f);
+        }
         return;
     }
     uint32_t tok = prompt[(size_t)(t_abs0 + t) * batch_total + b_abs0 + b];
@@ -188,7 +194,14 @@ __global__ void embed_rows_kernel(const WT* __restrict__ emb, const uint32_t* __
         float v;
         if (sizeof(WT) == 4) v = reinterpret_cast<const float*>(row)[k];
         else v = __uint_as_float((uint32_t)reinterpret_cast<const uint16_t*>(row)[k] << 16);
-        x[(size_t)r * D + k] = v;
+        float one[1] = {v};
+        embed_post<1>(post, one, k, post.pos != nullptr ? post.pos[b] + t : 0);
+        x[(size_t)r * D + k] = one[0];
+        if (post.hi != nullptr) {
+            const __nv_bfloat16 hh = __float2bfloat16_rn(one[0]);
+            post.hi[(size_t)r * D + k] = hh;
+            if (post.lo != nullptr) post.lo[(size_t)r * D + k] = __float2bfloat16_rn(one[0] - __bfloat162float(hh));
+        }
     }
 }
 
@@ -644,11 +657,11 @@ bool prefill_ssd_supported(const Config& c) {
 }
 
 cudaError_t launch_prefill_embed(const void* emb, int dtype, const uint32_t* prompt, float* x, int D, int vocab, int rows, int ts,
-                                 int t_abs0, int b_abs0, int batch_total, StepCtl* ctl, cudaStream_t st, const int32_t* lens) {
+                                 int t_abs0, int b_abs0, int batch_total, StepCtl* ctl, cudaStream_t st, const int32_t* lens, const EmbedPost& post) {
     if (dtype == LUMI_DTYPE_BF16)
-        embed_rows_kernel<__nv_bfloat16><<<rows, 128, 0, st>>>((const __nv_bfloat16*)emb, prompt, x, D, vocab, ts, t_abs0, b_abs0, batch_total, ctl, lens);
+        embed_rows_kernel<__nv_bfloat16><<<rows, 128, 0, st>>>((const __nv_bfloat16*)emb, prompt, x, D, vocab, ts, t_abs0, b_abs0, batch_total, ctl, lens, post);
     else
-        embed_rows_kernel<float><<<rows, 128, 0, st>>>((const float*)emb, prompt, x, D, vocab, ts, t_abs0, b_abs0, batch_total, ctl, lens);
+        embed_rows_kernel<float><<<rows, 128, 0, st>>>((const float*)emb, prompt, x, D, vocab, ts, t_abs0, b_abs0, batch_total, ctl, lens, post);
     return cudaGetLastError();
 }
 

@@ -53,7 +53,7 @@ extern "C" int32_t lumi_model_load_safetensors(lumi_model* m, const char* path) 
                 if (dt->str == "F32") dtype = LUMI_DTYPE_F32;
                 else if (dt->str == "BF16") dtype = LUMI_DTYPE_BF16;
                 else {
-                    if (kv.first.rfind("item.", 0) != 0) continue;
+                    if (kv.first.rfind(m->cfg.arch != nullptr ? m->cfg.arch->tensor_prefix : "item.", 0) != 0) continue;
                     status = fail(LUMI_E_TENSOR, "tensor '%s': dtype %s not supported (F32, BF16)", kv.first.c_str(), dt->str.c_str());
                     break;
                 }

@@ -250,3 +250,14 @@ BENCH_CONFIGS = {
                 dict(temperature=0.8, top_k=50, seed=1234), 0),
     "config5": (dict(n_layers=96, byte_level=True), "bf16", 2048, 512, 256, dict(), 1000),
 }
+
+
+def config_from_json(text: str):
+    """The configuration class a config.json asks for: registered designs by their "architecture", else ModelConfig."""
+    from . import zozonex
+    name = json.loads(text).get("architecture")
+    if name is None:
+        return ModelConfig.from_json(text)
+    if name == zozonex.ARCHITECTURE:
+        return zozonex.ZozonexConfig.from_json(text)
+    raise ValueError(f"architecture {name!r} is not known")
