@@ -282,6 +282,81 @@ def scan_compare(nb=64, T=2048, reps=3):
     return out
 
 
+# --workload zozonex: (name, width, layers, delta heads / kv heads / dim / vdim, attention heads / kv heads / dim, window, ff) beside the
+# hybrid of the same width, depth, state size per layer, attention heads and feed-forward parameters.  Every sixth layer is attention.
+ZOZONEX_SIZES = {
+    "w1024": (1024, 12, (16, 16, 64, 128), (16, 4, 64), 1024, 4224),
+    "w2048": (2048, 6, (16, 16, 128, 128), (32, 8, 64), 1024, 8448),
+}
+ZOZONEX_VOCAB = 32000
+
+
+def zozonex_pair(name):
+    """(Zozonex config and tensors, hybrid config and tensors) of one size; bf16 weights."""
+    from lumi_b200 import zozonex as zz
+    width, n, (H, G, dk, dv), (ah, ag, ad), window, ff = ZOZONEX_SIZES[name]
+    layers, shared = [], None
+    for i in range(n):
+        if (i + 1) % 6:
+            layers.append(zz.delta(H, dk, dv, kv_heads=G))
+        else:                                    # the second attention layer of a pair reads the first one's keys and values
+            layers.append(zz.attention(ah, ad, window, kv_heads=ag, ff=ff, kv_from=shared))
+            shared = i if shared is None else None
+    zcfg = zz.config(width, ZOZONEX_VOCAB, layers, max_seq_len=8192)
+    hcfg = synth.base_config(d_model=width, n_layers=n, n_heads=2 * width // 32, vocab_size=ZOZONEX_VOCAB, attention_interval=6, attn_n_heads=ah,
+                             attn_kv_heads=ag, attn_mlp_dim=2 * ff // 3, max_seq_len=8192)
+    return (zcfg, zz.iter_tensors(zcfg, seed=0)), (hcfg, synth.iter_tensors(hcfg, seed=0, weights_dtype="bf16"))
+
+
+def run_zozonex(args, rank, local_rank, world):
+    """Prefill and decode throughput of the Zozonex design beside the Mamba-3 / attention hybrid of equal size: CUDA events inside
+    the library, random weights, greedy decode; device times by kernel family from one profiled step."""
+    if rank != 0:
+        return
+    import lumi_b200
+    peak_gbs, peak_src = measured_peak_gbs()
+    out = []
+    sampler = ClockSampler(local_rank)
+    sampler.start()
+    for name in (args.zozonex_sizes.split(",") if args.zozonex_sizes else ZOZONEX_SIZES):
+        entry = {"size": name}
+        for kind, (cfg, tens) in zip(("zozonex", "hybrid"), zozonex_pair(name)):
+            model = lumi_b200.NmModel.from_tensors(cfg, tens, device=local_rank)
+            runs = {"weight_bytes": model.info()["weight_bytes"]}
+            for batch, T in ((1, 2048), (16, 2048), (64, 512), (512, 128)):
+                if args.zozonex_batch and batch != args.zozonex_batch:
+                    continue
+                sess = model.init_states(batch, T + 256)
+                prompts = synth.random_prompts(batch, T, cfg.vocab_size, seed=1)
+                sess.generate(prompts, 3, ignore_eos=True)                 # warm-up: buffers, graphs, attributes
+                best_p, best_d = None, None
+                for _ in range(3):
+                    sess.reset()
+                    _, _, _, st = sess.generate(prompts, 2, ignore_eos=True)
+                    best_p = st.ms_prefill if best_p is None else min(best_p, st.ms_prefill)
+                    sess.decode_loop_device(batch, 3)
+                    ms, launches = sess.decode_loop_device(batch, args.steps)
+                    best_d = ms if best_d is None else min(best_d, ms)
+                sess.profile_step(batch)
+                fam = sess.profile_step(batch)
+                runs[f"batch{batch}"] = {
+                    "prompt_tokens": T, "prefill_tok_s": batch * T / (best_p * 1e-3), "prefill_ms": best_p,
+                    "decode_tok_s": batch * args.steps / (best_d * 1e-3), "decode_ms_per_step": best_d / args.steps,
+                    "launches_per_step": launches / args.steps, "step_bytes": int(st.bytes_per_step),
+                    "step_frac_of_hbm": st.bytes_per_step / (best_d / args.steps * 1e-3) / 1e9 / peak_gbs,
+                    "family_ms": {k: round(v[0], 4) for k, v in fam.items()}}
+                sess.close()
+            model.close()
+            entry[kind] = runs
+        out.append(entry)
+    clocks = sampler.stop()
+    big = out[-1]["zozonex"][list(out[-1]["zozonex"])[-1]]
+    print(json.dumps({"metric": METRIC, "value": big["decode_tok_s"], "unit": UNIT, "n_gpus": 1, "steps": args.steps, "warmup": 3,
+                      "ms_per_step": big["decode_ms_per_step"], "higher_is_better": True, "scaling": "strong", "vs_baseline": None, "dtype": "bf16",
+                      "data": "synthetic", "config": {"workload": "zozonex: decode and prefill beside the hybrid of equal size", "peak_gbs": peak_gbs,
+                                                      "peak_source": peak_src}, "sizes": out, "clocks": clocks}), flush=True)
+
+
 def run_named_config(args, rank, local_rank, world):
     """The other benchmark configurations, one GPU, through Session.generate (prefill + decode timed
     by CUDA events inside the library).  Sequences would shard over ranks exactly as in the sweep."""
@@ -486,7 +561,9 @@ def main():
     ap.add_argument("--no-batch1", action="store_true")
     ap.add_argument("--only-batch1", action="store_true", help="run just the batch-1 figure (profiling)")
     ap.add_argument("--b1-layers", type=int, default=48)
-    ap.add_argument("--workload", default="sweep", choices=["sweep", "scan"] + sorted(CONFIGS))
+    ap.add_argument("--workload", default="sweep", choices=["sweep", "scan", "zozonex"] + sorted(CONFIGS))
+    ap.add_argument("--zozonex-sizes", default="", help="--workload zozonex: only these sizes (commas between them)")
+    ap.add_argument("--zozonex-batch", type=int, default=0, help="--workload zozonex: only this batch")
     ap.add_argument("--scan-seqs", type=int, default=64, help="--workload scan: sequences")
     ap.add_argument("--scan-tokens", type=int, default=2048, help="--workload scan: tokens per sequence")
     ap.add_argument("--steps-override", type=int, default=0, help="decode tokens for --workload configN (0 = the configuration's own)")
@@ -499,6 +576,8 @@ def main():
             import torch
             torch.cuda.set_device(local_rank)
             print(json.dumps({"prefill_scan": scan_compare(args.scan_seqs, args.scan_tokens)}), flush=True)
+    elif args.workload == "zozonex":
+        run_zozonex(args, rank, local_rank, world)
     elif args.workload != "sweep":
         run_named_config(args, rank, local_rank, world)
     elif args.only_batch1:

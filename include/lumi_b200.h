@@ -273,6 +273,35 @@ int32_t lumi_k_ssd_prefill(uint64_t proj, int32_t ldp, uint64_t b_gamma, uint64_
                            uint64_t y_hi, uint64_t y_lo, uint64_t scratch, int32_t nb, int32_t ts, int32_t H, int32_t G,
                            uint64_t stream);
 
+/* The gated delta rule alone, from the rows of its stacked input projections to the gated, normalised output rows, for
+ * `nseq` sequences x `ts` tokens (row = sequence * ts + token).  proj[rows][ldp] holds q at off[0] (kv_heads x dk), k at off[1],
+ * v at off[2] (heads x dv), the step size's logit at off[3] (heads), the decay's input at off[4] (heads), the gate at off[5]
+ * (heads x dv).  conv_*: [channels][taps], last column = current token.  State, updated in place: S[nseq][heads][dk][dv rounded up to 4]
+ * and ring[nseq][taps][2 kv_heads dk + heads dv] (slot = position % taps); pos[nseq]: position of each sequence's first row.
+ * chunked = 0: token after token in fp32; 1: chunks of 64 tokens on the tensor cores, which needs scratch of
+ * rows * (2 kv_heads round4(dk) + 2 heads round4(dv) + 2 heads) floats.  y[rows][heads * dv]. */
+int32_t lumi_k_delta_rule(uint64_t proj, int32_t ldp, const int32_t* off, uint64_t conv_q, uint64_t conv_k, uint64_t conv_v, uint64_t a_log,
+                          uint64_t dt_bias, uint64_t o_norm, uint64_t S, uint64_t ring, uint64_t pos, uint64_t y, uint64_t scratch,
+                          int32_t heads, int32_t kv_heads, int32_t dk, int32_t dv, int32_t taps, float eps, int32_t nseq, int32_t ts,
+                          int32_t chunked, uint64_t stream);
+
+/* Windowed attention alone: appends the keys (over their root mean square when qk_norm) and values of nseq x ts rows to a paged
+ * ring and lets every row attend to the `window` positions that end with its own (0 = all).  proj[rows][ldp]: q at off[0]
+ * (heads x dk), k at off[1], v at off[2] (append = 0: the ring is another layer's and already complete).  sink: the softmax has
+ * one more score, 0, without a value.  kv: [page][kv_head][K 64 x round16(dk) | V 64 x round16(dv)], fp32 or bf16;
+ * page_table[nseq][pages_per_seq]; position p lives in ring slot p % (64 pages_per_seq), so window + ts - 1 must fit.
+ * y[rows][heads * dv]. */
+int32_t lumi_k_window_attention(uint64_t proj, int32_t ldp, const int32_t* off, uint64_t kv, int32_t kv_dtype, uint64_t page_table,
+                                int32_t pages_per_seq, uint64_t pos, uint64_t y, int32_t heads, int32_t kv_heads, int32_t dk, int32_t dv,
+                                int32_t window, float scale, int32_t qk_norm, int32_t sink, float eps, int32_t append, int32_t nseq,
+                                int32_t ts, uint64_t stream);
+
+/* x[r] += o[r] / sqrt(mean(o[r]^2) + eps) * w over `width` elements of rows of ld elements (ld % 4 == 0, padding zero in all
+ * three); hi / lo (may be 0) receive the new rows as bf16 halves.  o = 0: x is left alone and y (fp32) / hi / lo receive its
+ * normalised rows. */
+int32_t lumi_k_norm_add(uint64_t x, uint64_t o, uint64_t w, uint64_t y, uint64_t hi, uint64_t lo, int32_t rows, int32_t width, int32_t ld,
+                        float eps, uint64_t stream);
+
 /* One Mamba block (RMSNorm -> in_proj -> state step -> out_proj + residual, inference/src/model.rs:296-375
  * in arithmetic) WITHOUT any allocation.  This entry point has no counterpart in the reference.
  *

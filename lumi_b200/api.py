@@ -25,7 +25,8 @@ EXPORTS = [
     "lumi_model_finalize", "lumi_model_free", "lumi_model_info", "lumi_session_create", "lumi_session_reset",
     "lumi_session_free", "lumi_session_set_option", "lumi_prefill", "lumi_prefill_ragged", "lumi_extend", "lumi_model_set_option", "lumi_decode_step", "lumi_generate",
     "lumi_decode_loop_device", "lumi_profile_step", "lumi_score", "lumi_session_read_state", "lumi_session_state_bytes", "lumi_session_save_state", "lumi_session_load_state", "lumi_debug_run_block", "lumi_k_gemm_bf16_tcgen05",
-    "lumi_k_gemv", "lumi_debug_gemm_wait_timeout", "lumi_debug_gemm_plan", "lumi_k_ssm_step", "lumi_k_ssd_prefill", "lumi_mamba_block_static",
+    "lumi_k_gemv", "lumi_debug_gemm_wait_timeout", "lumi_debug_gemm_plan", "lumi_k_ssm_step", "lumi_k_ssd_prefill", "lumi_k_delta_rule",
+    "lumi_k_window_attention", "lumi_k_norm_add", "lumi_mamba_block_static",
 ]
 
 
@@ -88,6 +89,11 @@ def lib():
         L.lumi_debug_gemm_wait_timeout.argtypes = [u64, u64, u64, i32, i32, i32, u64, i32, u64]
         L.lumi_debug_gemm_plan.argtypes = [i32, i32, i32, i32, i32, C.POINTER(C.c_int32), C.POINTER(C.c_int32)]
         L.lumi_k_ssd_prefill.argtypes = [u64, i32] + [u64] * 13 + [i32] * 4 + [u64]
+        f32, ip = C.c_float, C.c_void_p
+        L.lumi_k_delta_rule.argtypes = [u64, i32, ip] + [u64] * 11 + [i32] * 5 + [f32] + [i32] * 3 + [u64]
+        L.lumi_k_window_attention.argtypes = ([u64, i32, ip, u64, i32, u64, i32, u64, u64] + [i32] * 5 + [f32, i32, i32, f32]
+                                              + [i32] * 3 + [u64])
+        L.lumi_k_norm_add.argtypes = [u64] * 6 + [i32] * 3 + [f32, u64]
         L.lumi_mamba_block_static.argtypes = [vp, i32, u64, u64, u64, u64, u64, i32, u64]
         _lib = L
     return _lib

@@ -458,7 +458,7 @@ extern "C" int32_t lumi_model_info(const lumi_model* m, int64_t* o) {
 static size_t state_h_per_seq(const Config& c) { return (size_t)c.n_heads * c.head_dim() * c.d_state; }
 
 static void free_rows(RowBufs& b) {
-    void* all[] = {b.x, b.proj, b.mix, b.qkv, b.gates, b.y32, b.xh, b.xl, b.ah, b.al};
+    void* all[] = {b.x, b.x2, b.proj, b.mix, b.qkv, b.gates, b.y32, b.xh, b.xl, b.ah, b.al};
     for (void* p : all) if (p) cudaFree(p);
     b = RowBufs();
 }
@@ -494,6 +494,7 @@ static int32_t alloc_rows(lumi_session* s, RowBufs& b, size_t rows, bool slices)
     if (b.x == nullptr) LUMI_TRY(get(b.x, rp * ldx));
     LUMI_TRY(get(b.proj, rp * w.proj));
     LUMI_TRY(get(b.mix, rp * w.mix));
+    LUMI_TRY(get(b.x2, std::min<size_t>(rp, 8) * ldx));
     LUMI_TRY(get(b.y32, (half && s->opt_gemm != 1 ? std::min<size_t>(rp, 8) : rp) * std::max(w.act, ldx)));
     if (half) {
         LUMI_TRY(get(b.xh, rp * ldx));
@@ -1013,6 +1014,9 @@ struct RowPass {
     int nseq, ts, b0;
     const int32_t* row_len;      // prompts of different lengths (null otherwise)
     int t_abs0;                  // first prompt position of a slice; -1 = decode form (the step's prompt position decides)
+    // few rows on the weight-streaming path: b->mix still has to join the residual stream, under this norm weight; the next
+    // product's prologue does it (x and x2 of the row buffers change places)
+    const float* pending = nullptr;
     int rows() const { return nseq * ts; }
 };
 
@@ -1031,12 +1035,13 @@ EmbedPost embed_post_of(const lumi_session* s, const RowBufs& b, int slot0, bool
 // D = act(A W^T) over `rows` rows: tensor cores from the bf16 halves, or the weight-streaming kernel from fp32 rows.  The result
 // goes to out32, or (tensor cores, out_hi given) as bf16 halves only.
 int32_t product(StepPlan& p, int rows, const DevTensor& W, const float* in32, const __nv_bfloat16* hi, const __nv_bfloat16* lo, float* out32,
-                int ldd, int act, __nv_bfloat16* out_hi = nullptr, __nv_bfloat16* out_lo = nullptr) {
+                int ldd, int act, __nv_bfloat16* out_hi = nullptr, __nv_bfloat16* out_lo = nullptr, const PostAdd& post = PostAdd()) {
     lumi_session* s = p.s;
     const int N = (int)W.rows, K = (int)W.cols;
     mark(p);
     if (!p.tc) {
         GemvArgs g{in32, K, W.p, W.dtype, out32, ldd, nullptr, nullptr, rows, N, K, s->m->cfg.eps, act, &s->ctl->status};
+        g.post = post;
         const cudaError_t e = launch_gemv(g, p.st_hi);
         if (e == cudaErrorInvalidValue) return fail(LUMI_E_UNSUPPORTED, "a product over %d inputs is longer than the streaming kernel takes", K);
         LUMI_CUDA(e);
@@ -1051,15 +1056,28 @@ int32_t product(StepPlan& p, int rows, const DevTensor& W, const float* in32, co
 }
 
 // The residual stream takes the norm of a sublayer's output; on the tensor-core path its bf16 halves are renewed as well.
-int32_t add_normed(StepPlan& p, RowPass& r, const float* w) {
+int32_t add_normed(StepPlan& p, RowPass& r, const float* w, float* settle_to = nullptr) {
     const Config& c = p.s->m->cfg;
     RowBufs& b = *r.b;
-    RowNormArgs a{b.x, b.mix, w, nullptr, p.tc ? b.xh : nullptr, p.tc && p.s->opt_split ? b.xl : nullptr, nullptr, r.rows(), c.d_model, c.x_ld(), c.eps};
+    r.pending = nullptr;
+    if (settle_to == nullptr && !p.tc && r.rows() <= 8) { r.pending = w; return LUMI_OK; }
+    RowNormArgs a{b.x, b.mix, w, nullptr, p.tc ? b.xh : nullptr, p.tc && p.s->opt_split ? b.xl : nullptr, nullptr, r.rows(), c.d_model, c.x_ld(), c.eps, settle_to};
     const int fam = p.fam;
     p.fam = FAM_NORM;
     mark(p);
     LUMI_CUDA(launch_row_norm(a, p.st_hi));
     p.fam = fam;
+    return LUMI_OK;
+}
+
+// A product of the residual stream, which first takes what is pending.
+int32_t product_of_x(StepPlan& p, RowPass& r, const DevTensor& W, float* out32, int ldd, int act, __nv_bfloat16* out_hi = nullptr,
+                     __nv_bfloat16* out_lo = nullptr) {
+    RowBufs& b = *r.b;
+    PostAdd post;
+    if (r.pending != nullptr) { post.o = b.mix; post.w = r.pending; post.x_out = b.x2; post.width = p.s->m->cfg.d_model; }
+    LUMI_TRY(product(p, r.rows(), W, b.x, b.xh, b.xl, out32, ldd, act, out_hi, out_lo, post));
+    if (r.pending != nullptr) { std::swap(b.x, b.x2); r.pending = nullptr; }
     return LUMI_OK;
 }
 
@@ -1073,7 +1091,7 @@ int32_t listed_layer(StepPlan& p, RowPass& r, const Layer& L) {
     __nv_bfloat16* al = p.tc && s->opt_split ? b.al : nullptr;
     float* y32 = p.tc ? nullptr : b.y32;
     p.fam = m.kind == MIXER_DELTA ? FAM_IN_PROJ : FAM_ATTN;
-    LUMI_TRY(product(p, rows, L.s.in, b.x, b.xh, b.xl, b.proj, (int)L.s.in.rows, 0));
+    LUMI_TRY(product_of_x(p, r, L.s.in, b.proj, (int)L.s.in.rows, 0));
     int n = 0;
     if (m.kind == MIXER_DELTA) {
         const LayerState& S = s->lstate[li];
@@ -1089,6 +1107,7 @@ int32_t listed_layer(StepPlan& p, RowPass& r, const Layer& L) {
         a.nseq = r.nseq; a.ts = r.ts; a.b0 = r.b0;
         a.y32 = y32; a.yhi = ah; a.ylo = al; a.ldy = (int)L.s.out.cols;
         a.qkv = b.qkv; a.ldqkv = 2 * m.kv_heads * ((m.dim + 3) / 4 * 4) + m.heads * S.dvp; a.gates = b.gates; a.o32 = b.mix;
+        a.status = &s->ctl->status;
         p.fam = FAM_SSM;
         mark(p);
         // short slices and fp32 models go token by token (the chunked form's products are tf32 terms)
@@ -1121,10 +1140,18 @@ int32_t listed_layer(StepPlan& p, RowPass& r, const Layer& L) {
     LUMI_TRY(add_normed(p, r, L.s.norm1));
     if (L.spec->ff > 0) {
         p.fam = FAM_ATTN;
-        LUMI_TRY(product(p, rows, L.s.up, b.x, b.xh, b.xl, b.y32, (int)L.s.up.rows, 2, ah, b.al));
+        LUMI_TRY(product_of_x(p, r, L.s.up, b.y32, (int)L.s.up.rows, 2, ah, b.al));
         LUMI_TRY(product(p, rows, L.s.down, b.y32, b.ah, b.al, b.mix, ldx, 0));
         LUMI_TRY(add_normed(p, r, L.s.norm2));
     }
+    return LUMI_OK;
+}
+
+// What is still pending joins the residual stream in a kernel of its own; the stream ends up in `x`, one of the two buffers.
+int32_t settle(StepPlan& p, RowPass& r, float* x) {
+    if (r.pending == nullptr) return LUMI_OK;
+    LUMI_TRY(add_normed(p, r, r.pending, x));
+    if (r.b->x != x) std::swap(r.b->x, r.b->x2);
     return LUMI_OK;
 }
 
@@ -1134,8 +1161,15 @@ int32_t listed_head(StepPlan& p, RowBufs& b, const int32_t* row_idx, int rows, f
     const Config& c = s->m->cfg;
     const bool tc = use_tc(s, rows);
     RowNormArgs a{b.x, nullptr, s->m->final_norm_g, tc ? nullptr : b.y32, tc ? b.xh : nullptr, tc && s->opt_split ? b.xl : nullptr, row_idx, rows,
-                  c.d_model, c.x_ld(), c.eps};
+                  c.d_model, c.x_ld(), c.eps, nullptr};
     p.fam = FAM_HEAD;
+    if (!tc && row_idx == nullptr && c.d_model == c.x_ld()) {           // the norm rides in the product's prologue
+        GemvArgs g{b.x, c.d_model, s->m->embedding.p, s->m->embedding.dtype, out, c.vocab, nullptr, s->m->final_norm_g, rows, c.vocab, c.d_model,
+                   c.eps, 0, &s->ctl->status};
+        mark(p);
+        LUMI_CUDA(launch_gemv(g, p.st_hi));
+        return LUMI_OK;
+    }
     mark(p);
     LUMI_CUDA(launch_row_norm(a, p.st_hi));
     const bool keep = p.tc;
@@ -1191,12 +1225,14 @@ int32_t enqueue_step(lumi_session* s, int B, bool with_head, int64_t* launches,
                            embed_post_of(s, s->dec, 0, p.tc)));
     const bool two_lanes = !c.stacked() && p.tc && prof == nullptr && row_len == nullptr && s->opt_overlap > 0 && B >= s->opt_overlap && s->m->n_attn == 0 && B >= 2;
     if (!two_lanes) {
-        RowPass rows{&s->dec, B, 1, 0, row_len, -1};
+        RowBufs bufs = s->dec;                            // a copy: x and x2 change places inside a step only
+        RowPass rows{&bufs, B, 1, 0, row_len, -1};
         for (const Layer& L : s->m->layers) {
             if (L.spec != nullptr) LUMI_TRY(listed_layer(p, rows, L));
             else if (L.is_attn) LUMI_TRY(attention_block(p, L));
             else LUMI_TRY(mamba_block(p, L));
         }
+        LUMI_TRY(settle(p, rows, s->x));
     } else {
         // Two lanes of sequences run the whole layer chain independently.  The GEMMs (tensor pipe,
         // shared memory) of one lane are meant to run under the state step (HBM) of the other, so
@@ -1240,7 +1276,7 @@ int32_t enqueue_step(lumi_session* s, int B, bool with_head, int64_t* launches,
         GemvArgs g{s->x, c.x_ld(), s->m->embedding.p, s->m->embedding.dtype, nullptr, c.vocab, nullptr, s->m->final_norm_g, B, c.vocab,
                    c.x_ld(), c.eps, 0, &s->ctl->status};
         if (c.x_ld() != c.d_model) {                      // padded rows: the mean runs over the true width, in a kernel of its own
-            RowNormArgs rn{s->x, nullptr, s->m->final_norm_g, s->dec.y32, nullptr, nullptr, nullptr, B, c.d_model, c.x_ld(), c.eps};
+            RowNormArgs rn{s->x, nullptr, s->m->final_norm_g, s->dec.y32, nullptr, nullptr, nullptr, B, c.d_model, c.x_ld(), c.eps, nullptr};
             mark(p);
             LUMI_CUDA(launch_row_norm(rn, s->stream));
             g.A = s->dec.y32;
@@ -1462,7 +1498,9 @@ int32_t prefill_listed(lumi_session* s, int batch, int T, bool with_head, float*
             mark(p);
             LUMI_CUDA(launch_prefill_embed(s->m->embedding.p, s->m->embedding.dtype, s->prompt_dev, b.x, ldx, V, M, r.ts, t0, b0, batch, s->ctl,
                                            s->stream, lens, embed_post_of(s, b, slot0 + b0, p.tc)));
+            float* const stream = b.x;
             for (const Layer& L : s->m->layers) LUMI_TRY(listed_layer(p, r, L));
+            LUMI_TRY(settle(p, r, stream));
             mark(p);
             LUMI_CUDA(launch_kv_advance(s->kv_pos, slot0 + b0, nb, r.ts, s->stream, lens, t0));
             if (score_out != nullptr) {
@@ -2171,6 +2209,7 @@ extern "C" int32_t lumi_debug_run_block(lumi_session* s, int32_t layer, float* x
         if (p.tc) LUMI_CUDA(launch_norm_split(s->x, nullptr, s->dec.xh, s->opt_split ? s->dec.xl : nullptr, batch, c.x_ld(), c.eps, s->stream));
         RowPass r{&s->dec, batch, 1, 0, nullptr, -1};
         LUMI_TRY(listed_layer(p, r, L));
+        LUMI_TRY(settle(p, r, s->x));
         if (layer == c.n_layers - 1) LUMI_CUDA(launch_advance_step(s->ctl, s->kv_pos, batch, 0, s->stream));
     } else if (L.is_attn) {
         LUMI_TRY(attention_block(p, L));
@@ -2290,5 +2329,64 @@ extern "C" int32_t lumi_k_ssd_prefill(uint64_t proj, int32_t ldp, uint64_t b_gam
     a.yhi = (__nv_bfloat16*)y_hi; a.ylo = (__nv_bfloat16*)y_lo;
     a.H = H; a.G = G; a.ts = ts; a.nb = nb; a.b0 = 0; a.eps = 1e-5f;
     LUMI_CUDA(launch_prefill_scan(a, (cudaStream_t)stream));
+    return LUMI_OK;
+}
+
+extern "C" int32_t lumi_k_delta_rule(uint64_t proj, int32_t ldp, const int32_t* off, uint64_t conv_q, uint64_t conv_k, uint64_t conv_v,
+                                     uint64_t a_log, uint64_t dt_bias, uint64_t o_norm, uint64_t S, uint64_t ring, uint64_t pos, uint64_t y,
+                                     uint64_t scratch, int32_t heads, int32_t kv_heads, int32_t dk, int32_t dv, int32_t taps, float eps,
+                                     int32_t nseq, int32_t ts, int32_t chunked, uint64_t stream) {
+    if (!proj || !off || !conv_q || !conv_k || !conv_v || !a_log || !dt_bias || !o_norm || !S || !ring || !pos || !y || (chunked && !scratch))
+        return fail(LUMI_E_INVALID, "null pointer to lumi_k_delta_rule");
+    if (heads <= 0 || kv_heads <= 0 || heads % kv_heads || dk <= 0 || dv <= 0 || taps <= 0 || nseq <= 0 || ts <= 0 || ldp <= 0 ||
+        (chunked && !delta_chunk_supported(dk, dv)))
+        return fail(LUMI_E_UNSUPPORTED, "unsupported shape for lumi_k_delta_rule");
+    DeltaArgs a{};
+    a.proj = (const float*)proj; a.ldp = ldp;
+    a.off_q = off[0]; a.off_k = off[1]; a.off_v = off[2]; a.off_b = off[3]; a.off_a = off[4]; a.off_g = off[5];
+    a.conv_q = (const float*)conv_q; a.conv_k = (const float*)conv_k; a.conv_v = (const float*)conv_v;
+    a.a_log = (const float*)a_log; a.dt_bias = (const float*)dt_bias; a.o_norm = (const float*)o_norm;
+    a.S = (float*)S; a.conv = (float*)ring;
+    a.H = heads; a.G = kv_heads; a.dk = dk; a.dv = dv; a.dvp = (dv + 3) / 4 * 4; a.taps = taps;
+    a.eps = eps; a.unit_eps = MixerSpec().unit_eps;
+    a.pos = (const int32_t*)pos; a.nseq = nseq; a.ts = ts;
+    a.y32 = (float*)y; a.ldy = heads * dv;
+    const size_t rows = (size_t)nseq * ts;
+    a.ldqkv = 2 * kv_heads * ((dk + 3) / 4 * 4) + heads * a.dvp;
+    a.qkv = (float*)scratch; a.o32 = a.qkv + rows * a.ldqkv; a.gates = a.o32 + rows * heads * a.dvp;
+    int n = 0;
+    const cudaError_t e = chunked ? launch_delta_chunk(a, (cudaStream_t)stream, &n) : launch_delta_step(a, (cudaStream_t)stream, &n);
+    if (e == cudaErrorInvalidValue) return fail(LUMI_E_UNSUPPORTED, "delta-rule heads of %d x %d are not built", dk, dv);
+    LUMI_CUDA(e);
+    return LUMI_OK;
+}
+
+extern "C" int32_t lumi_k_window_attention(uint64_t proj, int32_t ldp, const int32_t* off, uint64_t kv, int32_t kv_dtype, uint64_t page_table,
+                                           int32_t pages_per_seq, uint64_t pos, uint64_t y, int32_t heads, int32_t kv_heads, int32_t dk,
+                                           int32_t dv, int32_t window, float scale, int32_t qk_norm, int32_t sink, float eps, int32_t append,
+                                           int32_t nseq, int32_t ts, uint64_t stream) {
+    if (!proj || !off || !kv || !page_table || !pos || !y) return fail(LUMI_E_INVALID, "null pointer to lumi_k_window_attention");
+    if (heads <= 0 || kv_heads <= 0 || heads % kv_heads || dk <= 0 || dv <= 0 || window < 0 || nseq <= 0 || ts <= 0 || ldp <= 0 || pages_per_seq <= 0 ||
+        std::max(window, 1) + ts - 1 > pages_per_seq * kPageTokens)
+        return fail(LUMI_E_UNSUPPORTED, "unsupported shape for lumi_k_window_attention");
+    WinAttnArgs a{};
+    a.proj = (const float*)proj; a.ldp = ldp; a.off_q = off[0]; a.off_k = off[1]; a.off_v = off[2];
+    a.kv = (void*)kv; a.kv_is_f32 = kv_dtype == LUMI_DTYPE_F32; a.dk_pad = (dk + 15) / 16 * 16; a.dv_pad = (dv + 15) / 16 * 16;
+    a.page_table = (const int32_t*)page_table; a.pages_per_seq = pages_per_seq; a.pos = (const int32_t*)pos;
+    a.H = heads; a.G = kv_heads; a.dk = dk; a.dv = dv;
+    a.m.kind = MIXER_ATTENTION; a.m.heads = heads; a.m.kv_heads = kv_heads; a.m.dim = dk; a.m.vdim = dv;
+    a.m.scale = scale; a.m.window = window; a.m.qk_norm = qk_norm != 0; a.m.sink = sink != 0;
+    a.append = append; a.eps = eps; a.nseq = nseq; a.ts = ts;
+    a.y32 = (float*)y; a.ldy = heads * dv;
+    int n = 0;
+    LUMI_CUDA(launch_window_attention(a, (cudaStream_t)stream, &n));
+    return LUMI_OK;
+}
+
+extern "C" int32_t lumi_k_norm_add(uint64_t x, uint64_t o, uint64_t w, uint64_t y, uint64_t hi, uint64_t lo, int32_t rows, int32_t width, int32_t ld,
+                                   float eps, uint64_t stream) {
+    if (!x || !w || rows <= 0 || width <= 0 || ld < width || (ld % 4)) return fail(LUMI_E_INVALID, "bad argument to lumi_k_norm_add");
+    RowNormArgs a{(float*)x, (const float*)o, (const float*)w, (float*)y, (__nv_bfloat16*)hi, (__nv_bfloat16*)lo, nullptr, rows, width, ld, eps, nullptr};
+    LUMI_CUDA(launch_row_norm(a, (cudaStream_t)stream));
     return LUMI_OK;
 }

@@ -5,7 +5,7 @@
 // with q, k, v from short causal convolutions + silu, q and k unit vectors, one decay g and one step size b per head, and a
 // gated RMS norm per head behind the read-out.  Two forms of the same recurrence:
 //
-//   delta_step_kernel    token after token, the head's state in registers: decode steps (one token, everything from the
+//   delta_step_kernel    token after token, the head's state in shared memory: decode steps (one token, everything from the
 //                        convolution to the gated norm in one launch), and prompts of fp32 models or unusual sizes.
 //   delta_chunk_kernel   prompt slices in chunks of 64 tokens on the tensor cores.  With G_t the running sum of log g inside a
 //                        chunk and S_0 the state ahead of it, the rows U of the chunk solve the unit lower triangular system
@@ -42,12 +42,32 @@ __device__ __forceinline__ float conv_at(const DeltaArgs& a, int row, int t, int
 }
 
 // ---- token after token ----------------------------------------------------------------------------------
-// CTA = (head, sequence).  Thread (rg, cg) keeps rows rg, rg + RG, ... of four neighbouring columns of the state; S^T k and
-// S^T q are taken in one walk over the old state (S_t^T q = g S_{t-1}^T q + (k.q) u), so a token needs one reduction.
-// RPT: rows per thread held in registers; 0 = the state stays in global memory (sizes beyond the register file).
-template <int RPT, int NT>
+__device__ __forceinline__ uint32_t smem_of(const void* p) { return (uint32_t)__cvta_generic_to_shared(p); }
+constexpr uint64_t kStateWaitNs = 500000000ull;           // limit of the wait for a head's state
+// false if the phase did not complete within the limit
+__device__ __forceinline__ bool state_wait(uint64_t* bar) {
+    uint32_t done = 0, polls = 0;
+    uint64_t t0 = 0;
+    while (true) {
+        asm volatile("{\n.reg .pred p;\nmbarrier.try_wait.parity.shared::cta.b64 p, [%1], 0;\nselp.u32 %0, 1, 0, p;\n}" : "=r"(done) : "r"(smem_of(bar)) : "memory");
+        if (done) return true;
+        if ((++polls & 255u) == 0u) {
+            uint64_t now;
+            asm volatile("mov.u64 %0, %%globaltimer;" : "=l"(now));
+            if (t0 == 0) t0 = now;
+            else if (now - t0 > kStateWaitNs) return false;
+        }
+    }
+}
+
+// CTA = (head, sequence).  The head's state is one contiguous block: a bulk copy brings it into shared memory (requested ahead
+// of the predecessor's results), a bulk copy takes it back.  Thread (rg, cg) works on rows rg, rg + RG, ... of four neighbouring
+// columns; S^T k and S^T q are taken in one walk over the old state (S_t^T q = g S_{t-1}^T q + (k.q) u), so a token needs one
+// reduction.  STAGED = false: the state stays in global memory (heads beyond shared memory).
+template <int NT, bool STAGED>
 __global__ void __launch_bounds__(NT) delta_step_kernel(DeltaArgs a, int cwl) {
-    extern __shared__ float sm[];
+    extern __shared__ __align__(128) float dyn[];
+    __shared__ __align__(8) uint64_t bar;
     const int h = blockIdx.x, sl = blockIdx.y, slot = a.b0 + sl;
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
     const int dk = a.dk, dv = a.dv, dvp = a.dvp, kvh = h / (a.H / a.G);
@@ -56,6 +76,7 @@ __global__ void __launch_bounds__(NT) delta_step_kernel(DeltaArgs a, int cwl) {
     const bool act = cg < c4n;
     const int share = CW < 32 ? 32 : CW;                  // threads that leave one partial row behind
     const int slots = NT / share;
+    float* sm = dyn + (STAGED ? (size_t)dk * dvp : 0);
     float* qs = sm;
     float* ks = qs + dk;
     float* vs = ks + dk;
@@ -65,22 +86,25 @@ __global__ void __launch_bounds__(NT) delta_step_kernel(DeltaArgs a, int cwl) {
     float* rq_s = rk_s + slots * dvp;                     // [slots][dvp] partial S^T q
     float* sc = rq_s + slots * dvp;                       // sums: q.q, k.k, q.k, beta, decay
 
-    float4* Sg = reinterpret_cast<float4*>(a.S + ((size_t)slot * a.H + h) * dk * dvp);
-    float4 S[RPT > 0 ? RPT : 1];
+    float* Sg = a.S + ((size_t)slot * a.H + h) * dk * dvp;
+    const uint32_t bytes = (uint32_t)dk * dvp * 4u;
+    auto request = [&]() {                                // thread 0
+        asm volatile("mbarrier.init.shared::cta.b64 [%0], 1;" ::"r"(smem_of(&bar)));
+        asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
+        asm volatile("mbarrier.arrive.expect_tx.shared::cta.b64 _, [%0], %1;" ::"r"(smem_of(&bar)), "r"(bytes) : "memory");
+        asm volatile("cp.async.bulk.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1], %2, [%3];"
+                     ::"r"(smem_of(dyn)), "l"(Sg), "r"(bytes), "r"(smem_of(&bar)) : "memory");
+    };
     pdl_release();
-    if constexpr (RPT > 0) {
-        // the state belongs to the step before this one, which has ended: requested ahead of the predecessor's results
-#pragma unroll
-        for (int j = 0; j < RPT; ++j) {
-            const int row = rg + j * RG;
-            S[j] = act && row < dk ? Sg[(size_t)row * c4n + cg] : make_float4(0.f, 0.f, 0.f, 0.f);
-        }
-    }
+    // the state belongs to the step before this one, which has ended: requested ahead of the predecessor's results
+    if (STAGED && a.row_len == nullptr && tid == 0) request();
     pdl_sync();
     const int pos0 = a.pos[slot];
     const int n = pass_tokens(a.row_len, a.ctl, slot, a.ts, a.t_abs0);
     if (n == 0 && a.ts == 1) return;
+    if (STAGED && a.row_len != nullptr && n > 0 && tid == 0) request();
     const int Cq = a.G * dk, channels = 2 * Cq + a.H * dv;
+    float4* St = reinterpret_cast<float4*>(STAGED ? dyn : Sg);
 
     for (int t = 0; t < n; ++t) {
         const int row = sl * a.ts + t;
@@ -105,17 +129,25 @@ __global__ void __launch_bounds__(NT) delta_step_kernel(DeltaArgs a, int cwl) {
             sc[4] = expf(-expf(a.a_log[h]) * softplus_f(pr[a.off_a + h] + a.dt_bias[h]));
         }
         // partial S^T k and S^T q over this thread's rows (old state, raw k and q: the factors come afterwards)
+        if (STAGED && t == 0) {
+            if (__syncthreads_or(!state_wait(&bar))) {    // report, and let the copy land (again with a limit) before the memory goes away
+                if (tid == 0) {
+                    if (a.status != nullptr) atomicOr(a.status, STATUS_TIMEOUT);
+                    state_wait(&bar);
+                }
+                __syncthreads();
+                return;
+            }
+        }
         float4 pk = make_float4(0.f, 0.f, 0.f, 0.f), pq = pk;
-        auto walk = [&](const float4& s4, int r) {
-            const float kv = ks[r], qv = qs[r];
-            pk.x = fmaf(kv, s4.x, pk.x); pk.y = fmaf(kv, s4.y, pk.y); pk.z = fmaf(kv, s4.z, pk.z); pk.w = fmaf(kv, s4.w, pk.w);
-            pq.x = fmaf(qv, s4.x, pq.x); pq.y = fmaf(qv, s4.y, pq.y); pq.z = fmaf(qv, s4.z, pq.z); pq.w = fmaf(qv, s4.w, pq.w);
-        };
-        if constexpr (RPT > 0) {
-#pragma unroll
-            for (int j = 0; j < RPT; ++j) if (rg + j * RG < dk) walk(S[j], rg + j * RG);
-        } else {
-            if (act) for (int r = rg; r < dk; r += RG) walk(Sg[(size_t)r * c4n + cg], r);
+        if (act) {
+#pragma unroll 8
+            for (int r = rg; r < dk; r += RG) {
+                const float4 s4 = St[(size_t)r * c4n + cg];
+                const float kv = ks[r], qv = qs[r];
+                pk.x = fmaf(kv, s4.x, pk.x); pk.y = fmaf(kv, s4.y, pk.y); pk.z = fmaf(kv, s4.z, pk.z); pk.w = fmaf(kv, s4.w, pk.w);
+                pq.x = fmaf(qv, s4.x, pq.x); pq.y = fmaf(qv, s4.y, pq.y); pq.z = fmaf(qv, s4.z, pq.z); pq.w = fmaf(qv, s4.w, pq.w);
+            }
         }
         for (int o = CW; o < 32; o <<= 1) {
             pk.x += __shfl_xor_sync(0xffffffffu, pk.x, o); pk.y += __shfl_xor_sync(0xffffffffu, pk.y, o);
@@ -143,16 +175,13 @@ __global__ void __launch_bounds__(NT) delta_step_kernel(DeltaArgs a, int cwl) {
         __syncthreads();
         if (act) {
             const float4 u4 = make_float4(us[4 * cg], us[4 * cg + 1], us[4 * cg + 2], us[4 * cg + 3]);
-            auto upd = [&](float4 s4, int r) {
+#pragma unroll 8
+            for (int r = rg; r < dk; r += RG) {
+                const float4 s4 = St[(size_t)r * c4n + cg];
                 const float kv = rk * ks[r];
-                return make_float4(fmaf(kv, u4.x, g * s4.x), fmaf(kv, u4.y, g * s4.y), fmaf(kv, u4.z, g * s4.z), fmaf(kv, u4.w, g * s4.w));
-            };
-            if constexpr (RPT > 0) {
-#pragma unroll
-                for (int j = 0; j < RPT; ++j) if (rg + j * RG < dk) S[j] = upd(S[j], rg + j * RG);
-            } else {
-                for (int r = rg; r < dk; r += RG) Sg[(size_t)r * c4n + cg] = upd(Sg[(size_t)r * c4n + cg], r);
+                St[(size_t)r * c4n + cg] = make_float4(fmaf(kv, u4.x, g * s4.x), fmaf(kv, u4.y, g * s4.y), fmaf(kv, u4.z, g * s4.z), fmaf(kv, u4.w, g * s4.w));
             }
+            if (STAGED && t + 1 == n) asm volatile("fence.proxy.async.shared::cta;" ::: "memory");      // ahead of the copy back
         }
         float ss = 0.f;
         for (int c = lane; c < dv; c += 32) ss = fmaf(os[c], os[c], ss);
@@ -165,9 +194,12 @@ __global__ void __launch_bounds__(NT) delta_step_kernel(DeltaArgs a, int cwl) {
     for (int t = n; t < a.ts; ++t)                        // rows behind a shorter prompt: zero, so that what follows stays finite
         for (int c = tid; c < dv; c += NT) put_row(a.y32, a.yhi, a.ylo, (size_t)(sl * a.ts + t) * a.ldy + h * dv + c, 0.f);
     if (n == 0) return;
-    if constexpr (RPT > 0) {
-#pragma unroll
-        for (int j = 0; j < RPT; ++j) if (act && rg + j * RG < dk) Sg[(size_t)(rg + j * RG) * c4n + cg] = S[j];
+    if (STAGED) {
+        __syncthreads();
+        if (tid == 0) {
+            asm volatile("cp.async.bulk.global.shared::cta.bulk_group [%0], [%1], %2;" ::"l"(Sg), "r"(smem_of(dyn)), "r"(bytes) : "memory");
+            asm volatile("cp.async.bulk.commit_group;" ::: "memory");
+        }
     }
     if (a.ts == 1) {                                      // this token's raw convolution inputs
         const float* pr = a.proj + (size_t)sl * a.ldp;
@@ -180,6 +212,7 @@ __global__ void __launch_bounds__(NT) delta_step_kernel(DeltaArgs a, int cwl) {
         }
         for (int c = tid; c < dv; c += NT) ring[2 * Cq + h * dv + c] = pr[a.off_v + h * dv + c];
     }
+    if (STAGED && tid == 0) asm volatile("cp.async.bulk.wait_group 0;" ::: "memory");
 }
 
 // After a pass of several tokens: the last taps - 1 raw inputs of every channel go into the ring (a launch of its own, since
@@ -252,6 +285,98 @@ __global__ void __launch_bounds__(256) delta_prep_kernel(DeltaArgs a, int dk4) {
     }
 }
 
+// The same for short filters of TAPS <= 4 taps and heads of up to 32 NI channels, kPrepRows rows per warp: a row's inputs stay in
+// registers for the taps of the rows behind it, so every projection element is read once.
+constexpr int kPrepRows = 16;
+template <int TAPS, int NI>
+__global__ void __launch_bounds__(256) delta_prep_rows_kernel(DeltaArgs a, int dk4, int blocks_per_seq) {
+    const int units = 2 * a.G + a.H + 1;
+    const long w = ((long)blockIdx.x * 256 + threadIdx.x) >> 5;
+    const int lane = threadIdx.x & 31;
+    if (w >= (long)a.nseq * blocks_per_seq * units) return;
+    const int un = (int)(w % units), sl = (int)(w / units) / blocks_per_seq, tb = ((int)(w / units) % blocks_per_seq) * kPrepRows, slot = a.b0 + sl;
+    const int n = pass_tokens(a.row_len, a.ctl, slot, a.ts, a.t_abs0), te = min(a.ts, tb + kPrepRows);
+    const int pos0 = a.pos[slot], Cq = a.G * a.dk;
+    if (un == 2 * a.G + a.H) {                            // the gates
+        for (int i = lane; i < (te - tb) * a.H; i += 32) {
+            const int t = tb + i / a.H, h = i % a.H, row = sl * a.ts + t;
+            const float* pr = a.proj + (size_t)row * a.ldp;
+            float2 bg = make_float2(0.f, 0.f);
+            if (t < n) {
+                bg.x = __fdiv_rn(1.0f, 1.0f + expf(-pr[a.off_b + h]));
+                bg.y = -expf(a.a_log[h]) * softplus_f(pr[a.off_a + h] + a.dt_bias[h]);
+            }
+            reinterpret_cast<float2*>(a.gates)[(size_t)row * a.H + h] = bg;
+        }
+        return;
+    }
+    const bool is_v = un >= 2 * a.G, is_k = !is_v && un >= a.G;
+    const int head = is_v ? un - 2 * a.G : (is_k ? un - a.G : un), d = is_v ? a.dv : a.dk, dpad = is_v ? a.dvp : dk4;
+    const int ch0 = head * d;                             // first channel of the head in its projection part
+    const int off = (is_v ? a.off_v : (is_k ? a.off_k : a.off_q)) + ch0, rc = (is_v ? 2 * Cq : (is_k ? Cq : 0)) + ch0;
+    const float* cw = (is_v ? a.conv_v : (is_k ? a.conv_k : a.conv_q)) + (size_t)ch0 * TAPS;
+    const size_t oo = is_v ? (size_t)2 * a.G * dk4 + (size_t)head * a.dvp : (size_t)un * dk4;
+    const int channels = 2 * Cq + a.H * a.dv;
+    for (int c0 = 0; c0 < d; c0 += 32 * NI) {             // value heads may be wider than the key heads NI was chosen for
+        float wt[NI][TAPS], hist[NI][TAPS];               // hist[TAPS - 1] = current input
+#pragma unroll
+        for (int i = 0; i < NI; ++i) {
+            const int c = c0 + lane + 32 * i;
+#pragma unroll
+            for (int j = 0; j < TAPS; ++j) wt[i][j] = c < d ? cw[(size_t)c * TAPS + j] : 0.f;
+#pragma unroll
+            for (int j = 1; j < TAPS; ++j) {              // inputs of tokens tb - (TAPS - j), ... tb - 1
+                const int t = tb - TAPS + j;
+                float x = 0.f;
+                if (c < d) {
+                    if (t >= 0) x = a.proj[(size_t)(sl * a.ts + t) * a.ldp + off + c];
+                    else if (pos0 + t >= 0) x = a.conv[((size_t)slot * TAPS + (pos0 + t) % TAPS) * channels + rc + c];
+                }
+                hist[i][j] = x;
+            }
+        }
+        float nx[NI];
+        auto fetch = [&](int t) {
+#pragma unroll
+            for (int i = 0; i < NI; ++i) {
+                const int c = c0 + lane + 32 * i;
+                nx[i] = c < d && t < te ? a.proj[(size_t)(sl * a.ts + t) * a.ldp + off + c] : 0.f;
+            }
+        };
+        fetch(tb);
+        for (int t = tb; t < te; ++t) {
+            float v[NI];
+            float s = 0.f;
+#pragma unroll
+            for (int i = 0; i < NI; ++i) {
+#pragma unroll
+                for (int j = 0; j + 1 < TAPS; ++j) hist[i][j] = hist[i][j + 1];
+                hist[i][TAPS - 1] = nx[i];
+            }
+            fetch(t + 1);
+#pragma unroll
+            for (int i = 0; i < NI; ++i) {
+                float acc = 0.f;
+#pragma unroll
+                for (int j = 0; j < TAPS; ++j) acc = fmaf(wt[i][j], hist[i][j], acc);
+                v[i] = t < n && c0 + lane + 32 * i < d ? __fdividef(acc, 1.0f + __expf(-acc)) : 0.f;
+                s = fmaf(v[i], v[i], s);
+            }
+            float r = 1.f;
+            if (!is_v) {
+                r = __frcp_rn(__fsqrt_rn(warp_total(s) + a.unit_eps));
+                if (!is_k) r = __fdiv_rn(r, __fsqrt_rn((float)a.dk));
+            }
+            float* out = a.qkv + (size_t)(sl * a.ts + t) * a.ldqkv + oo;
+#pragma unroll
+            for (int i = 0; i < NI; ++i) {
+                const int c = c0 + lane + 32 * i;
+                if (c < dpad) out[c] = v[i] * r;
+            }
+        }
+    }
+}
+
 // One warp per (row, head): RMS norm of the read-out, weight, gate.
 __global__ void __launch_bounds__(256) delta_out_kernel(DeltaArgs a) {
     const long w = ((long)blockIdx.x * 256 + threadIdx.x) >> 5;
@@ -260,13 +385,51 @@ __global__ void __launch_bounds__(256) delta_out_kernel(DeltaArgs a) {
     const int row = (int)(w / a.H), h = (int)(w % a.H), sl = row / a.ts, t = row % a.ts;
     const bool live = t < pass_tokens(a.row_len, a.ctl, a.b0 + sl, a.ts, a.t_abs0);
     const float* o = a.o32 + ((size_t)row * a.H + h) * a.dvp;
+    const float* gate = a.proj + (size_t)row * a.ldp + a.off_g + h * a.dv;
+    const size_t oo = (size_t)row * a.ldy + h * a.dv;
+    if ((a.dv & 3) == 0 && a.dv <= 512 && ((a.ldp | a.off_g | a.ldy) & 3) == 0) {      // four neighbouring elements per lane
+        float4 v[4];
+        float s = 0.f;
+#pragma unroll
+        for (int i = 0; i < 4; ++i) {
+            const int c = 4 * (lane + 32 * i);
+            v[i] = live && c < a.dv ? *reinterpret_cast<const float4*>(o + c) : make_float4(0.f, 0.f, 0.f, 0.f);
+            s = fmaf(v[i].x, v[i].x, fmaf(v[i].y, v[i].y, fmaf(v[i].z, v[i].z, fmaf(v[i].w, v[i].w, s))));
+        }
+        const float rs = __frcp_rn(__fsqrt_rn(__fdiv_rn(warp_total(s), (float)a.dv) + a.eps));
+#pragma unroll
+        for (int i = 0; i < 4; ++i) {
+            const int c = 4 * (lane + 32 * i);
+            if (c >= a.dv) break;
+            float y[4] = {0.f, 0.f, 0.f, 0.f};
+            if (live) {
+                const float4 gt = *reinterpret_cast<const float4*>(gate + c);
+                const float ov[4] = {v[i].x, v[i].y, v[i].z, v[i].w}, gv[4] = {gt.x, gt.y, gt.z, gt.w};
+#pragma unroll
+                for (int e = 0; e < 4; ++e) y[e] = ov[e] * rs * a.o_norm[c + e] * __fdividef(gv[e], 1.0f + __expf(-gv[e]));
+            }
+            if (a.y32 != nullptr) *reinterpret_cast<float4*>(a.y32 + oo + c) = make_float4(y[0], y[1], y[2], y[3]);
+            if (a.yhi != nullptr) {
+                const __nv_bfloat162 h0 = __floats2bfloat162_rn(y[0], y[1]), h1 = __floats2bfloat162_rn(y[2], y[3]);
+                uint2 u;
+                u.x = *reinterpret_cast<const uint32_t*>(&h0); u.y = *reinterpret_cast<const uint32_t*>(&h1);
+                *reinterpret_cast<uint2*>(a.yhi + oo + c) = u;
+                if (a.ylo != nullptr) {
+                    const float2 f0 = __bfloat1622float2(h0), f1 = __bfloat1622float2(h1);
+                    const __nv_bfloat162 l0 = __floats2bfloat162_rn(y[0] - f0.x, y[1] - f0.y), l1 = __floats2bfloat162_rn(y[2] - f1.x, y[3] - f1.y);
+                    u.x = *reinterpret_cast<const uint32_t*>(&l0); u.y = *reinterpret_cast<const uint32_t*>(&l1);
+                    *reinterpret_cast<uint2*>(a.ylo + oo + c) = u;
+                }
+            }
+        }
+        return;
+    }
     float s = 0.f;
     if (live) for (int c = lane; c < a.dv; c += 32) s = fmaf(o[c], o[c], s);
     s = warp_total(s);
     const float rs = __frcp_rn(__fsqrt_rn(__fdiv_rn(s, (float)a.dv) + a.eps));
-    const float* gate = a.proj + (size_t)row * a.ldp + a.off_g + h * a.dv;
     for (int c = lane; c < a.dv; c += 32)
-        put_row(a.y32, a.yhi, a.ylo, (size_t)row * a.ldy + h * a.dv + c, live ? o[c] * rs * a.o_norm[c] * silu_f(gate[c]) : 0.f);
+        put_row(a.y32, a.yhi, a.ylo, oo + c, live ? o[c] * rs * a.o_norm[c] * silu_f(gate[c]) : 0.f);
 }
 
 struct Tf2 { uint32_t hi, lo; };
@@ -560,14 +723,18 @@ __global__ void __launch_bounds__(256) delta_chunk_kernel(DeltaArgs a, int dk4, 
     }
 }
 
-constexpr size_t kSmemMax = 227 * 1024;
+constexpr size_t kSmemMax = 227 * 1024 - 1024;
 
-template <int RPT, int NT>
-cudaError_t step_launch(const DeltaArgs& a, int cwl, cudaStream_t st) {
+size_t step_smem(const DeltaArgs& a, int cwl, int nt, bool staged) {
     const int share = (1 << cwl) < 32 ? 32 : (1 << cwl);
-    const size_t smem = sizeof(float) * (2 * (size_t)a.dk + 3 * (size_t)a.dvp + 2 * (size_t)(NT / share) * a.dvp + 8);
+    return sizeof(float) * (2 * (size_t)a.dk + 3 * (size_t)a.dvp + 2 * (size_t)(nt / share) * a.dvp + 8 + (staged ? (size_t)a.dk * a.dvp : 0));
+}
+
+template <int NT, bool STAGED>
+cudaError_t step_launch(const DeltaArgs& a, int cwl, cudaStream_t st) {
+    const size_t smem = step_smem(a, cwl, NT, STAGED);
     if (smem > kSmemMax) return cudaErrorInvalidValue;
-    auto kern = delta_step_kernel<RPT, NT>;
+    auto kern = delta_step_kernel<NT, STAGED>;
     if (smem > 48 * 1024) {
         const cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
         if (e != cudaSuccess) return e;
@@ -613,21 +780,11 @@ cudaError_t launch_delta_step(const DeltaArgs& a, cudaStream_t st, int* launches
     const int CW = 1 << cwl;
     *launches = 1;
     cudaError_t e;
-    if (CW <= 128) {
-        const int r128 = (a.dk * CW + 127) / 128, r256 = (a.dk * CW + 255) / 256, r512 = (a.dk * CW + 511) / 512;
-        if (r128 <= 1) e = step_launch<1, 128>(a, cwl, st);
-        else if (r128 <= 2) e = step_launch<2, 128>(a, cwl, st);
-        else if (r128 <= 4) e = step_launch<4, 128>(a, cwl, st);
-        else if (r128 <= 8) e = step_launch<8, 128>(a, cwl, st);
-        else if (r256 <= 8) e = step_launch<8, 256>(a, cwl, st);
-        else if (r256 <= 16) e = step_launch<16, 256>(a, cwl, st);
-        else if (r512 <= 16) e = step_launch<16, 512>(a, cwl, st);
-        else e = step_launch<0, 512>(a, cwl, st);
-    } else if (CW <= 512) {
-        e = step_launch<0, 512>(a, cwl, st);
-    } else {
-        return cudaErrorInvalidValue;
-    }
+    if (CW > 256) return cudaErrorInvalidValue;
+    const bool small = (size_t)a.dk * a.dvp <= 4096 && CW <= 128;
+    if (step_smem(a, cwl, 256, true) > kSmemMax) e = step_launch<256, false>(a, cwl, st);
+    else if (small) e = step_launch<128, true>(a, cwl, st);
+    else e = step_launch<256, true>(a, cwl, st);
     if (e != cudaSuccess) return e;
     if (a.ts > 1) { *launches = 2; e = launch_tail(a, st); }
     return e;
@@ -643,8 +800,20 @@ cudaError_t launch_delta_chunk(const DeltaArgs& a, cudaStream_t st, int* launche
     if (!chunk_shape(a.dk, a.dv, &nw, &ntw)) return cudaErrorInvalidValue;
     const int dk4 = (a.dk + 3) / 4 * 4, dk16 = (a.dk + 15) / 16 * 16, dvb = nw * ntw * 8;
     const size_t smem = chunk_smem(dk16, dvb);
-    const long pw = (long)a.nseq * a.ts * (2 * a.G + a.H + 1), ow = (long)a.nseq * a.ts * a.H;
-    delta_prep_kernel<<<(unsigned)((pw + 7) / 8), 256, 0, st>>>(a, dk4);
+    const long ow = (long)a.nseq * a.ts * a.H;
+    const int bps = (a.ts + kPrepRows - 1) / kPrepRows;
+    const unsigned pg = (unsigned)(((long)a.nseq * bps * (2 * a.G + a.H + 1) + 7) / 8);
+    bool prepared = false;
+#define LUMI_PREP(T_, NI_) \
+    if (!prepared && a.taps == T_ && a.dk <= 32 * NI_) { delta_prep_rows_kernel<T_, NI_><<<pg, 256, 0, st>>>(a, dk4, bps); prepared = true; }
+    LUMI_PREP(2, 1) LUMI_PREP(2, 2) LUMI_PREP(2, 4) LUMI_PREP(2, 8)
+    LUMI_PREP(3, 1) LUMI_PREP(3, 2) LUMI_PREP(3, 4) LUMI_PREP(3, 8)
+    LUMI_PREP(4, 1) LUMI_PREP(4, 2) LUMI_PREP(4, 4) LUMI_PREP(4, 8)
+#undef LUMI_PREP
+    if (!prepared) {                                      // other filter lengths
+        const long pw = (long)a.nseq * a.ts * (2 * a.G + a.H + 1);
+        delta_prep_kernel<<<(unsigned)((pw + 7) / 8), 256, 0, st>>>(a, dk4);
+    }
     cudaError_t e = cudaGetLastError();
     if (e != cudaSuccess) return e;
     const dim3 grid(a.H, (a.dv + dvb - 1) / dvb, a.nseq);

@@ -206,6 +206,7 @@ struct LayerState {
 struct RowBufs {
     size_t rows = 0;
     float *x = nullptr;                              // residual stream [rows][x_ld] (the decode set uses the session's x)
+    float *x2 = nullptr;                             // where x goes when a product's prologue adds to it (few rows)
     float *proj = nullptr, *mix = nullptr, *qkv = nullptr, *gates = nullptr, *y32 = nullptr;
     __nv_bfloat16 *xh = nullptr, *xl = nullptr, *ah = nullptr, *al = nullptr;
 };
@@ -296,6 +297,14 @@ constexpr size_t kGemmScratchFloats = (size_t)4 << 20;      // 16 MiB per lane
 
 // ---- kernel launchers (kernels.cu) --------------------------------------------------------------
 // All take the stream to enqueue on and return a cudaError_t from the launch.
+// A row operand that is still to take the norm of a sublayer's output: A + o / rms(o) * w over `width` elements (rows of K
+// elements); the product is taken of the sum, which also goes to x_out (not the memory of A or o).  o null: nothing.
+struct PostAdd {
+    const float* o = nullptr;
+    const float* w = nullptr;
+    float* x_out = nullptr;
+    int width = 0;
+};
 struct GemvArgs {
     const float* A; int lda;         // [M][K] fp32
     const void* W; int w_dtype;      // [N][K]
@@ -313,6 +322,7 @@ struct GemvArgs {
     int* amax_idx = nullptr;
     int amax_stride = 0;
     int* amax_parts = nullptr;
+    PostAdd post;                    // applied before gamma
 };
 cudaError_t launch_gemv(const GemvArgs& a, cudaStream_t st);
 cudaError_t launch_logprob(const float* logits, int B, int V, const uint32_t* targets, float* out, int out_stride, int out_col,
@@ -505,6 +515,7 @@ struct RowNormArgs {
     const int32_t* row_idx;
     int rows, width, ld;
     float eps;
+    float* x_out;                        // where the new residual rows go (null = back into x)
 };
 cudaError_t launch_row_norm(const RowNormArgs& a, cudaStream_t st);
 
@@ -526,6 +537,7 @@ struct DeltaArgs {
     // chunked form: prepared q | k | v rows (unit vectors, activations applied), [rows][2 G dk + H dv] padded, and per (row, head)
     // beta and the logarithm of the decay; the read-out before its norm
     float* qkv; int ldqkv; float* gates; float* o32;
+    int32_t* status;                                 // receives STATUS_TIMEOUT if a bounded wait gives up; may be null
 };
 cudaError_t launch_delta_step(const DeltaArgs& a, cudaStream_t st, int* launches);
 bool delta_chunk_supported(int dk, int dv);

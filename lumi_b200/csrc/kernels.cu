@@ -195,7 +195,7 @@ template <typename WT, int NB, int RPW, int ACT>
 __global__ void __launch_bounds__(256) gemv_kernel(const float* A, int lda, const WT* __restrict__ W,
                                                    float* D, int ldd, const float* R,
                                                    const float* __restrict__ gamma, int M, int N, int K, float eps, int KS,
-                                                   float* amax_val, int* amax_idx, int amax_stride) {
+                                                   float* amax_val, int* amax_idx, int amax_stride, PostAdd post) {
     extern __shared__ float4 gemv_smem4[];
     float* xs = reinterpret_cast<float*>(gemv_smem4);
     constexpr int E = WLoad<WT>::E;
@@ -233,6 +233,34 @@ __global__ void __launch_bounds__(256) gemv_kernel(const float* A, int lda, cons
         reinterpret_cast<float4*>(xs)[i] = v;
     }
     __syncthreads();
+    if (post.o != nullptr) {
+        // the residual stream takes the norm of the sublayer that came before: x + o / rms(o) * w, by every CTA for itself;
+        // the first one also writes the new rows
+        __shared__ float pred[NB][8];
+#pragma unroll
+        for (int b = 0; b < NB; ++b) {
+            float s = 0.f;
+            if (b < nb) for (int k = threadIdx.x; k < K; k += 256) { const float v = post.o[(size_t)(m0 + b) * K + k]; s = fmaf(v, v, s); }
+            s = warp_sum(s);
+            if (lane == 0) pred[b][warp] = s;
+        }
+        __syncthreads();
+#pragma unroll
+        for (int b = 0; b < NB; ++b) {
+            if (b < nb) {
+                float t = 0.f;
+#pragma unroll
+                for (int w = 0; w < 8; ++w) t += pred[b][w];
+                const float r = rms_scale(t, post.width, eps);
+                for (int k = threadIdx.x; k < K; k += 256) {
+                    const float v = fmaf(post.o[(size_t)(m0 + b) * K + k] * r, post.w[k], xs[b * K + k]);
+                    xs[b * K + k] = v;
+                    if (blockIdx.x == 0) post.x_out[(size_t)(m0 + b) * K + k] = v;
+                }
+            }
+        }
+        __syncthreads();
+    }
     if (gamma != nullptr) {
         // RMSNorm of the NB staged rows by the whole CTA: per-thread partials in ascending k, xor tree,
         // then the 8 warp sums in warp order
@@ -376,7 +404,7 @@ template <typename WT, int NB, int U, int RPW>
 __global__ void __launch_bounds__(256, 2) gemv_pre_kernel(const float* A, int lda, const WT* __restrict__ W,
                                                           float* D, int ldd, const float* R,
                                                           const float* __restrict__ gamma, int M, int N, int K, float eps,
-                                                          int rows_per_cta, int pace_ns, int pre_delay_ns, int32_t* status) {
+                                                          int rows_per_cta, int pace_ns, int pre_delay_ns, int32_t* status, PostAdd post) {
     extern __shared__ float4 gemv_smem4[];
     constexpr int E = WLoad<WT>::E;
     constexpr int GN = (U * E + 7) / 8;                 // gamma values per thread: K / 256 rounded up
@@ -439,10 +467,11 @@ __global__ void __launch_bounds__(256, 2) gemv_pre_kernel(const float* A, int ld
         }
     }
     float gam[XREG ? 1 : GN];
+    const float* __restrict__ nw = post.o != nullptr ? post.w : gamma;      // this kernel takes one norm: of the input, or of what joins it
     if constexpr (XREG) {
         // the norm weights wait in the staging area (the activations themselves never go there)
-        if (gamma != nullptr) {
-            for (int i = threadIdx.x; i < K4; i += 256) reinterpret_cast<float4*>(xs)[i] = reinterpret_cast<const float4*>(gamma)[i];
+        if (nw != nullptr) {
+            for (int i = threadIdx.x; i < K4; i += 256) reinterpret_cast<float4*>(xs)[i] = reinterpret_cast<const float4*>(nw)[i];
         }
         gam[0] = 0.f;
         __syncthreads();
@@ -450,7 +479,7 @@ __global__ void __launch_bounds__(256, 2) gemv_pre_kernel(const float* A, int ld
 #pragma unroll
         for (int i = 0; i < GN; ++i) {
             const int k = threadIdx.x + 256 * i;
-            gam[i] = (gamma != nullptr && k < K) ? gamma[k] : 0.f;
+            gam[i] = (nw != nullptr && k < K) ? nw[k] : 0.f;
         }
     }
     pdl_wait();
@@ -484,7 +513,34 @@ __global__ void __launch_bounds__(256, 2) gemv_pre_kernel(const float* A, int ld
                 xr[u * E + 4 * q] = v.x; xr[u * E + 4 * q + 1] = v.y; xr[u * E + 4 * q + 2] = v.z; xr[u * E + 4 * q + 3] = v.w;
             }
         }
-        if (gamma != nullptr) {
+        if (post.o != nullptr) {
+            float ov[U * E];
+            float s0 = 0.f;
+#pragma unroll
+            for (int u = 0; u < U; ++u) {
+                const int c = lane + 32 * u;
+#pragma unroll
+                for (int q = 0; q < E / 4; ++q) {
+                    const float4 v = *reinterpret_cast<const float4*>(post.o + c * E + 4 * q);
+                    const int i = u * E + 4 * q;
+                    ov[i] = v.x; ov[i + 1] = v.y; ov[i + 2] = v.z; ov[i + 3] = v.w;
+                    s0 = fmaf(v.x, v.x, fmaf(v.y, v.y, fmaf(v.z, v.z, fmaf(v.w, v.w, s0))));
+                }
+            }
+            const float rs = rms_scale(warp_sum(s0), post.width, eps);
+#pragma unroll
+            for (int u = 0; u < U; ++u) {
+                const int c = lane + 32 * u;
+#pragma unroll
+                for (int q = 0; q < E / 4; ++q) {
+                    const float4 gq = *reinterpret_cast<const float4*>(xs + c * E + 4 * q);
+                    const int i = u * E + 4 * q;
+                    xr[i] = fmaf(ov[i] * rs, gq.x, xr[i]); xr[i + 1] = fmaf(ov[i + 1] * rs, gq.y, xr[i + 1]);
+                    xr[i + 2] = fmaf(ov[i + 2] * rs, gq.z, xr[i + 2]); xr[i + 3] = fmaf(ov[i + 3] * rs, gq.w, xr[i + 3]);
+                    if (blockIdx.x == 0 && warp == 0) *reinterpret_cast<float4*>(post.x_out + c * E + 4 * q) = make_float4(xr[i], xr[i + 1], xr[i + 2], xr[i + 3]);
+                }
+            }
+        } else if (gamma != nullptr) {
             // sum of squares: four running sums per lane (elements 0, 1, 2, 3 of its quads in ascending k),
             // (s0 + s1) + (s2 + s3), then the xor tree
             float s0 = 0.f, s1 = 0.f, s2 = 0.f, s3 = 0.f;
@@ -517,7 +573,35 @@ __global__ void __launch_bounds__(256, 2) gemv_pre_kernel(const float* A, int ld
         }
         __syncthreads();
         TL_MARK(2)
-        if (gamma != nullptr) {
+        if (post.o != nullptr) {
+#pragma unroll
+            for (int b = 0; b < NB; ++b) {
+                float s = 0.f;
+                if (b < nb) for (int k = threadIdx.x; k < K; k += 256) { const float v = post.o[(size_t)b * K + k]; s = fmaf(v, v, s); }
+                s = warp_sum(s);
+                if (lane == 0) nred[b][warp] = s;
+            }
+            __syncthreads();
+#pragma unroll
+            for (int b = 0; b < NB; ++b) {
+                if (b < nb) {
+                    float t = 0.f;
+#pragma unroll
+                    for (int w = 0; w < 8; ++w) t += nred[b][w];
+                    const float r = rms_scale(t, post.width, eps);
+#pragma unroll
+                    for (int i = 0; i < GN; ++i) {
+                        const int k = threadIdx.x + 256 * i;
+                        if (k < K) {
+                            const float v = fmaf(post.o[(size_t)b * K + k] * r, gam[i], xs[b * K + k]);
+                            xs[b * K + k] = v;
+                            if (blockIdx.x == 0) post.x_out[(size_t)b * K + k] = v;
+                        }
+                    }
+                }
+            }
+            __syncthreads();
+        } else if (gamma != nullptr) {
 #pragma unroll
             for (int b = 0; b < NB; ++b) {
                 float s = 0.f;
@@ -1330,7 +1414,7 @@ static cudaError_t gemv_launch(const GemvArgs& a, int KS, cudaStream_t st) {
         if (a.amax_parts != nullptr) *a.amax_parts = (int)grid.x;
     }
     return launch_k(kern, grid, dim3(256), smem, st, a.A, a.lda, (const WT*)a.W, a.D, a.ldd, a.R, a.gamma, a.M, a.N, a.K, a.eps, KS,
-                    a.amax_val, a.amax_idx, a.amax_stride);
+                    a.amax_val, a.amax_idx, a.amax_stride, a.post);
 }
 
 template <typename WT, int NB, int ACT>
@@ -1419,13 +1503,14 @@ static cudaError_t gemv_pre_launch(const GemvArgs& a, int rows_per_cta, size_t s
     }
     dim3 grid((a.N + rows_per_cta - 1) / rows_per_cta);
     return launch_k(kern, grid, dim3(256), smem, st, a.A, a.lda, (const WT*)a.W, a.D, a.ldd, a.R, a.gamma, a.M, a.N, a.K, a.eps,
-                    rows_per_cta, gemv_pre_pace_ns(), smem > 64 * 1024 ? gemv_pre_delay_ns() : 0, a.status);
+                    rows_per_cta, gemv_pre_pace_ns(), smem > 64 * 1024 ? gemv_pre_delay_ns() : 0, a.status, a.post);
 }
 
 // Returns true (and the launch result in *err) when the product was given to the preloading kernel.
 template <typename WT>
 static bool gemv_pre_try(const GemvArgs& a, cudaStream_t st, cudaError_t* err) {
     constexpr int E = WLoad<WT>::E;
+    if (a.post.o != nullptr && (a.gamma != nullptr || a.lda != a.K)) return false;
     if (!gemv_pre_enabled() || !a.allow_preload || a.amax_val != nullptr || a.act != 0 || a.M > 4 || a.M < 1 || (a.K % E) != 0 || a.K < E) return false;
     const int KC = a.K / E;
     const int U = (KC + 31) / 32;

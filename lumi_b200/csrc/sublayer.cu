@@ -40,10 +40,9 @@ __global__ void __launch_bounds__(NT) row_norm_kernel(RowNormArgs a) {
         float4 y = make_float4(t.x * rs * w.x, t.y * rs * w.y, t.z * rs * w.z, t.w * rs * w.w);
         const size_t oo = (size_t)r * a.ld + 4 * (size_t)c;
         if (a.o != nullptr) {
-            float4* xp = reinterpret_cast<float4*>(a.x + oo);
-            const float4 x = *xp;
+            const float4 x = *reinterpret_cast<const float4*>(a.x + oo);
             y = make_float4(x.x + y.x, x.y + y.y, x.z + y.z, x.w + y.w);
-            *xp = y;
+            *reinterpret_cast<float4*>((a.x_out != nullptr ? a.x_out : a.x) + oo) = y;
         } else if (a.y32 != nullptr) {
             *reinterpret_cast<float4*>(a.y32 + oo) = y;
         }

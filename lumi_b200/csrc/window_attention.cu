@@ -165,12 +165,14 @@ __device__ __forceinline__ void halves2(float v0, float v1, uint32_t& hi, uint32
     hi = *reinterpret_cast<const uint32_t*>(&h);
     lo = *reinterpret_cast<const uint32_t*>(&l);
 }
+__device__ __forceinline__ float ex2(float x) { float y; asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x)); return y; }
 __device__ __forceinline__ void cp16b(__nv_bfloat16* dst, const __nv_bfloat16* src, bool ok) {
     const int bytes = ok ? 16 : 0;                        // 0: filled with zeros
     asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"((uint32_t)__cvta_generic_to_shared(dst)), "l"(src), "r"(bytes) : "memory");
 }
 
 constexpr int kWinStages = 2;
+constexpr int kMmaDim = 256;                              // widest key head of the tensor-core form
 constexpr int kWinSlices = 16;
 constexpr int kWinSliceMin = 256;                         // tokens from which a slice of the context is worth a CTA
 
@@ -221,36 +223,54 @@ __global__ void __launch_bounds__(128) win_mma_kernel(WinAttnArgs a, int hb, int
     const int per = (pages + nsplit - 1) / nsplit, pb = pg0 + split * per, pe = min(pg0 + pages, pb + per);
     const int local = DECODE && a.append ? pos0 : -1;     // the row that this launch itself appends
     const int kc = a.dk_pad / 8, vc = a.dv_pad / 8;       // 16-byte chunks per row
+    // this thread's first chunk of a page and the step to its next one (a division per chunk would cost more than the copy)
+    const int kr0 = tid / kc, kc0 = tid % kc, kdr = 128 / kc, kdc = 128 % kc;
+    const int vr0 = tid / vc, vc0 = tid % vc, vdr = 128 / vc, vdc = 128 % vc;
     auto issue = [&](int pg) {
         __nv_bfloat16* ks = stage + ((pg - pb) % kWinStages) * stage_elems;
         __nv_bfloat16* vs = ks + kPageTokens * KS;
         const int pidx = pt[pg % a.pages_per_seq];
         const __nv_bfloat16* kp = pool + (size_t)pidx * s.page_elems + (size_t)kvh * kPageTokens * (a.dk_pad + a.dv_pad);
         const __nv_bfloat16* vp = kp + s.v_off;
-        for (int i = tid; i < kPageTokens * kc; i += 128) {
-            const int r = i / kc, c = i % kc, p = pg * kPageTokens + r;
-            cp16b(ks + r * KS + c * 8, kp + (size_t)r * a.dk_pad + c * 8, p >= lo && p <= hi && p != local);
+        for (int r = kr0, c = kc0; r < kPageTokens;) {
+            const int p = pg * kPageTokens + r;
+            cp16b(ks + r * KS + c * 8, kp + r * a.dk_pad + c * 8, p >= lo && p <= hi && p != local);
+            r += kdr; c += kdc;
+            if (c >= kc) { c -= kc; ++r; }
         }
-        for (int i = tid; i < kPageTokens * vc; i += 128) {
-            const int r = i / vc, c = i % vc, p = pg * kPageTokens + r;
-            cp16b(vs + r * VS + c * 8, vp + (size_t)r * a.dv_pad + c * 8, p >= lo && p <= hi && p != local);
+        for (int r = vr0, c = vc0; r < kPageTokens;) {
+            const int p = pg * kPageTokens + r;
+            cp16b(vs + r * VS + c * 8, vp + r * a.dv_pad + c * 8, p >= lo && p <= hi && p != local);
+            r += vdr; c += vdc;
+            if (c >= vc) { c -= vc; ++r; }
         }
     };
-#pragma unroll
-    for (int i = 0; i < kWinStages - 1; ++i) {
-        if (pb + i < pe) issue(pb + i);
-        asm volatile("cp.async.commit_group;" ::: "memory");
-    }
+    if (pb < pe) issue(pb);
+    asm volatile("cp.async.commit_group;" ::: "memory");
     // query columns: normalised, as bf16 halves; unused columns are zero
-    for (int m = warp; m < QW * 16; m += 4) {
-        const int set = m / 16, mm = m % 16, rr = set * q_rows + mm / hb, hh = mm % hb;
-        const bool ok = mm < q_rows * hb && rr < nvalid && hh < nh;
-        const float* q = a.proj + (size_t)(sl * a.ts + i0 + (ok ? rr : 0)) * a.ldp + a.off_q + (size_t)(kvh * s.hpk + h0 + (ok ? hh : 0)) * a.dk;
-        const float r = a.m.qk_norm ? rms_factor(q, a.dk, a.eps, lane) : 1.f;
-        for (int c = lane; c < a.dk_pad; c += 32) {
-            __nv_bfloat16 vh, vl;
-            bf16_halves(ok && c < a.dk ? q[c] * r : 0.f, vh, vl);
-            qh[m * KS + c] = vh; ql[m * KS + c] = vl;
+    // (four columns at a time, so that their loads overlap)
+    for (int m0 = warp * QW * 4; m0 < (warp + 1) * QW * 4; m0 += 4) {
+        float v[4][kMmaDim / 32];
+#pragma unroll
+        for (int j = 0; j < 4; ++j) {
+            const int mm = (m0 + j) % 16, rr = (m0 + j) / 16 * q_rows + mm / hb, hh = mm % hb;
+            const bool ok = mm < q_rows * hb && rr < nvalid && hh < nh;
+            const float* q = a.proj + (size_t)(sl * a.ts + i0 + (ok ? rr : 0)) * a.ldp + a.off_q + (size_t)(kvh * s.hpk + h0 + (ok ? hh : 0)) * a.dk;
+#pragma unroll
+            for (int i = 0; i < kMmaDim / 32; ++i) v[j][i] = ok && lane + 32 * i < a.dk ? q[lane + 32 * i] : 0.f;
+        }
+#pragma unroll
+        for (int j = 0; j < 4; ++j) {
+            float r = 1.f;
+            if (a.m.qk_norm) {
+                float sq = 0.f;
+#pragma unroll
+                for (int i = 0; i < kMmaDim / 32; ++i) sq = fmaf(v[j][i], v[j][i], sq);
+                r = __frcp_rn(__fsqrt_rn(__fdiv_rn(warp_total(sq), (float)a.dk) + a.eps));
+            }
+#pragma unroll
+            for (int i = 0; i < kMmaDim / 32; ++i)
+                if (lane + 32 * i < a.dk_pad) bf16_halves(v[j][i] * r, qh[(m0 + j) * KS + lane + 32 * i], ql[(m0 + j) * KS + lane + 32 * i]);
         }
     }
     if (DECODE && a.append) {
@@ -293,10 +313,10 @@ __global__ void __launch_bounds__(128) win_mma_kernel(WinAttnArgs a, int hb, int
     const int whi = DECODE ? hi : min(hi, pos0 + (set + 1) * q_rows - 1);
     const int wlo = DECODE ? lo : (a.m.window > 0 ? pos0 + set * q_rows - a.m.window + 1 : 0);
     for (int pg = pb; pg < pe; ++pg) {
-        if (pg + kWinStages - 1 < pe) issue(pg + kWinStages - 1);
+        asm volatile("cp.async.wait_group 0;" ::: "memory");
+        __syncthreads();                                  // this page is here, and every warp has finished with the other stage
+        if (pg + 1 < pe) issue(pg + 1);
         asm volatile("cp.async.commit_group;" ::: "memory");
-        asm volatile("cp.async.wait_group %0;" ::"n"(kWinStages - 1) : "memory");
-        __syncthreads();
         __nv_bfloat16* ks = stage + ((pg - pb) % kWinStages) * stage_elems;
         __nv_bfloat16* vs = ks + kPageTokens * KS;
         if (DECODE && local >= pg * kPageTokens && local < (pg + 1) * kPageTokens) {
@@ -330,6 +350,8 @@ __global__ void __launch_bounds__(128) win_mma_kernel(WinAttnArgs a, int hb, int
                     mma_bf16(sc[st][1], fl, kb[2], kb[3]);
                 }
             }
+            // a page that every used column of the warp sees whole needs no mask (unused columns may then hold anything finite)
+            const bool whole = p0 + kPageTokens - 1 <= (DECODE ? hi : pos0 + set * q_rows) && (a.m.window <= 0 || p0 > whi - a.m.window);
             float tm[2] = {kNoScore, kNoScore};
 #pragma unroll
             for (int st = 0; st < STRIPS; ++st)
@@ -338,17 +360,18 @@ __global__ void __launch_bounds__(128) win_mma_kernel(WinAttnArgs a, int hb, int
 #pragma unroll
                     for (int i = 0; i < 4; ++i) {
                         const int p = p0 + (strip0 + st) * 16 + e * 8 + 2 * tq + (i & 1), c = i >> 1;
-                        sc[st][e][i] = p <= last[c] && p > first[c] ? sc[st][e][i] * sc2 : kNoScore;
+                        sc[st][e][i] = whole || (p <= last[c] && p > first[c]) ? sc[st][e][i] * sc2 : kNoScore;
                         tm[c] = fmaxf(tm[c], sc[st][e][i]);
                     }
-            float f[2];
+            float f[2], mu[2];
 #pragma unroll
             for (int c = 0; c < 2; ++c) {
                 tm[c] = fmaxf(tm[c], __shfl_xor_sync(0xffffffffu, tm[c], 1));
                 tm[c] = fmaxf(tm[c], __shfl_xor_sync(0xffffffffu, tm[c], 2));
                 const float mn = fmaxf(mx[c], tm[c]);
-                f[c] = exp2f(mx[c] - mn);
+                f[c] = ex2(mx[c] - mn);
                 mx[c] = mn;
+                mu[c] = mn > 0.5f * kNoScore ? mn : 0.f;  // nothing seen yet: masked scores still weigh nothing
                 ls[c] *= f[c];
             }
 #pragma unroll
@@ -360,7 +383,7 @@ __global__ void __launch_bounds__(128) win_mma_kernel(WinAttnArgs a, int hb, int
                 for (int e = 0; e < 2; ++e)
 #pragma unroll
                     for (int i = 0; i < 4; ++i) {
-                        pr[e][i] = sc[st][e][i] > 0.5f * kNoScore ? exp2f(sc[st][e][i] - mx[i >> 1]) : 0.f;
+                        pr[e][i] = ex2(sc[st][e][i] - mu[i >> 1]);
                         ls[i >> 1] += pr[e][i];
                     }
                 uint32_t ph[4], pl[4];                    // the weights as the A operand of P V
@@ -382,7 +405,6 @@ __global__ void __launch_bounds__(128) win_mma_kernel(WinAttnArgs a, int hb, int
                 }
             }
         }
-        __syncthreads();                                  // this stage is free again
     }
     asm volatile("cp.async.wait_group 0;" ::: "memory");
 #pragma unroll
@@ -399,11 +421,25 @@ __global__ void __launch_bounds__(128) win_mma_kernel(WinAttnArgs a, int hb, int
             if (last[c] < 0) continue;
             const int m = g + 8 * c, rr = set * q_rows + m / hb, hh = m % hb;
             const float inv = __frcp_rn(ls[c] + (a.m.sink ? exp2f(a.m.sink_score * kLog2e - mx[c]) : 0.f));
+            const size_t oo = (size_t)(sl * a.ts + i0 + rr) * a.ldy + (size_t)(kvh * s.hpk + h0 + hh) * a.dv;
+            const bool pairs = ((a.dv | a.ldy) & 1) == 0;
 #pragma unroll
-            for (int i = 0; i < NT; ++i)
-#pragma unroll
-                for (int e = 0; e < 2; ++e)
-                    if (i * 8 + 2 * tq + e < a.dv) emit(rr, hh, i * 8 + 2 * tq + e, o[i][2 * c + e] * inv);
+            for (int i = 0; i < NT; ++i) {
+                const int d = i * 8 + 2 * tq;
+                const float v0 = o[i][2 * c] * inv, v1 = o[i][2 * c + 1] * inv;
+                if (pairs && d < a.dv) {
+                    if (a.y32 != nullptr) *reinterpret_cast<float2*>(a.y32 + oo + d) = make_float2(v0, v1);
+                    if (a.yhi != nullptr) {
+                        uint32_t h2, l2;
+                        halves2(v0, v1, h2, l2);
+                        *reinterpret_cast<uint32_t*>(a.yhi + oo + d) = h2;
+                        if (a.ylo != nullptr) *reinterpret_cast<uint32_t*>(a.ylo + oo + d) = l2;
+                    }
+                } else if (!pairs) {
+                    if (d < a.dv) emit(rr, hh, d, v0);
+                    if (d + 1 < a.dv) emit(rr, hh, d + 1, v1);
+                }
+            }
         }
         return;
     }
@@ -423,7 +459,7 @@ __global__ void __launch_bounds__(128) win_mma_kernel(WinAttnArgs a, int hb, int
         }
     }
     __syncthreads();
-    const int PW = nh * (a.dv + 2);                       // per slice: [nh] maxima, [nh] sums, [nh][dv] context
+    // per slice: [nh] maxima, [nh] sums, [nh][dv] context
     const size_t unit = (size_t)grp * gridDim.y + blockIdx.y;
     float* part = nsplit > 1 ? a.part + (unit * kWinSlices + split) * (size_t)(hb * (a.dv + 2)) : nullptr;
     for (int i = tid; i < nh * a.dv; i += 128) {
@@ -447,7 +483,6 @@ __global__ void __launch_bounds__(128) win_mma_kernel(WinAttnArgs a, int hb, int
         }
     }
     if (nsplit == 1) return;
-    (void)PW;
     __threadfence();
     __syncthreads();
     if (tid == 0) {
@@ -549,7 +584,7 @@ size_t window_attention_part_floats(const MixerSpec& m) { return (size_t)kWinSli
 
 cudaError_t launch_window_attention(const WinAttnArgs& a, cudaStream_t st, int* launches) {
     *launches = 0;
-    const bool mma = !a.kv_is_f32 && a.dv_pad <= 256 && mma_smem(a, a.ts == 1) <= kSmemMax;
+    const bool mma = !a.kv_is_f32 && a.dk_pad <= kMmaDim && a.dv_pad <= 256 && mma_smem(a, a.ts == 1) <= kSmemMax;
     cudaError_t e;
     if (a.append && !(mma && a.ts == 1)) {
         e = a.kv_is_f32 ? append<float>(a, st) : append<__nv_bfloat16>(a, st);

@@ -103,3 +103,15 @@ def iter_tensors(cfg: ZozonexConfig, seed: int = 0, weights_dtype: str = "bf16")
             yield name, synth.BF16, bits
         else:
             yield name, synth.F32, synth.bf16_bits_to_f32(bits)
+
+
+def write_model_dir(dirpath: str, cfg: ZozonexConfig, seed: int = 0, weights_dtype: str = "bf16") -> Tuple[str, str]:
+    """Write `config.json` and `model.safetensors`; returns their paths."""
+    import os
+    from . import synth
+    os.makedirs(dirpath, exist_ok=True)
+    cpath, mpath = os.path.join(dirpath, "config.json"), os.path.join(dirpath, "model.safetensors")
+    with open(cpath, "w") as f:
+        f.write(cfg.to_json())
+    synth.write_safetensors(mpath, {n: (dt, a) for n, dt, a in iter_tensors(cfg, seed, weights_dtype)})
+    return cpath, mpath
