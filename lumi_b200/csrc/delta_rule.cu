@@ -98,23 +98,60 @@ __global__ void __launch_bounds__(NT) delta_step_kernel(DeltaArgs a, int cwl) {
     pdl_release();
     // the state belongs to the step before this one, which has ended: requested ahead of the predecessor's results
     if (STAGED && a.row_len == nullptr && tid == 0) request();
-    pdl_sync();
+    // Channel c of the head's q | k | v: its projection column, its place in the ring, its filter; false for padding.
+    const int Cq = a.G * dk, channels = 2 * Cq + a.H * dv;
+    auto channel = [&](int c, int& off, int& rc, const float*& w) {
+        if (c < dk) { off = a.off_q + kvh * dk + c; rc = kvh * dk + c; w = a.conv_q + (size_t)rc * a.taps; return true; }
+        if (c < 2 * dk) { const int k = kvh * dk + c - dk; off = a.off_k + k; rc = Cq + k; w = a.conv_k + (size_t)k * a.taps; return true; }
+        if (c - 2 * dk >= dv) return false;
+        const int v = h * dv + c - 2 * dk;
+        off = a.off_v + v; rc = 2 * Cq + v; w = a.conv_v + (size_t)v * a.taps;
+        return true;
+    };
+    // A single token: what earlier tokens put into the convolutions belongs to the steps before this one as well
+    constexpr int PRE = 2;
     const int pos0 = a.pos[slot];
+    float past[PRE], wcur[PRE];
+    if (a.ts == 1) {
+#pragma unroll
+        for (int i = 0; i < PRE; ++i) {
+            const int c = tid + i * NT;
+            int off, rc;
+            const float* w;
+            past[i] = wcur[i] = 0.f;
+            if (c < 2 * dk + dvp && channel(c, off, rc, w)) {
+                const float* ring = a.conv + (size_t)slot * a.taps * channels + rc;
+                for (int j = 0; j + 1 < a.taps; ++j) {
+                    const int p = pos0 - (a.taps - 1 - j);
+                    past[i] = fmaf(w[j], p >= 0 ? ring[(size_t)(p % a.taps) * channels] : 0.f, past[i]);
+                }
+                wcur[i] = w[a.taps - 1];
+            }
+        }
+    }
+    pdl_sync();
     const int n = pass_tokens(a.row_len, a.ctl, slot, a.ts, a.t_abs0);
     if (n == 0 && a.ts == 1) return;
     if (STAGED && a.row_len != nullptr && n > 0 && tid == 0) request();
-    const int Cq = a.G * dk, channels = 2 * Cq + a.H * dv;
     float4* St = reinterpret_cast<float4*>(STAGED ? dyn : Sg);
 
     for (int t = 0; t < n; ++t) {
         const int row = sl * a.ts + t;
         const float* pr = a.proj + (size_t)row * a.ldp;
-        for (int c = tid; c < 2 * dk + dvp; c += NT) {
-            float v = 0.f;
-            if (c < dk) v = silu_f(conv_at(a, row, t, pos0, slot, a.off_q + kvh * dk + c, kvh * dk + c, a.conv_q + (size_t)(kvh * dk + c) * a.taps));
-            else if (c < 2 * dk) v = silu_f(conv_at(a, row, t, pos0, slot, a.off_k + kvh * dk + c - dk, Cq + kvh * dk + c - dk, a.conv_k + (size_t)(kvh * dk + c - dk) * a.taps));
-            else if (c - 2 * dk < dv) v = silu_f(conv_at(a, row, t, pos0, slot, a.off_v + h * dv + c - 2 * dk, 2 * Cq + h * dv + c - 2 * dk, a.conv_v + (size_t)(h * dv + c - 2 * dk) * a.taps));
-            sm[c] = v;                                    // qs | ks | vs are contiguous
+        // (qs | ks | vs are contiguous)
+        int first = tid;
+        if (a.ts == 1) {
+#pragma unroll
+            for (int i = 0; i < PRE; ++i, first += NT) {
+                int off, rc;
+                const float* w;
+                if (first < 2 * dk + dvp) sm[first] = channel(first, off, rc, w) ? silu_f(fmaf(wcur[i], pr[off], past[i])) : 0.f;
+            }
+        }
+        for (int c = first; c < 2 * dk + dvp; c += NT) {
+            int off, rc;
+            const float* w;
+            sm[c] = channel(c, off, rc, w) ? silu_f(conv_at(a, row, t, pos0, slot, off, rc, w)) : 0.f;
         }
         __syncthreads();
         if (warp < 3) {
@@ -476,13 +513,12 @@ static size_t chunk_smem(int dk16, int dvb) {
     return sizeof(float) * (2 * (size_t)CH * chunk_sk(dk16) + (size_t)(dk16 + CH) * chunk_ss(dvb) + 2 * (size_t)CH * SA + 5 * CH);
 }
 
-// CTA = (head, block of value columns, sequence).  Warp w owns 8 NTW columns of the state, of U and of O from start to end,
-// so that between the CTA-wide products (A, P, the inverses of A's diagonal blocks) and the next chunk's staging no barrier
-// is needed.
+// CTA = (head, block of value columns, sequence).  A pair of warps owns 8 NTW columns of the state and of O from start to end,
+// each of the two half of the rows; the triangular solve, sequential in the rows, goes by columns alone.
 template <int NTW>
-__global__ void __launch_bounds__(256) delta_chunk_kernel(DeltaArgs a, int dk4, int dk16) {
+__global__ void __launch_bounds__(512) delta_chunk_kernel(DeltaArgs a, int dk4, int dk16) {
     extern __shared__ __align__(16) float sm[];
-    const int nthr = blockDim.x, nw = nthr >> 5, dvb = nw * 8 * NTW;
+    const int nthr = blockDim.x, nw = nthr >> 5, dvb = nw * 4 * NTW;
     const int SK = chunk_sk(dk16), SS = chunk_ss(dvb);
     float* Ks = sm;                                       // [CH][SK]
     float* Qs = Ks + CH * SK;
@@ -505,7 +541,7 @@ __global__ void __launch_bounds__(256) delta_chunk_kernel(DeltaArgs a, int dk4, 
         const int r = i / dvb, c = i % dvb;
         Ss[r * SS + c] = r < a.dk && v0 + c < a.dvp ? Sg[(size_t)r * a.dvp + v0 + c] : 0.f;
     }
-    const int n0 = warp * 8 * NTW;                        // this warp's columns of the block
+    const int n0 = (warp >> 1) * 8 * NTW, half = warp & 1;      // this warp's columns of the block, and its half of the rows
     const int q4 = dk16 >> 2, d4 = dvb >> 2;
     for (int t0 = 0; t0 < n; t0 += CH) {
         const int nt = min(CH, n - t0);
@@ -579,36 +615,37 @@ __global__ void __launch_bounds__(256) delta_chunk_kernel(DeltaArgs a, int dk4, 
                 }
         }
         // K S_0 and Q S_0 for this warp's columns
-        float rk[4][NTW][4], ro[4][NTW][4];
+        float rk[2][NTW][4], ro[2][NTW][4];
 #pragma unroll
-        for (int rt = 0; rt < 4; ++rt)
+        for (int r2 = 0; r2 < 2; ++r2)
 #pragma unroll
             for (int e = 0; e < NTW; ++e)
 #pragma unroll
-                for (int i = 0; i < 4; ++i) rk[rt][e][i] = ro[rt][e][i] = 0.f;
+                for (int i = 0; i < 4; ++i) rk[r2][e][i] = ro[r2][e][i] = 0.f;
         for (int ks = 0; ks < dk16; ks += 8) {
             FragB fb[NTW];
 #pragma unroll
             for (int e = 0; e < NTW; ++e) fb[e] = frag_b(Ss + ks * SS + n0 + 8 * e, SS, g, tq);
 #pragma unroll
-            for (int rt = 0; rt < 4; ++rt) {
+            for (int r2 = 0; r2 < 2; ++r2) {
+                const int rt = half + 2 * r2;             // row tiles of 16: the read-out below grows with the row, so they alternate
                 const FragA fk = frag_a(Ks + rt * 16 * SK + ks, SK, g, tq);
 #pragma unroll
-                for (int e = 0; e < NTW; ++e) mma3(rk[rt][e], fk, fb[e]);
+                for (int e = 0; e < NTW; ++e) mma3(rk[r2][e], fk, fb[e]);
                 const FragA fq = frag_a(Qs + rt * 16 * SK + ks, SK, g, tq);
 #pragma unroll
-                for (int e = 0; e < NTW; ++e) mma3(ro[rt][e], fq, fb[e]);
+                for (int e = 0; e < NTW; ++e) mma3(ro[r2][e], fq, fb[e]);
             }
         }
 #pragma unroll
-        for (int rt = 0; rt < 4; ++rt)
+        for (int r2 = 0; r2 < 2; ++r2)
 #pragma unroll
             for (int e = 0; e < NTW; ++e)
 #pragma unroll
                 for (int i = 0; i < 4; ++i) {
-                    const int t = rt * 16 + g + (i >> 1) * 8, c = n0 + 8 * e + 2 * tq + (i & 1);
-                    Us[t * SS + c] = be[t] * (Us[t * SS + c] - eG[t] * rk[rt][e][i]);
-                    ro[rt][e][i] *= eG[t];
+                    const int rt = half + 2 * r2, t = rt * 16 + g + (i >> 1) * 8, c = n0 + 8 * e + 2 * tq + (i & 1);
+                    Us[t * SS + c] = be[t] * (Us[t * SS + c] - eG[t] * rk[r2][e][i]);
+                    ro[r2][e][i] *= eG[t];
                 }
         __syncthreads();                                  // A and P are complete
         if (warp < 4) {
@@ -630,46 +667,39 @@ __global__ void __launch_bounds__(256) delta_chunk_kernel(DeltaArgs a, int dk4, 
             }
         }
         __syncthreads();
-        // forward substitution by blocks of 16 rows, each warp for its own columns
+        // forward substitution by blocks of 16 rows, eight columns per warp
+        if (warp * 8 < dvb) {
+            float* Uw = Us + warp * 8;
 #pragma unroll
-        for (int i4 = 0; i4 < 4; ++i4) {
-            float acc[NTW][4] = {};
+            for (int i4 = 0; i4 < 4; ++i4) {
+                float acc[2][4] = {};                     // two chains of products
 #pragma unroll
-            for (int kk = 0; kk < 2 * i4; ++kk) {
-                const FragA fa = frag_a(As + i4 * 16 * SA + kk * 8, SA, g, tq);
-#pragma unroll
-                for (int e = 0; e < NTW; ++e) mma3(acc[e], fa, frag_b(Us + kk * 8 * SS + n0 + 8 * e, SS, g, tq));
-            }
-#pragma unroll
-            for (int e = 0; e < NTW; ++e)
+                for (int kk = 0; kk < 2 * i4; ++kk)
+                    mma3(acc[kk & 1], frag_a(As + i4 * 16 * SA + kk * 8, SA, g, tq), frag_b(Uw + kk * 8 * SS, SS, g, tq));
 #pragma unroll
                 for (int i = 0; i < 4; ++i) {
-                    const int t = i4 * 16 + g + (i >> 1) * 8, c = n0 + 8 * e + 2 * tq + (i & 1);
-                    Us[t * SS + c] -= acc[e][i];
-                    acc[e][i] = 0.f;
+                    Uw[(i4 * 16 + g + (i >> 1) * 8) * SS + 2 * tq + (i & 1)] -= acc[0][i] + acc[1][i];
+                    acc[0][i] = acc[1][i] = 0.f;
                 }
-            __syncwarp();
+                __syncwarp();
 #pragma unroll
-            for (int kk = 0; kk < 2; ++kk) {
-                const FragA fa = frag_a(As + i4 * 16 * SA + i4 * 16 + kk * 8, SA, g, tq);
+                for (int kk = 0; kk < 2; ++kk)
+                    mma3(acc[kk], frag_a(As + i4 * 16 * SA + i4 * 16 + kk * 8, SA, g, tq), frag_b(Uw + (i4 * 16 + kk * 8) * SS, SS, g, tq));
+                __syncwarp();
 #pragma unroll
-                for (int e = 0; e < NTW; ++e) mma3(acc[e], fa, frag_b(Us + (i4 * 16 + kk * 8) * SS + n0 + 8 * e, SS, g, tq));
+                for (int i = 0; i < 4; ++i) Uw[(i4 * 16 + g + (i >> 1) * 8) * SS + 2 * tq + (i & 1)] = acc[0][i] + acc[1][i];
+                __syncwarp();
             }
-            __syncwarp();
-#pragma unroll
-            for (int e = 0; e < NTW; ++e)
-#pragma unroll
-                for (int i = 0; i < 4; ++i) Us[(i4 * 16 + g + (i >> 1) * 8) * SS + n0 + 8 * e + 2 * tq + (i & 1)] = acc[e][i];
-            __syncwarp();
         }
+        __syncthreads();
         // read-out
 #pragma unroll
-        for (int rt = 0; rt < 4; ++rt) {
-#pragma unroll
+        for (int r2 = 0; r2 < 2; ++r2) {
+            const int rt = half + 2 * r2;
             for (int kk = 0; kk < 2 * rt + 2; ++kk) {
                 const FragA fa = frag_a(Ps + rt * 16 * SA + kk * 8, SA, g, tq);
 #pragma unroll
-                for (int e = 0; e < NTW; ++e) mma3(ro[rt][e], fa, frag_b(Us + kk * 8 * SS + n0 + 8 * e, SS, g, tq));
+                for (int e = 0; e < NTW; ++e) mma3(ro[r2][e], fa, frag_b(Us + kk * 8 * SS + n0 + 8 * e, SS, g, tq));
             }
 #pragma unroll
             for (int e = 0; e < NTW; ++e)
@@ -677,13 +707,13 @@ __global__ void __launch_bounds__(256) delta_chunk_kernel(DeltaArgs a, int dk4, 
                 for (int i = 0; i < 4; i += 2) {
                     const int t = rt * 16 + g + (i >> 1) * 8, c = v0 + n0 + 8 * e + 2 * tq;
                     if (t < nt && c < a.dvp)
-                        *reinterpret_cast<float2*>(a.o32 + ((size_t)(sl * a.ts + t0 + t) * a.H + h) * a.dvp + c) = make_float2(ro[rt][e][i], ro[rt][e][i + 1]);
+                        *reinterpret_cast<float2*>(a.o32 + ((size_t)(sl * a.ts + t0 + t) * a.H + h) * a.dvp + c) = make_float2(ro[r2][e][i], ro[r2][e][i + 1]);
                 }
         }
         // state: e^(G_C) S + K^T diag(e^(G_C - G)) U, 64 rows of the state at a time
         const float dec = eG[CH - 1];
         for (int mb = 0; mb < dk16; mb += 64) {
-            float acc[4][NTW][4] = {};
+            float acc[2][NTW][4] = {};
             for (int kk = 0; kk < 8; ++kk) {
                 FragB fb[NTW];
                 const float e0 = eE[kk * 8 + tq], e1 = eE[kk * 8 + tq + 4];
@@ -693,27 +723,30 @@ __global__ void __launch_bounds__(256) delta_chunk_kernel(DeltaArgs a, int dk4, 
                     fb[e].v[0] = split_tf32(up[tq * SS] * e0); fb[e].v[1] = split_tf32(up[(tq + 4) * SS] * e1);
                 }
 #pragma unroll
-                for (int mt = 0; mt < 4; ++mt) {
+                for (int m2 = 0; m2 < 2; ++m2) {
+                    const int mt = half + 2 * m2;
                     if (mb + mt * 16 < dk16) {
                         const float* kp = Ks + kk * 8 * SK + mb + mt * 16 + g;        // A[m][k] = K[k][m]
                         FragA fa;
                         fa.v[0] = split_tf32(kp[tq * SK]); fa.v[1] = split_tf32(kp[tq * SK + 8]);
                         fa.v[2] = split_tf32(kp[(tq + 4) * SK]); fa.v[3] = split_tf32(kp[(tq + 4) * SK + 8]);
 #pragma unroll
-                        for (int e = 0; e < NTW; ++e) mma3(acc[mt][e], fa, fb[e]);
+                        for (int e = 0; e < NTW; ++e) mma3(acc[m2][e], fa, fb[e]);
                     }
                 }
             }
 #pragma unroll
-            for (int mt = 0; mt < 4; ++mt)
+            for (int m2 = 0; m2 < 2; ++m2) {
+                const int mt = half + 2 * m2;
                 if (mb + mt * 16 < dk16)
 #pragma unroll
                     for (int e = 0; e < NTW; ++e)
 #pragma unroll
                         for (int i = 0; i < 4; ++i) {
                             float* sp = Ss + (mb + mt * 16 + g + (i >> 1) * 8) * SS + n0 + 8 * e + 2 * tq + (i & 1);
-                            *sp = fmaf(dec, *sp, acc[mt][e][i]);
+                            *sp = fmaf(dec, *sp, acc[m2][e][i]);
                         }
+            }
         }
     }
     __syncthreads();
@@ -757,8 +790,9 @@ cudaError_t launch_tail(const DeltaArgs& a, cudaStream_t st) {
     return cudaGetLastError();
 }
 
-// columns per CTA: as many as the value dimension has and shared memory takes; false if not even 32 fit
-bool chunk_shape(int dk, int dv, int* nw, int* ntw) {
+// columns per CTA (nw warp pairs of 8 ntw each): as many as the value dimension has and shared memory takes, fewer where the
+// heads of the batch alone would leave SMs idle; false if not even 32 fit
+bool chunk_shape(int dk, int dv, long heads, int* nw, int* ntw) {
     if (dk > kMaxChunkDim) return false;
     const int dk16 = (dk + 15) / 16 * 16;
     const int cand[3][2] = {{8, 2}, {4, 2}, {4, 1}};      // 128, 64, 32 columns
@@ -766,6 +800,7 @@ bool chunk_shape(int dk, int dv, int* nw, int* ntw) {
         const int dvb = cand[i][0] * cand[i][1] * 8;
         if (i < 2 && dv <= dvb / 2) continue;             // half of the columns would be empty
         if (chunk_smem(dk16, dvb) > kSmemMax) continue;
+        if (i < 2 && heads * ((dv + dvb - 1) / dvb) <= 74) continue;
         *nw = cand[i][0]; *ntw = cand[i][1];
         return true;
     }
@@ -792,12 +827,12 @@ cudaError_t launch_delta_step(const DeltaArgs& a, cudaStream_t st, int* launches
 
 bool delta_chunk_supported(int dk, int dv) {
     int nw, ntw;
-    return chunk_shape(dk, dv, &nw, &ntw);
+    return chunk_shape(dk, dv, 1 << 20, &nw, &ntw) || chunk_shape(dk, dv, 1, &nw, &ntw);
 }
 
 cudaError_t launch_delta_chunk(const DeltaArgs& a, cudaStream_t st, int* launches) {
     int nw = 0, ntw = 0;
-    if (!chunk_shape(a.dk, a.dv, &nw, &ntw)) return cudaErrorInvalidValue;
+    if (!chunk_shape(a.dk, a.dv, (long)a.nseq * a.H, &nw, &ntw)) return cudaErrorInvalidValue;
     const int dk4 = (a.dk + 3) / 4 * 4, dk16 = (a.dk + 15) / 16 * 16, dvb = nw * ntw * 8;
     const size_t smem = chunk_smem(dk16, dvb);
     const long ow = (long)a.nseq * a.ts * a.H;
@@ -820,11 +855,11 @@ cudaError_t launch_delta_chunk(const DeltaArgs& a, cudaStream_t st, int* launche
     if (ntw == 2) {
         e = cudaFuncSetAttribute(delta_chunk_kernel<2>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
         if (e != cudaSuccess) return e;
-        delta_chunk_kernel<2><<<grid, nw * 32, smem, st>>>(a, dk4, dk16);
+        delta_chunk_kernel<2><<<grid, nw * 64, smem, st>>>(a, dk4, dk16);
     } else {
         e = cudaFuncSetAttribute(delta_chunk_kernel<1>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
         if (e != cudaSuccess) return e;
-        delta_chunk_kernel<1><<<grid, nw * 32, smem, st>>>(a, dk4, dk16);
+        delta_chunk_kernel<1><<<grid, nw * 64, smem, st>>>(a, dk4, dk16);
     }
     if ((e = cudaGetLastError()) != cudaSuccess) return e;
     delta_out_kernel<<<(unsigned)((ow + 7) / 8), 256, 0, st>>>(a);

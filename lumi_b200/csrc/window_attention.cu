@@ -179,7 +179,7 @@ constexpr int kWinSliceMin = 256;                         // tokens from which a
 // Grid: (groups of query rows over all sequences, kv head x head subgroup, context slices).  A column m of a warp's 16 is
 // (row m / hb, head m % hb) with hb = heads of the subgroup (16 at most).  NT: 8-element tiles of the value row.
 template <int NT, bool DECODE>
-__global__ void __launch_bounds__(128) win_mma_kernel(WinAttnArgs a, int hb, int q_rows, int groups_per_seq) {
+__global__ void __launch_bounds__(128, NT <= 8 ? 4 : (NT <= 16 ? 3 : 2)) win_mma_kernel(WinAttnArgs a, int hb, int q_rows, int groups_per_seq) {
     extern __shared__ __align__(16) unsigned char smem_raw[];
     __shared__ int is_last;
     const WinShape s = shape_of(a);
@@ -353,16 +353,30 @@ __global__ void __launch_bounds__(128) win_mma_kernel(WinAttnArgs a, int hb, int
             // a page that every used column of the warp sees whole needs no mask (unused columns may then hold anything finite)
             const bool whole = p0 + kPageTokens - 1 <= (DECODE ? hi : pos0 + set * q_rows) && (a.m.window <= 0 || p0 > whi - a.m.window);
             float tm[2] = {kNoScore, kNoScore};
+            if (!whole) {
+#pragma unroll
+                for (int st = 0; st < STRIPS; ++st)
+#pragma unroll
+                    for (int e = 0; e < 2; ++e)
+#pragma unroll
+                        for (int i = 0; i < 4; ++i) {
+                            const int p = p0 + (strip0 + st) * 16 + e * 8 + 2 * tq + (i & 1), c = i >> 1;
+                            sc[st][e][i] = p <= last[c] && p > first[c] ? sc[st][e][i] * sc2 : kNoScore;
+                        }
+            } else {
+#pragma unroll
+                for (int st = 0; st < STRIPS; ++st)
+#pragma unroll
+                    for (int e = 0; e < 2; ++e)
+#pragma unroll
+                        for (int i = 0; i < 4; ++i) sc[st][e][i] *= sc2;
+            }
 #pragma unroll
             for (int st = 0; st < STRIPS; ++st)
 #pragma unroll
                 for (int e = 0; e < 2; ++e)
 #pragma unroll
-                    for (int i = 0; i < 4; ++i) {
-                        const int p = p0 + (strip0 + st) * 16 + e * 8 + 2 * tq + (i & 1), c = i >> 1;
-                        sc[st][e][i] = whole || (p <= last[c] && p > first[c]) ? sc[st][e][i] * sc2 : kNoScore;
-                        tm[c] = fmaxf(tm[c], sc[st][e][i]);
-                    }
+                    for (int i = 0; i < 4; ++i) tm[i >> 1] = fmaxf(tm[i >> 1], sc[st][e][i]);
             float f[2], mu[2];
 #pragma unroll
             for (int c = 0; c < 2; ++c) {

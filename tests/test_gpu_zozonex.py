@@ -178,7 +178,7 @@ def test_attention_alone(H, G, dk, dv, window, bf16):
     T = 230
     proj, off = attention_rows(2, T, H, G, dk, dv, dk + dv)
     scale = 1.7 * dk ** -0.5
-    tol = 2e-3 if bf16 else 2e-5            # (a key on a rounding border may fall to the other side)
+    tol = 4e-3 if bf16 else 2e-5            # (a key on a rounding border may fall to the other side)
     whole_pages = (max(window, 1) + T - 1 + 63) // 64 if window else (T + 63) // 64
     small_pages = (max(window, 1) + 70 - 1 + 63) // 64 if window else whole_pages
     ref = attention_reference(proj, off, H, G, dk, dv, window, scale, bf16=bf16)
