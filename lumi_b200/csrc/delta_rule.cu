@@ -65,7 +65,7 @@ __device__ __forceinline__ bool state_wait(uint64_t* bar) {
 // columns; S^T k and S^T q are taken in one walk over the old state (S_t^T q = g S_{t-1}^T q + (k.q) u), so a token needs one
 // reduction.  STAGED = false: the state stays in global memory (heads beyond shared memory).
 template <int NT, bool STAGED>
-__global__ void __launch_bounds__(NT) delta_step_kernel(DeltaArgs a, int cwl) {
+__global__ void __launch_bounds__(NT, NT == 128 ? 8 : 5) delta_step_kernel(DeltaArgs a, int cwl) {
     extern __shared__ __align__(128) float dyn[];
     __shared__ __align__(8) uint64_t bar;
     const int h = blockIdx.x, sl = blockIdx.y, slot = a.b0 + sl;
@@ -110,7 +110,7 @@ __global__ void __launch_bounds__(NT) delta_step_kernel(DeltaArgs a, int cwl) {
     };
     // A single token: what earlier tokens put into the convolutions belongs to the steps before this one as well
     constexpr int PRE = 2;
-    const int pos0 = a.pos[slot];
+    const int pos0 = a.pos[slot], here = pos0 % a.taps;
     float past[PRE], wcur[PRE];
     if (a.ts == 1) {
 #pragma unroll
@@ -122,8 +122,8 @@ __global__ void __launch_bounds__(NT) delta_step_kernel(DeltaArgs a, int cwl) {
             if (c < 2 * dk + dvp && channel(c, off, rc, w)) {
                 const float* ring = a.conv + (size_t)slot * a.taps * channels + rc;
                 for (int j = 0; j + 1 < a.taps; ++j) {
-                    const int p = pos0 - (a.taps - 1 - j);
-                    past[i] = fmaf(w[j], p >= 0 ? ring[(size_t)(p % a.taps) * channels] : 0.f, past[i]);
+                    const int d = a.taps - 1 - j, rs = here - d;          // ring slot of position pos0 - d
+                    past[i] = fmaf(w[j], pos0 >= d ? ring[(size_t)(rs < 0 ? rs + a.taps : rs) * channels] : 0.f, past[i]);
                 }
                 wcur[i] = w[a.taps - 1];
             }
@@ -240,7 +240,7 @@ __global__ void __launch_bounds__(NT) delta_step_kernel(DeltaArgs a, int cwl) {
     }
     if (a.ts == 1) {                                      // this token's raw convolution inputs
         const float* pr = a.proj + (size_t)sl * a.ldp;
-        float* ring = a.conv + ((size_t)slot * a.taps + pos0 % a.taps) * channels;
+        float* ring = a.conv + ((size_t)slot * a.taps + here) * channels;
         if (h % (a.H / a.G) == 0) {
             for (int c = tid; c < dk; c += NT) {
                 ring[kvh * dk + c] = pr[a.off_q + kvh * dk + c];
@@ -249,7 +249,8 @@ __global__ void __launch_bounds__(NT) delta_step_kernel(DeltaArgs a, int cwl) {
         }
         for (int c = tid; c < dv; c += NT) ring[2 * Cq + h * dv + c] = pr[a.off_v + h * dv + c];
     }
-    if (STAGED && tid == 0) asm volatile("cp.async.bulk.wait_group 0;" ::: "memory");
+    // the memory of the CTA has been read; the writes themselves end with the kernel
+    if (STAGED && tid == 0) asm volatile("cp.async.bulk.wait_group.read 0;" ::: "memory");
 }
 
 // After a pass of several tokens: the last taps - 1 raw inputs of every channel go into the ring (a launch of its own, since

@@ -177,20 +177,22 @@ constexpr int kWinSlices = 16;
 constexpr int kWinSliceMin = 256;                         // tokens from which a slice of the context is worth a CTA
 
 // Grid: (groups of query rows over all sequences, kv head x head subgroup, context slices).  A column m of a warp's 16 is
-// (row m / hb, head m % hb) with hb = heads of the subgroup (16 at most).  NT: 8-element tiles of the value row.
-template <int NT, bool DECODE>
+// (row m / hb, head m % hb) with hb = heads of the subgroup (16 at most).  NT: 8-element tiles of the value row, at least;
+// NK > 0: the key row is exactly NK times 16 elements and the value row exactly NT tiles, so that strides and loops are constants.
+template <int NT, int NK, bool DECODE>
 __global__ void __launch_bounds__(128, NT <= 8 ? 4 : (NT <= 16 ? 3 : 2)) win_mma_kernel(WinAttnArgs a, int hb, int q_rows, int groups_per_seq) {
     extern __shared__ __align__(16) unsigned char smem_raw[];
     __shared__ int is_last;
     const WinShape s = shape_of(a);
-    const int KS = a.dk_pad + kPadRow, VS = a.dv_pad + kPadRow;
+    const int DKP = NK > 0 ? NK * 16 : a.dk_pad, DVP = NK > 0 ? NT * 8 : a.dv_pad;
+    const int KS = DKP + kPadRow, VS = DVP + kPadRow;
     constexpr int QW = DECODE ? 1 : 4;                    // sets of 16 query columns
     __nv_bfloat16* stage = reinterpret_cast<__nv_bfloat16*>(smem_raw);
     const int stage_elems = kPageTokens * (KS + VS);
     __nv_bfloat16* qh = stage + kWinStages * stage_elems;               // [QW * 16][KS] Q as bf16 halves
     __nv_bfloat16* ql = qh + QW * 16 * KS;
     __nv_bfloat16* kn = ql + QW * 16 * KS;                              // decode: the new token's rows as the cache holds them
-    __nv_bfloat16* vn = kn + a.dk_pad;
+    __nv_bfloat16* vn = kn + DKP;
 
     const int grp = blockIdx.x, kvh = blockIdx.y % a.G, sub = blockIdx.y / a.G, split = blockIdx.z, nsplit = gridDim.z;
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, tq = lane & 3;
@@ -222,7 +224,7 @@ __global__ void __launch_bounds__(128, NT <= 8 ? 4 : (NT <= 16 ? 3 : 2)) win_mma
     const int pg0 = lo / kPageTokens, pages = hi / kPageTokens - pg0 + 1;
     const int per = (pages + nsplit - 1) / nsplit, pb = pg0 + split * per, pe = min(pg0 + pages, pb + per);
     const int local = DECODE && a.append ? pos0 : -1;     // the row that this launch itself appends
-    const int kc = a.dk_pad / 8, vc = a.dv_pad / 8;       // 16-byte chunks per row
+    const int kc = DKP / 8, vc = DVP / 8;       // 16-byte chunks per row
     // this thread's first chunk of a page and the step to its next one (a division per chunk would cost more than the copy)
     const int kr0 = tid / kc, kc0 = tid % kc, kdr = 128 / kc, kdc = 128 % kc;
     const int vr0 = tid / vc, vc0 = tid % vc, vdr = 128 / vc, vdc = 128 % vc;
@@ -230,17 +232,17 @@ __global__ void __launch_bounds__(128, NT <= 8 ? 4 : (NT <= 16 ? 3 : 2)) win_mma
         __nv_bfloat16* ks = stage + ((pg - pb) % kWinStages) * stage_elems;
         __nv_bfloat16* vs = ks + kPageTokens * KS;
         const int pidx = pt[pg % a.pages_per_seq];
-        const __nv_bfloat16* kp = pool + (size_t)pidx * s.page_elems + (size_t)kvh * kPageTokens * (a.dk_pad + a.dv_pad);
+        const __nv_bfloat16* kp = pool + (size_t)pidx * s.page_elems + (size_t)kvh * kPageTokens * (DKP + DVP);
         const __nv_bfloat16* vp = kp + s.v_off;
         for (int r = kr0, c = kc0; r < kPageTokens;) {
             const int p = pg * kPageTokens + r;
-            cp16b(ks + r * KS + c * 8, kp + r * a.dk_pad + c * 8, p >= lo && p <= hi && p != local);
+            cp16b(ks + r * KS + c * 8, kp + r * DKP + c * 8, p >= lo && p <= hi && p != local);
             r += kdr; c += kdc;
             if (c >= kc) { c -= kc; ++r; }
         }
         for (int r = vr0, c = vc0; r < kPageTokens;) {
             const int p = pg * kPageTokens + r;
-            cp16b(vs + r * VS + c * 8, vp + r * a.dv_pad + c * 8, p >= lo && p <= hi && p != local);
+            cp16b(vs + r * VS + c * 8, vp + r * DVP + c * 8, p >= lo && p <= hi && p != local);
             r += vdr; c += vdc;
             if (c >= vc) { c -= vc; ++r; }
         }
@@ -270,7 +272,7 @@ __global__ void __launch_bounds__(128, NT <= 8 ? 4 : (NT <= 16 ? 3 : 2)) win_mma
             }
 #pragma unroll
             for (int i = 0; i < kMmaDim / 32; ++i)
-                if (lane + 32 * i < a.dk_pad) bf16_halves(v[j][i] * r, qh[(m0 + j) * KS + lane + 32 * i], ql[(m0 + j) * KS + lane + 32 * i]);
+                if (lane + 32 * i < DKP) bf16_halves(v[j][i] * r, qh[(m0 + j) * KS + lane + 32 * i], ql[(m0 + j) * KS + lane + 32 * i]);
         }
     }
     if (DECODE && a.append) {
@@ -278,16 +280,16 @@ __global__ void __launch_bounds__(128, NT <= 8 ? 4 : (NT <= 16 ? 3 : 2)) win_mma
         const float* v = a.proj + (size_t)(sl * a.ts) * a.ldp + a.off_v + kvh * a.dv;
         if (warp == 0) {
             const float r = a.m.qk_norm ? rms_factor(k, a.dk, a.eps, lane) : 1.f;
-            for (int c = lane; c < a.dk_pad; c += 32) kn[c] = __float2bfloat16_rn(c < a.dk ? k[c] * r : 0.f);
+            for (int c = lane; c < DKP; c += 32) kn[c] = __float2bfloat16_rn(c < a.dk ? k[c] * r : 0.f);
         } else if (warp == 1) {
-            for (int c = lane; c < a.dv_pad; c += 32) vn[c] = __float2bfloat16_rn(c < a.dv ? v[c] : 0.f);
+            for (int c = lane; c < DVP; c += 32) vn[c] = __float2bfloat16_rn(c < a.dv ? v[c] : 0.f);
         }
         __syncthreads();
         if (split == 0 && sub == 0) {
             __nv_bfloat16* kd = pool + k_row(a, s, pt, kvh, pos0);
             __nv_bfloat16* vd = pool + v_row(a, s, pt, kvh, pos0);
-            for (int c = tid; c < a.dk_pad; c += 128) kd[c] = kn[c];
-            for (int c = tid; c < a.dv_pad; c += 128) vd[c] = vn[c];
+            for (int c = tid; c < DKP; c += 128) kd[c] = kn[c];
+            for (int c = tid; c < DVP; c += 128) vd[c] = vn[c];
         }
     }
 
@@ -307,7 +309,7 @@ __global__ void __launch_bounds__(128, NT <= 8 ? 4 : (NT <= 16 ? 3 : 2)) win_mma
     float o[NT][4];
 #pragma unroll
     for (int i = 0; i < NT; ++i) { o[i][0] = 0.f; o[i][1] = 0.f; o[i][2] = 0.f; o[i][3] = 0.f; }
-    const int nks = a.dk_pad / 16, ndn = a.dv_pad / 16;
+    const int nks = DKP / 16, ndn = DVP / 16;
     constexpr int STRIPS = DECODE ? 1 : 4;                // 16-token strips of a page that one warp works on
     // rows of this warp span [wlo, whi]; a page outside of it has nothing for the warp
     const int whi = DECODE ? hi : min(hi, pos0 + (set + 1) * q_rows - 1);
@@ -321,8 +323,8 @@ __global__ void __launch_bounds__(128, NT <= 8 ? 4 : (NT <= 16 ? 3 : 2)) win_mma
         __nv_bfloat16* vs = ks + kPageTokens * KS;
         if (DECODE && local >= pg * kPageTokens && local < (pg + 1) * kPageTokens) {
             const int r = local - pg * kPageTokens;
-            for (int c = tid; c < a.dk_pad; c += 128) ks[r * KS + c] = kn[c];
-            for (int c = tid; c < a.dv_pad; c += 128) vs[r * VS + c] = vn[c];
+            for (int c = tid; c < DKP; c += 128) ks[r * KS + c] = kn[c];
+            for (int c = tid; c < DVP; c += 128) vs[r * VS + c] = vn[c];
             __syncthreads();
         }
         const int p0 = pg * kPageTokens;
@@ -333,7 +335,7 @@ __global__ void __launch_bounds__(128, NT <= 8 ? 4 : (NT <= 16 ? 3 : 2)) win_mma
 #pragma unroll
                 for (int e = 0; e < 2; ++e) { sc[st][e][0] = 0.f; sc[st][e][1] = 0.f; sc[st][e][2] = 0.f; sc[st][e][3] = 0.f; }
             const int strip0 = DECODE ? warp : 0;
-#pragma unroll 2
+#pragma unroll(NK > 0 ? NK : 2)
             for (int k16 = 0; k16 < nks; ++k16) {
                 uint32_t fh[4], fl[4];
                 const int qo = (set * 16 + (lane & 15)) * KS + k16 * 16 + (lane >> 4) * 8;
@@ -459,7 +461,7 @@ __global__ void __launch_bounds__(128, NT <= 8 ? 4 : (NT <= 16 ? 3 : 2)) win_mma
     }
     // decode: the four warps' shares in warp order (the stages are free)
     __syncthreads();
-    const int CW = a.dv_pad + 2;
+    const int CW = DVP + 2;
     float* comb = reinterpret_cast<float*>(smem_raw);     // [4][16][CW]: maximum, sum, context
     {
         float* mine = comb + (size_t)warp * 16 * CW;
@@ -469,7 +471,7 @@ __global__ void __launch_bounds__(128, NT <= 8 ? 4 : (NT <= 16 ? 3 : 2)) win_mma
             if (tq == 0) { mine[m * CW] = mx[c]; mine[m * CW + 1] = ls[c]; }
 #pragma unroll
             for (int i = 0; i < NT; ++i)
-                if (i * 8 < a.dv_pad) { mine[m * CW + 2 + i * 8 + 2 * tq] = o[i][2 * c]; mine[m * CW + 3 + i * 8 + 2 * tq] = o[i][2 * c + 1]; }
+                if (i * 8 < DVP) { mine[m * CW + 2 + i * 8 + 2 * tq] = o[i][2 * c]; mine[m * CW + 3 + i * 8 + 2 * tq] = o[i][2 * c + 1]; }
         }
     }
     __syncthreads();
@@ -550,7 +552,7 @@ size_t mma_smem(const WinAttnArgs& a, bool decode) {
     return std::max(stages, decode ? comb : (size_t)0);
 }
 
-template <int NT>
+template <int NT, int NK>
 cudaError_t launch_mma(const WinAttnArgs& a, cudaStream_t st) {
     const bool decode = a.ts == 1;
     const int hb = head_block(a.m), hpk = a.H / a.G, subs = (hpk + hb - 1) / hb;
@@ -563,13 +565,13 @@ cudaError_t launch_mma(const WinAttnArgs& a, cudaStream_t st) {
             nsplit = std::min<int>({(int)((2L * 148 + units - 1) / units), (ctx + kWinSliceMin - 1) / kWinSliceMin, kWinSlices});
             if (nsplit < 1) nsplit = 1;
         }
-        auto kern = win_mma_kernel<NT, true>;
+        auto kern = win_mma_kernel<NT, NK, true>;
         cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
         if (e != cudaSuccess) return e;
         return launch_dep(kern, dim3(a.nseq, a.G * subs, nsplit), 128, smem, st, a, hb, 1, 1);
     }
     const int q_rows = 16 / hb, gps = (a.ts + 4 * q_rows - 1) / (4 * q_rows);
-    auto kern = win_mma_kernel<NT, false>;
+    auto kern = win_mma_kernel<NT, NK, false>;
     cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     if (e != cudaSuccess) return e;
     return launch_dep(kern, dim3((unsigned)a.nseq * gps, a.G * subs, 1), 128, smem, st, a, hb, q_rows, gps);
@@ -607,13 +609,17 @@ cudaError_t launch_window_attention(const WinAttnArgs& a, cudaStream_t st, int* 
     }
     *launches += 1;
     if (!mma) return a.kv_is_f32 ? simple<float>(a, st) : simple<__nv_bfloat16>(a, st);
-    const int nt = a.dv_pad / 8;
-    if (nt <= 4) return launch_mma<4>(a, st);
-    if (nt <= 8) return launch_mma<8>(a, st);
-    if (nt <= 12) return launch_mma<12>(a, st);
-    if (nt <= 16) return launch_mma<16>(a, st);
-    if (nt <= 24) return launch_mma<24>(a, st);
-    return launch_mma<32>(a, st);
+    const int nt = a.dv_pad / 8, nk = a.dk_pad / 16;
+    if (nt == 4 && nk == 2) return launch_mma<4, 2>(a, st);
+    if (nt == 8 && nk == 4) return launch_mma<8, 4>(a, st);
+    if (nt == 12 && nk == 6) return launch_mma<12, 6>(a, st);
+    if (nt == 16 && nk == 8) return launch_mma<16, 8>(a, st);
+    if (nt <= 4) return launch_mma<4, 0>(a, st);
+    if (nt <= 8) return launch_mma<8, 0>(a, st);
+    if (nt <= 12) return launch_mma<12, 0>(a, st);
+    if (nt <= 16) return launch_mma<16, 0>(a, st);
+    if (nt <= 24) return launch_mma<24, 0>(a, st);
+    return launch_mma<32, 0>(a, st);
 }
 
 }  // namespace lumi
