@@ -116,7 +116,9 @@ int32_t lumi_model_info(const lumi_model* m, int64_t* out12);
 /* ---- sessions: replaces NmModel::init_states + LayerState (inference/src/model.rs:112-159,
  *      731-763) for `max_batch` independent sequences ----------------------------------------- */
 
-/* Allocates SSM state (fp32, rank-1 factors for prev_bx), the attention cache for max_tokens_kv
+/* (Designs that list their layers: the attention cache is a ring of the widest window plus a slice of up to 1024 tokens, so
+ * positions may run past max_tokens_kv; where max_tokens_kv is smaller than the window, or a layer has none, it is the limit.)
+ * Allocates SSM state (fp32, rank-1 factors for prev_bx), the attention cache for max_tokens_kv
  * tokens per sequence (element type of the weights: bf16 or fp32; ignored for models without attention
  * layers) and the decode step's scratch, then resets every slot. */
 int32_t lumi_session_create(lumi_model* m, int32_t max_batch, int32_t max_tokens_kv, lumi_session** out);
@@ -138,6 +140,7 @@ void    lumi_session_free(lumi_session* s);
  *                         chunked SSD scan (chunk 64), attention over all rows of a slice and tensor-core GEMMs
  *                         over all prompt tokens instead of token by token (same state to rounding); "prefill_rows" =
  *                         token rows per pass of that path (default 131072; sets its workspace size: 41 KB per row);
+ *                         (designs that list their layers take slices for every prompt of two tokens and more, unless 0);
  *                         "overlap" = minimum batch (default 0 = never) from which the tensor-core path runs two
  *                         lanes of sequences side by side on prioritised streams (measured neutral: the state
  *                         step needs its L1 and cannot share an SM with the 198 KB GEMM);
