@@ -17,8 +17,9 @@ LIB = os.path.join(LIBDIR, "liblumi_b200.so")
 CLI = os.path.join(LIBDIR, "lumi-infer-b200")
 
 SOURCES = ["api.cu", "kernels.cu", "gemm_tcgen05.cu", "attention.cu", "decode_b1.cu", "block_static.cu", "prefill_ssd.cu", "safetensors.cpp",
-           "architectures.cpp", "sublayer.cu", "delta_rule.cu", "window_attention.cu"]
-HEADERS = ["internal.h", "json_min.h", "rows.cuh", "embed_post.cuh", os.path.join("..", "..", "include", "lumi_b200.h")]
+           "architectures.cpp", "sublayer.cu", "delta_rule.cu", "window_attention.cu", "block_product.cu", "retention.cu", "rglru.cu", "latent_attention.cu",
+           "moe.cu"]
+HEADERS = ["internal.h", "json_min.h", "rows.cuh", "tf32.cuh", "embed_post.cuh", os.path.join("..", "..", "include", "lumi_b200.h")]
 NVCC_FLAGS = ["-gencode", "arch=compute_100a,code=sm_100a", "-lineinfo", "-O3", "-std=c++17",
               "-Xcompiler", "-fPIC", "--expt-relaxed-constexpr", "-ccbin", "/usr/bin/g++"]
 

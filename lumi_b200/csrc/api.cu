@@ -151,7 +151,7 @@ extern "C" int32_t lumi_model_set_option(lumi_model* m, const char* name, int64_
 }
 
 // Expected shape of a tensor by its name (without the design's prefix); rank 0 = not a tensor of this model.
-static int expected_shape(const lumi_model* m, const std::string& name, int64_t shp[2], bool& wide) {
+static int expected_shape(const lumi_model* m, const std::string& name, int64_t shp[3], bool& wide) {
     const Config& c = m->cfg;
     wide = false;
     if (c.arch != nullptr) return c.arch->expected_shape(c, name, shp, wide);
@@ -191,7 +191,7 @@ extern "C" int32_t lumi_model_load_tensor(lumi_model* m, const char* name, int32
     const std::string prefix = m->cfg.arch != nullptr ? m->cfg.arch->tensor_prefix : "item.";
     if (n.rfind(prefix, 0) != 0) return LUMI_OK;          // the reference only reads names under "item." (main.rs:86)
     n = n.substr(prefix.size());
-    int64_t exp[2] = {0, 0};
+    int64_t exp[3] = {0, 0, 0};
     bool wide = false;
     const int erank = expected_shape(m, n, exp, wide);
     if (erank == 0) return LUMI_OK;                       // tensors the model never asks for are ignored, as VarBuilder does
@@ -212,12 +212,12 @@ extern "C" int32_t lumi_model_load_tensor(lumi_model* m, const char* name, int32
     if ((uint64_t)count * esz != nbytes) return fail(LUMI_E_TENSOR, "tensor '%s': %llu bytes given, shape needs %llu", name, (unsigned long long)nbytes, (unsigned long long)(count * esz));
     LUMI_CUDA(cudaSetDevice(m->device));
     DevTensor t;
-    const bool keep_width = (erank == 2) && !is_hinit && !wide;
+    const bool keep_width = (erank >= 2) && !is_hinit && !wide;
     if (keep_width && !(m->widen && dtype == LUMI_DTYPE_BF16)) {
-        if (m->wdtype >= 0 && m->wdtype != dtype) return fail(LUMI_E_TENSOR, "tensor '%s': rank-2 tensors mix F32 and BF16", name);
+        if (m->wdtype >= 0 && m->wdtype != dtype) return fail(LUMI_E_TENSOR, "tensor '%s': matrices mix F32 and BF16", name);
         m->wdtype = dtype;
         t.dtype = dtype;
-        t.rows = exp[0]; t.cols = exp[1];
+        t.rows = count / exp[erank - 1]; t.cols = exp[erank - 1];      // the leading dimensions as rows
         t.bytes = nbytes;
         LUMI_CUDA(cudaMalloc(&t.p, t.bytes));
         LUMI_CUDA(cudaMemcpy(t.p, host_data, t.bytes, cudaMemcpyHostToDevice));
@@ -231,11 +231,11 @@ extern "C" int32_t lumi_model_load_tensor(lumi_model* m, const char* name, int32
             src = tmp.data();
         }
         if (keep_width) {                                 // a bf16 matrix widened to fp32
-            if (m->wdtype >= 0 && m->wdtype != LUMI_DTYPE_F32) return fail(LUMI_E_TENSOR, "tensor '%s': rank-2 tensors mix F32 and BF16", name);
+            if (m->wdtype >= 0 && m->wdtype != LUMI_DTYPE_F32) return fail(LUMI_E_TENSOR, "tensor '%s': matrices mix F32 and BF16", name);
             m->wdtype = LUMI_DTYPE_F32;
         }
         t.dtype = LUMI_DTYPE_F32;
-        t.rows = keep_width ? exp[0] : 1; t.cols = keep_width ? exp[1] : count;
+        t.rows = keep_width ? count / exp[erank - 1] : 1; t.cols = keep_width ? exp[erank - 1] : count;
         t.bytes = (size_t)count * 4;
         LUMI_CUDA(cudaMalloc(&t.p, t.bytes));
         LUMI_CUDA(cudaMemcpy(t.p, src, t.bytes, cudaMemcpyHostToDevice));
@@ -318,13 +318,13 @@ static int32_t stack_padded(lumi_model* m, const std::vector<std::string>& names
     }
     return LUMI_OK;
 }
-// The factor of a norm whose stored weight is an offset from one, padded with zeros.
+// The factor of a norm (stored as such, or as an offset from one), padded with zeros.
 static int32_t norm_factor(lumi_model* m, const std::string& n, const float*& out) {
     DevTensor t;
     LUMI_TRY(need(m, n, t));
     std::vector<float> w(up64(t.cols), 0.f);
     LUMI_CUDA(cudaMemcpy(w.data(), t.p, (size_t)t.cols * 4, cudaMemcpyDeviceToHost));
-    for (int64_t i = 0; i < t.cols; ++i) w[i] = 1.0f + w[i];
+    if (m->cfg.norm_offset) for (int64_t i = 0; i < t.cols; ++i) w[i] = 1.0f + w[i];
     void* p = nullptr;
     LUMI_CUDA(cudaMalloc(&p, w.size() * 4));
     m->owned.push_back(p);
@@ -333,24 +333,190 @@ static int32_t norm_factor(lumi_model* m, const std::string& n, const float*& ou
     return LUMI_OK;
 }
 
+static int32_t upload(lumi_model* m, const void* host, size_t bytes, void** out) {
+    LUMI_CUDA(cudaMalloc(out, bytes));
+    m->owned.push_back(*out);
+    LUMI_CUDA(cudaMemcpy(*out, host, bytes, cudaMemcpyHostToDevice));
+    return LUMI_OK;
+}
+// A matrix of zeros in the model's element type.
+static int32_t new_matrix(lumi_model* m, int64_t rows, int64_t cols, DevTensor& out) {
+    out.dtype = m->wdtype < 0 ? LUMI_DTYPE_F32 : m->wdtype;
+    out.rows = rows; out.cols = cols;
+    out.bytes = (size_t)rows * cols * (out.dtype == LUMI_DTYPE_BF16 ? 2 : 4);
+    LUMI_CUDA(cudaMalloc(&out.p, out.bytes));
+    m->owned.push_back(out.p);
+    LUMI_CUDA(cudaMemset(out.p, 0, out.bytes));
+    return LUMI_OK;
+}
+// Rows [r0, r0 + rows) of a tensor into a matrix, as launch_pack_rows places them.
+static int32_t pack(const DevTensor& dst, const DevTensor& src, int64_t r0, int64_t rows, int64_t rg, int64_t rs, int64_t ro, int64_t co = 0, bool transpose = false) {
+    const int esz = dst.dtype == LUMI_DTYPE_BF16 ? 2 : 4;
+    LUMI_CUDA(launch_pack_rows(dst.p, dst.cols, (const char*)src.p + (size_t)r0 * src.cols * esz, rows, src.cols, esz, rg, rs, ro, co, transpose, nullptr));
+    return LUMI_OK;
+}
+static int32_t release(lumi_model* m, const std::string& n) {
+    LUMI_CUDA(cudaStreamSynchronize(nullptr));
+    LUMI_CUDA(cudaFree(m->tensors[n].p));
+    m->tensors[n].p = nullptr;
+    return LUMI_OK;
+}
+// fp32 vectors placed into one of `total` zeros; place(part, i) = where element i of a part goes
+static int32_t place_vectors(lumi_model* m, const std::vector<std::string>& names, size_t total, const float*& out, size_t (*place)(const int64_t*, size_t, size_t),
+                             const int64_t* arg) {
+    std::vector<float> all(total, 0.f), one;
+    for (size_t p = 0; p < names.size(); ++p) {
+        DevTensor t;
+        LUMI_TRY(need(m, names[p], t));
+        one.resize(t.bytes / 4);
+        LUMI_CUDA(cudaMemcpy(one.data(), t.p, t.bytes, cudaMemcpyDeviceToHost));
+        for (size_t i = 0; i < one.size(); ++i) all[place(arg, p, i)] = one[i];
+    }
+    void* d = nullptr;
+    LUMI_TRY(upload(m, all.data(), total * 4, &d));
+    out = (const float*)d;
+    return LUMI_OK;
+}
+static size_t place_at(const int64_t* offs, size_t p, size_t i) { return (size_t)offs[p] + i; }
+static size_t place_paired(const int64_t*, size_t p, size_t i) { return i / 16 * 32 + i % 16 + 16 * p; }
+// arg: block size, padded block size
+static size_t place_block_pairs(const int64_t* b, size_t p, size_t i) { return i / b[0] * 2 * b[1] + place_paired(nullptr, p, i % b[0]); }
+
+static int32_t rot_frequencies(lumi_model* m, const RotSpec& rot, const double*& out) {
+    std::vector<double> f(std::max(1, rot.dims / 2), 0.0);
+    for (int i = 0; i < rot.dims / 2; ++i) f[i] = std::pow(rot.base, -2.0 * i / rot.dims) / 3.14159265358979323846;      // half turns per position
+    void* d = nullptr;
+    LUMI_TRY(upload(m, f.data(), f.size() * sizeof(double), &d));
+    out = (const double*)d;
+    return LUMI_OK;
+}
+
+// Pre-norm layers: the mixer's weights.
+static int32_t finalize_mixer(lumi_model* m, const LayerSpec& spec, const std::string& q, SubW& s) {
+    const MixerSpec& mx = spec.mixer;
+    std::vector<int> off;
+    if (mx.kind == MIXER_RETENTION) {
+        LUMI_TRY(stack_padded(m, {q + "q", q + "k", q + "v", q + "g"}, s.in, &off));
+        s.off_q = off[0]; s.off_k = off[1]; s.off_v = off[2]; s.off_g = off[3];
+        LUMI_TRY(rot_frequencies(m, mx.rot, s.rot_freq));
+        std::vector<float> pw((size_t)mx.heads * kDecayPowers);
+        for (int h = 0; h < mx.heads; ++h) {
+            double x = 1.0;
+            for (int i = 0; i < kDecayPowers; ++i, x *= (double)spec.decay[h]) pw[(size_t)h * kDecayPowers + i] = (float)x;
+        }
+        void* d = nullptr;
+        LUMI_TRY(upload(m, pw.data(), pw.size() * 4, &d));
+        s.decay_pow = (const float*)d;
+    } else if (mx.kind == MIXER_RGLRU) {
+        LUMI_TRY(stack_padded(m, {q + "y", q + "x"}, s.in, &off));
+        s.off_y = off[0]; s.off_x = off[1];
+        const int64_t offs[2] = {off[0], off[1]};
+        LUMI_TRY(place_vectors(m, {q + "y.b", q + "x.b"}, (size_t)s.in.rows, s.in_b, place_at, offs));
+        LUMI_TRY(need_f(m, q + "conv", s.conv_q));
+        LUMI_TRY(need_f(m, q + "conv.b", s.conv_b));
+        LUMI_TRY(need_f(m, q + "lam", s.lam));
+        const int64_t bs = mx.channels / mx.blocks, bp = up64(bs);
+        DevTensor ra, ri;
+        LUMI_TRY(need(m, q + "ra", ra));
+        LUMI_TRY(need(m, q + "ri", ri));
+        LUMI_TRY(new_matrix(m, mx.blocks * 2 * bp, bp, s.rg));
+        for (int64_t b = 0; b < mx.blocks; ++b) {
+            LUMI_TRY(pack(s.rg, ra, b * bs, bs, 16, 32, b * 2 * bp));
+            LUMI_TRY(pack(s.rg, ri, b * bs, bs, 16, 32, b * 2 * bp + 16));
+        }
+        LUMI_TRY(release(m, q + "ra"));
+        LUMI_TRY(release(m, q + "ri"));
+        const int64_t sizes[2] = {bs, bp};
+        LUMI_TRY(place_vectors(m, {q + "ra.b", q + "ri.b"}, (size_t)(mx.blocks * 2 * bp), s.rg_b, place_block_pairs, sizes));
+    } else {
+        const LatentShape ls(mx);
+        LUMI_TRY(stack_padded(m, {q + "q", q + "dkv", q + "g"}, s.in, &off));
+        s.off_q = off[0]; s.off_c = off[1]; s.off_g = off[2];
+        LUMI_TRY(rot_frequencies(m, mx.rot, s.rot_freq));
+        LUMI_TRY(need_f(m, q + "dkv.norm", s.c_norm));
+        DevTensor uk, uv;
+        LUMI_TRY(need(m, q + "uk", uk));
+        LUMI_TRY(need(m, q + "uv", uv));
+        const int64_t vp = (mx.vdim + 31) / 32 * 32;
+        LUMI_TRY(new_matrix(m, (int64_t)mx.heads * ls.lp, ls.dp, s.uk));
+        LUMI_TRY(pack(s.uk, uk, 0, uk.rows, mx.dim, ls.lp, 0, 0, true));
+        LUMI_TRY(new_matrix(m, (int64_t)mx.heads * vp, ls.lp, s.uv));
+        LUMI_TRY(pack(s.uv, uv, 0, uv.rows, mx.vdim, vp, 0));
+        if (m->wdtype == LUMI_DTYPE_BF16) {
+            // keys and values of all heads as one product of a cache row: the rotated part is passed through
+            const int64_t hw = ls.dk_pad + ls.dv_pad;
+            LUMI_TRY(new_matrix(m, mx.heads * hw, ls.row, s.ukv));
+            LUMI_TRY(pack(s.ukv, uk, 0, uk.rows, mx.dim, hw, 0));
+            LUMI_TRY(pack(s.ukv, uv, 0, uv.rows, mx.vdim, hw, ls.dk_pad));
+            if (mx.rot_dim > 0) {
+                std::vector<uint16_t> eye((size_t)mx.heads * mx.rot_dim * mx.rot_dim, 0);
+                for (size_t r = 0; r < (size_t)mx.heads * mx.rot_dim; ++r) eye[r * mx.rot_dim + r % mx.rot_dim] = 0x3f80;       // 1.0
+                DevTensor id;
+                id.rows = (int64_t)mx.heads * mx.rot_dim; id.cols = mx.rot_dim;
+                LUMI_TRY(upload(m, eye.data(), eye.size() * 2, &id.p));
+                LUMI_TRY(pack(s.ukv, id, 0, id.rows, mx.rot_dim, hw, mx.dim, ls.lp));
+            }
+        }
+        LUMI_TRY(release(m, q + "uk"));
+        LUMI_TRY(release(m, q + "uv"));
+    }
+    return stack_padded(m, {q + "o"}, s.out, nullptr);
+}
+
+// Gated feed-forwards, dense or experts.
+static int32_t finalize_gated_ff(lumi_model* m, const FfSpec& f, const std::string& p, SubW& s) {
+    const int64_t ffp = up64(f.ff), ldx = m->cfg.x_ld();
+    auto paired = [&](const std::string& base, int64_t ro) -> int32_t {
+        DevTensor g, u;
+        LUMI_TRY(need(m, base + "gate", g));
+        LUMI_TRY(need(m, base + "up", u));
+        LUMI_TRY(pack(s.up, g, 0, g.rows, 16, 32, ro));
+        LUMI_TRY(pack(s.up, u, 0, u.rows, 16, 32, ro + 16));
+        LUMI_TRY(release(m, base + "gate"));
+        return release(m, base + "up");
+    };
+    if (f.experts == 0) {
+        LUMI_TRY(new_matrix(m, 2 * ffp, ldx, s.up));
+        LUMI_TRY(paired(p, 0));
+        LUMI_TRY(stack_padded(m, {p + "down"}, s.down, nullptr));
+        if (f.bias) {
+            LUMI_TRY(place_vectors(m, {p + "gate.b", p + "up.b"}, (size_t)(2 * ffp), s.up_b, place_paired, nullptr));
+            const int64_t zero[1] = {0};
+            LUMI_TRY(place_vectors(m, {p + "down.b"}, (size_t)ldx, s.down_b, place_at, zero));
+        }
+        return LUMI_OK;
+    }
+    LUMI_TRY(stack_padded(m, {p + "router"}, s.router, nullptr));
+    LUMI_TRY(new_matrix(m, f.experts * 2 * ffp, ldx, s.up));
+    LUMI_TRY(new_matrix(m, f.experts * ldx, ffp, s.down));
+    for (int64_t e = 0; e < f.experts; ++e) {
+        const std::string base = p + "e" + std::to_string(e) + ".";
+        LUMI_TRY(paired(base, e * 2 * ffp));
+        DevTensor d;
+        LUMI_TRY(need(m, base + "down", d));
+        LUMI_TRY(pack(s.down, d, 0, d.rows, d.rows, 0, e * ldx));
+        LUMI_TRY(release(m, base + "down"));
+    }
+    return LUMI_OK;
+}
+
+// A vocabulary matrix: its rows stay, its columns are padded.
+static int32_t vocab_matrix(lumi_model* m, const std::string& n, DevTensor& out) {
+    DevTensor t;
+    LUMI_TRY(need(m, n, t));
+    out = t;
+    if (t.cols == up64(t.cols)) return LUMI_OK;
+    LUMI_TRY(new_matrix(m, t.rows, up64(t.cols), out));
+    LUMI_TRY(pack(out, t, 0, t.rows, t.rows, 0, 0));
+    return release(m, n);
+}
+
 static int32_t finalize_stacked(lumi_model* m) {
     const Config& c = m->cfg;
     for (auto& kv : m->tensors) m->weight_bytes += (int64_t)kv.second.bytes;
-    {
-        // the embedding keeps its row count (the vocabulary), its columns are padded
-        DevTensor t;
-        LUMI_TRY(need(m, "embed", t));
-        m->embedding = t;
-        if (t.cols != up64(t.cols)) {
-            const size_t esz = t.dtype == LUMI_DTYPE_BF16 ? 2 : 4;
-            m->embedding.cols = up64(t.cols);
-            m->embedding.bytes = (size_t)t.rows * m->embedding.cols * esz;
-            LUMI_CUDA(cudaMalloc(&m->embedding.p, m->embedding.bytes));
-            m->owned.push_back(m->embedding.p);
-            LUMI_CUDA(cudaMemset(m->embedding.p, 0, m->embedding.bytes));
-            LUMI_CUDA(cudaMemcpy2D(m->embedding.p, m->embedding.cols * esz, t.p, t.cols * esz, t.cols * esz, t.rows, cudaMemcpyDeviceToDevice));
-        }
-    }
+    LUMI_TRY(vocab_matrix(m, "embed", m->embedding));
+    if (c.own_head) LUMI_TRY(vocab_matrix(m, "head", m->head));
+    else m->head = m->embedding;
     LUMI_TRY(norm_factor(m, "final.norm", m->final_norm_g));
     m->layers.assign(c.n_layers, Layer());
     for (int i = 0; i < c.n_layers; ++i) {
@@ -358,10 +524,18 @@ static int32_t finalize_stacked(lumi_model* m) {
         const MixerSpec& mx = c.specs[i].mixer;
         const std::string p = "l" + std::to_string(i) + ".", q = p + "mix.";
         L.spec = &c.specs[i];
+        L.kind_idx = mx.recurrent() ? m->n_recur++ : m->n_wattn++;
+        L.window = mx.window;
+        if (L.spec->weights_of >= 0) { L.s = m->layers[L.spec->weights_of].s; continue; }
         LUMI_TRY(norm_factor(m, p + "norm1", L.s.norm1));
+        if (L.spec->ff.ff > 0) LUMI_TRY(norm_factor(m, p + "norm2", L.s.norm2));
+        if (L.spec->pre_norm) {
+            LUMI_TRY(finalize_mixer(m, *L.spec, q, L.s));
+            if (L.spec->ff.ff > 0) LUMI_TRY(finalize_gated_ff(m, L.spec->ff, p + "mlp.", L.s));
+            continue;
+        }
         std::vector<int> off;
         if (mx.kind == MIXER_DELTA) {
-            L.kind_idx = m->n_delta++;
             LUMI_TRY(stack_padded(m, {q + "q", q + "k", q + "v", q + "b", q + "a", q + "g"}, L.s.in, &off));
             L.s.off_b = off[3]; L.s.off_a = off[4]; L.s.off_g = off[5];
             LUMI_TRY(need_f(m, q + "q.conv", L.s.conv_q));
@@ -371,21 +545,19 @@ static int32_t finalize_stacked(lumi_model* m) {
             LUMI_TRY(need_f(m, q + "dt_bias", L.s.dt_bias));
             LUMI_TRY(need_f(m, q + "norm", L.s.o_norm));
         } else {
-            L.kind_idx = m->n_wattn++;
-            L.window = mx.window;
             std::vector<std::string> names = {q + "q"};
             if (mx.kv_from < 0) { names.push_back(q + "k"); names.push_back(q + "v"); }
             LUMI_TRY(stack_padded(m, names, L.s.in, &off));
         }
         if (off.size() > 1) { L.s.off_k = off[1]; L.s.off_v = off[2]; }
         LUMI_TRY(stack_padded(m, {q + "o"}, L.s.out, nullptr));
-        if (L.spec->ff > 0) {
-            LUMI_TRY(norm_factor(m, p + "norm2", L.s.norm2));
+        if (L.spec->ff.ff > 0) {
             LUMI_TRY(stack_padded(m, {p + "mlp.up"}, L.s.up, nullptr));
             LUMI_TRY(stack_padded(m, {p + "mlp.down"}, L.s.down, nullptr));
         }
     }
     if (m->wdtype < 0) m->wdtype = LUMI_DTYPE_F32;
+    LUMI_CUDA(cudaDeviceSynchronize());
     m->finalized = true;
     return LUMI_OK;
 }
@@ -450,7 +622,7 @@ extern "C" int32_t lumi_model_info(const lumi_model* m, int64_t* o) {
     if (!m || !o) return fail(LUMI_E_INVALID, "null argument to lumi_model_info");
     const Config& c = m->cfg;
     o[0] = c.d_model; o[1] = c.n_layers; o[2] = c.d_state; o[3] = c.n_heads; o[4] = c.head_dim(); o[5] = c.n_groups;
-    o[6] = c.vocab; o[7] = m->n_mamba + m->n_delta; o[8] = m->n_attn + m->n_wattn; o[9] = c.in_proj_out(); o[10] = m->wdtype; o[11] = m->weight_bytes;
+    o[6] = c.vocab; o[7] = m->n_mamba + m->n_recur; o[8] = m->n_attn + m->n_wattn; o[9] = c.in_proj_out(); o[10] = m->wdtype; o[11] = m->weight_bytes;
     return LUMI_OK;
 }
 
@@ -458,39 +630,87 @@ extern "C" int32_t lumi_model_info(const lumi_model* m, int64_t* o) {
 static size_t state_h_per_seq(const Config& c) { return (size_t)c.n_heads * c.head_dim() * c.d_state; }
 
 static void free_rows(RowBufs& b) {
-    void* all[] = {b.x, b.x2, b.proj, b.mix, b.qkv, b.gates, b.y32, b.xh, b.xl, b.ah, b.al};
+    void* all[] = {b.x, b.x2, b.proj, b.mix, b.qkv, b.gates, b.y32, b.xh, b.xl, b.ah, b.al, b.ssq, b.bh, b.bl, b.qlat, b.ctx, b.lh, b.ll,
+                   b.moe.logits, b.moe.y, b.moe.h32, b.moe.gh, b.moe.gl, b.moe.hh, b.moe.hl, b.moe.plan};
     for (void* p : all) if (p) cudaFree(p);
     b = RowBufs();
 }
 
-// Widest rows of the passes over listed layers.
-struct RowWidths { size_t proj = 0, act = 0, mix = 0, qkv = 0, gates = 0; };
+// Widest rows of the passes over listed layers; `step` = what decode steps need beside slices of qkv and gates.
+struct RowWidths {
+    size_t proj = 0, act = 0, mix = 0, qkv = 0, gates = 0, step_qkv = 0, step_gates = 0, block = 0, lat_q = 0, lat_c = 0, lat_half = 0;
+    bool pre_norm = false;
+    int experts = 0, top = 0;                             // most experts, and most chosen ones, of a layer
+    size_t ffp = 0, router = 0;
+};
 static RowWidths row_widths(const lumi_model* m) {
     RowWidths w;
     w.mix = (size_t)m->cfg.x_ld();
     for (const Layer& L : m->layers) {
         const MixerSpec& x = L.spec->mixer;
+        const FfSpec& f = L.spec->ff;
+        w.pre_norm |= L.spec->pre_norm;
         w.proj = std::max(w.proj, (size_t)L.s.in.rows);
-        w.act = std::max({w.act, (size_t)L.s.out.cols, L.spec->ff > 0 ? (size_t)L.s.up.rows : 0});
+        w.act = std::max({w.act, (size_t)L.s.out.cols, f.ff > 0 && f.experts == 0 ? (size_t)(f.gated() ? L.s.down.cols : L.s.up.rows) : 0});
         if (x.kind == MIXER_DELTA) {
             const size_t dk4 = (x.dim + 3) / 4 * 4, dvp = (x.vdim + 3) / 4 * 4;
             w.mix = std::max(w.mix, x.heads * dvp);
             w.qkv = std::max(w.qkv, 2 * x.kv_heads * dk4 + x.heads * dvp);
             w.gates = std::max(w.gates, (size_t)2 * x.heads);
+        } else if (x.kind == MIXER_RETENTION) {
+            w.mix = std::max(w.mix, (size_t)x.heads * ((x.vdim + 3) / 4 * 4));
+        } else if (x.kind == MIXER_RGLRU) {
+            const size_t bp = (size_t)up64(x.channels / x.blocks);
+            w.step_qkv = std::max(w.step_qkv, (size_t)x.channels);
+            w.step_gates = std::max(w.step_gates, x.blocks * 2 * bp);
+            w.block = std::max(w.block, x.blocks * bp);
+        } else if (x.kind == MIXER_LATENT) {
+            const LatentShape ls(x);
+            w.lat_q = std::max(w.lat_q, (size_t)x.heads * ls.row);
+            w.lat_c = std::max(w.lat_c, (size_t)x.heads * ls.lp);
+            w.lat_half = std::max({w.lat_half, (size_t)x.heads * ls.lp, (size_t)x.heads * ls.dp});
+        }
+        if (f.experts > 0) {
+            w.experts = std::max(w.experts, f.experts);
+            w.top = std::max(w.top, f.top);
+            w.ffp = std::max(w.ffp, (size_t)up64(f.ff));
+            w.router = std::max(w.router, (size_t)L.s.router.rows);
         }
     }
+    w.qkv = std::max(w.qkv, w.step_qkv);
+    w.gates = std::max(w.gates, w.step_gates);
     return w;
+}
+static int32_t zeroed(lumi_session* s, void** p, size_t bytes) {
+    LUMI_CUDA(cudaMalloc(p, bytes));
+    LUMI_CUDA(cudaMemsetAsync(*p, 0, bytes, s->stream));
+    return LUMI_OK;
+}
+// Buffers of latent attention with queries in the latent space, for `rows` rows.  Not for the decode set once a step may have been captured.
+static int32_t ensure_latent_rows(lumi_session* s, RowBufs& b, size_t rows) {
+    if (rows <= b.lat_rows) return LUMI_OK;
+    const RowWidths w = row_widths(s->m);
+    if (w.lat_q == 0) return LUMI_OK;
+    LUMI_CUDA(cudaStreamSynchronize(s->stream));
+    void* old[] = {b.qlat, b.ctx, b.lh, b.ll};
+    for (void* p : old) if (p) LUMI_CUDA(cudaFree(p));
+    b.qlat = b.ctx = nullptr; b.lh = b.ll = nullptr; b.lat_rows = 0;
+    const size_t rp = (rows + 127) / 128 * 128;
+    LUMI_TRY(zeroed(s, (void**)&b.qlat, rp * w.lat_q * 4));
+    LUMI_TRY(zeroed(s, (void**)&b.ctx, rp * w.lat_c * 4));
+    if (s->m->wdtype == LUMI_DTYPE_BF16) {
+        LUMI_TRY(zeroed(s, (void**)&b.lh, rp * w.lat_half * 2));
+        LUMI_TRY(zeroed(s, (void**)&b.ll, rp * w.lat_half * 2));
+    }
+    b.lat_rows = rows;
+    return LUMI_OK;
 }
 // slices: the buffers of the chunked recurrence are needed as well.  Everything starts as zeros, so that padding stays finite.
 static int32_t alloc_rows(lumi_session* s, RowBufs& b, size_t rows, bool slices) {
     const RowWidths w = row_widths(s->m);
     const bool half = s->m->wdtype == LUMI_DTYPE_BF16;
     const size_t rp = (rows + 127) / 128 * 128, ldx = s->m->cfg.x_ld();
-    auto get = [&](auto*& p, size_t n) -> int32_t {
-        LUMI_CUDA(cudaMalloc(&p, n * sizeof(*p)));
-        LUMI_CUDA(cudaMemsetAsync(p, 0, n * sizeof(*p), s->stream));
-        return LUMI_OK;
-    };
+    auto get = [&](auto*& p, size_t n) -> int32_t { return n > 0 ? zeroed(s, (void**)&p, n * sizeof(*p)) : LUMI_OK; };
     if (b.x == nullptr) LUMI_TRY(get(b.x, rp * ldx));
     LUMI_TRY(get(b.proj, rp * w.proj));
     LUMI_TRY(get(b.mix, rp * w.mix));
@@ -501,10 +721,31 @@ static int32_t alloc_rows(lumi_session* s, RowBufs& b, size_t rows, bool slices)
         LUMI_TRY(get(b.xl, rp * ldx));
         LUMI_TRY(get(b.ah, rp * w.act));
         LUMI_TRY(get(b.al, rp * w.act));
+        LUMI_TRY(get(b.bh, rp * w.block));
+        LUMI_TRY(get(b.bl, rp * w.block));
+        if (w.pre_norm) {
+            b.ssq_stride = (int)((ldx + 127) / 128 * 4);
+            LUMI_TRY(get(b.ssq, rp * b.ssq_stride));
+        }
     }
-    if (slices && w.qkv > 0) {
-        LUMI_TRY(get(b.qkv, rp * w.qkv));
-        LUMI_TRY(get(b.gates, rp * w.gates));
+    LUMI_TRY(get(b.qkv, rp * (slices ? w.qkv : w.step_qkv)));
+    LUMI_TRY(get(b.gates, rp * (slices ? w.gates : w.step_gates)));
+    if (w.experts > 0) {
+        // (row, expert) pairs in blocks of rows, so that the sorted copies stay within bounds
+        MoeBufs& e = b.moe;
+        e.rows = (int)std::min<size_t>(rows, std::max<size_t>(128, (size_t)262144 / w.top));
+        const size_t pairs = ((size_t)e.rows * w.top + 127) / 128 * 128;
+        LUMI_TRY(get(e.logits, (size_t)e.rows * w.router));
+        LUMI_TRY(get(e.plan, moe_plan_ints(e.rows, w.top, w.experts)));
+        const size_t few = half ? std::min<size_t>(e.rows, 8) * w.top : pairs;
+        LUMI_TRY(get(e.h32, few * w.ffp));
+        if (half) {
+            LUMI_TRY(get(e.gh, pairs * ldx));
+            LUMI_TRY(get(e.gl, pairs * ldx));
+            LUMI_TRY(get(e.hh, pairs * w.ffp));
+            LUMI_TRY(get(e.hl, pairs * w.ffp));
+            LUMI_TRY(get(e.y, pairs * ldx));
+        }
     }
     b.rows = rows;
     return LUMI_OK;
@@ -535,7 +776,10 @@ static int32_t alloc_stacked(lumi_session* s) {
         LUMI_CUDA(cudaMalloc(&s->page_table, sizeof(int32_t) * pt.size()));
         LUMI_CUDA(cudaMemcpy(s->page_table, pt.data(), pt.size() * sizeof(int32_t), cudaMemcpyHostToDevice));
         size_t pw = 0;
-        for (const LayerSpec& L : c.specs) if (L.mixer.kind == MIXER_ATTENTION) pw = std::max(pw, window_attention_part_floats(L.mixer));
+        for (const LayerSpec& L : c.specs) {
+            if (L.mixer.kind == MIXER_ATTENTION) pw = std::max(pw, window_attention_part_floats(L.mixer));
+            if (L.mixer.kind == MIXER_LATENT) pw = std::max(pw, latent_part_floats(L.mixer));
+        }
         LUMI_CUDA(cudaMalloc(&s->attn_part, sizeof(float) * kAttnPartUnits * pw));
         LUMI_CUDA(cudaMalloc(&s->attn_part_count, sizeof(int32_t) * kAttnPartUnits));
         LUMI_CUDA(cudaMemset(s->attn_part_count, 0, sizeof(int32_t) * kAttnPartUnits));
@@ -552,6 +796,21 @@ static int32_t alloc_stacked(lumi_session* s) {
             LUMI_CUDA(cudaMalloc(&L.S, sizeof(float) * B * L.s_seq));
             LUMI_CUDA(cudaMalloc(&L.conv, sizeof(float) * B * L.conv_seq));
             LUMI_CUDA(cudaMemset(L.conv, 0, sizeof(float) * B * L.conv_seq));
+        } else if (m.kind == MIXER_RETENTION) {
+            L.dvp = (m.vdim + 3) / 4 * 4;
+            L.s_seq = (size_t)m.heads * m.dim * L.dvp;
+            LUMI_CUDA(cudaMalloc(&L.S, sizeof(float) * B * L.s_seq));
+        } else if (m.kind == MIXER_RGLRU) {
+            L.channels = m.channels;
+            L.s_seq = m.channels;
+            L.conv_seq = (size_t)m.taps * m.channels;
+            LUMI_CUDA(cudaMalloc(&L.S, sizeof(float) * B * L.s_seq));
+            LUMI_CUDA(cudaMalloc(&L.conv, sizeof(float) * B * L.conv_seq));
+            LUMI_CUDA(cudaMemset(L.conv, 0, sizeof(float) * B * L.conv_seq));
+        } else if (m.kind == MIXER_LATENT) {
+            L.kv_bytes = B * s->pages_per_seq * (size_t)kPageTokens * LatentShape(m).row * esz;
+            LUMI_CUDA(cudaMalloc(&L.kv, L.kv_bytes));
+            LUMI_CUDA(cudaMemset(L.kv, 0, L.kv_bytes));
         } else {
             L.dk_pad = (m.dim + 15) / 16 * 16; L.dv_pad = (m.vdim + 15) / 16 * 16;
             if (m.kv_from >= 0) continue;
@@ -586,6 +845,7 @@ extern "C" void lumi_session_free(lumi_session* s) {
     for (LayerState& L : s->lstate) { if (L.kv) cudaFree(L.kv); if (L.S) cudaFree(L.S); if (L.conv) cudaFree(L.conv); }
     if (s->pos_freq) cudaFree(s->pos_freq);
     if (s->want_idx) cudaFree(s->want_idx);
+    if (s->lat_kv) cudaFree(s->lat_kv);
     if (s->ctl_host) cudaFreeHost(s->ctl_host);
     if (s->pin_tokens) cudaFreeHost(s->pin_tokens);
     if (s->ev0) cudaEventDestroy(s->ev0);
@@ -661,6 +921,7 @@ static int32_t session_alloc(lumi_session* s) {
         LUMI_CUDA(cudaMemset(s->x, 0, sizeof(float) * (B + 127) / 128 * 128 * c.x_ld()));
         s->dec.x = s->x;
         LUMI_TRY(alloc_rows(s, s->dec, B, false));
+        LUMI_TRY(ensure_latent_rows(s, s->dec, B));
     }
     const size_t kmax = std::max<size_t>({(size_t)c.d_model, (size_t)c.d_inner(), na > 0 ? (size_t)c.mlp_dim() : 0});
     const size_t pmax = std::max<size_t>({nm > 0 ? (size_t)c.in_proj_out() : 0, na > 0 ? (size_t)(c.d_model + 2 * c.kv_dim()) : 0,
@@ -1017,6 +1278,10 @@ struct RowPass {
     // few rows on the weight-streaming path: b->mix still has to join the residual stream, under this norm weight; the next
     // product's prologue does it (x and x2 of the row buffers change places)
     const float* pending = nullptr;
+    // pre-norm layers, tensor-core path: the norm weights that b->xh / xl / ssq are current for (null = none), and how many partial
+    // sums of squares there are per row
+    const float* gamma_ready = nullptr;
+    int ssq_parts = 0;
     int rows() const { return nseq * ts; }
 };
 
@@ -1028,7 +1293,7 @@ EmbedPost embed_post_of(const lumi_session* s, const RowBufs& b, int slot0, bool
     e.freq = c.embed_positions ? s->pos_freq : nullptr;
     e.pos = s->kv_pos + slot0;
     e.width = c.d_model;
-    if (tc) { e.hi = b.xh; e.lo = s->opt_split ? b.xl : nullptr; }
+    if (tc && !c.specs[0].pre_norm) { e.hi = b.xh; e.lo = s->opt_split ? b.xl : nullptr; }
     return e;
 }
 
@@ -1081,7 +1346,7 @@ int32_t product_of_x(StepPlan& p, RowPass& r, const DevTensor& W, float* out32, 
     return LUMI_OK;
 }
 
-int32_t listed_layer(StepPlan& p, RowPass& r, const Layer& L) {
+int32_t post_norm_layer(StepPlan& p, RowPass& r, const Layer& L) {
     lumi_session* s = p.s;
     const Config& c = s->m->cfg;
     const MixerSpec& m = L.spec->mixer;
@@ -1138,7 +1403,7 @@ int32_t listed_layer(StepPlan& p, RowPass& r, const Layer& L) {
     p.fam = m.kind == MIXER_DELTA ? FAM_OUT_PROJ : FAM_ATTN;
     LUMI_TRY(product(p, rows, L.s.out, b.y32, b.ah, b.al, b.mix, ldx, 0));
     LUMI_TRY(add_normed(p, r, L.s.norm1));
-    if (L.spec->ff > 0) {
+    if (L.spec->ff.ff > 0) {
         p.fam = FAM_ATTN;
         LUMI_TRY(product_of_x(p, r, L.s.up, b.y32, (int)L.s.up.rows, 2, ah, b.al));
         LUMI_TRY(product(p, rows, L.s.down, b.y32, b.ah, b.al, b.mix, ldx, 0));
@@ -1146,6 +1411,322 @@ int32_t listed_layer(StepPlan& p, RowPass& r, const Layer& L) {
     }
     return LUMI_OK;
 }
+
+// ---- pre-norm layers ------------------------------------------------------------------------------------------
+// out = W norm(x) + bias: on the tensor cores with the norm folded around the product, else in the streaming kernel's prologue.
+// ext (tensor cores): gated results; act: Act of the streaming kernel, whose results are W.rows / 2 for gated kinds.
+int32_t norm_product(StepPlan& p, RowPass& r, const DevTensor& W, const float* gamma, const float* bias, float* out32, int ldd, int act = 0,
+                     __nv_bfloat16* out_hi = nullptr, __nv_bfloat16* out_lo = nullptr) {
+    lumi_session* s = p.s;
+    const Config& c = s->m->cfg;
+    RowBufs& b = *r.b;
+    const int N = (int)W.rows, K = (int)W.cols, rows = r.rows();
+    if (!p.tc) {
+        GemvArgs g{b.x, K, W.p, W.dtype, out32, ldd, nullptr, gamma, rows, act ? N / 2 : N, K, c.eps, act, &s->ctl->status};
+        g.norm_width = c.d_model;
+        g.bias = bias;
+        mark(p);
+        const cudaError_t e = launch_gemv(g, p.st_hi);
+        if (e == cudaErrorInvalidValue) return fail(LUMI_E_UNSUPPORTED, "a product over %d inputs is longer than the streaming kernel takes", K);
+        LUMI_CUDA(e);
+        return LUMI_OK;
+    }
+    if (r.gamma_ready != gamma) {
+        const int fam = p.fam;
+        p.fam = FAM_NORM;
+        mark(p);
+        LUMI_CUDA(launch_norm_split(b.x, gamma, b.xh, s->opt_split ? b.xl : nullptr, rows, K, c.eps, p.st_hi, b.ssq, b.ssq_stride));
+        p.fam = fam;
+        r.gamma_ready = gamma;
+        r.ssq_parts = 1;
+    }
+    GemmArgs g{b.xh, s->opt_split ? b.xl : nullptr, (const __nv_bfloat16*)W.p, out32, ldd, rows, N, K, 0, &s->ctl->status, s->gemm_counters, kGemmCounters,
+               s->gemm_scratch, kGemmScratchFloats};
+    g.nf.ssq_in = b.ssq; g.nf.ssq_parts = r.ssq_parts; g.nf.ssq_stride = b.ssq_stride;
+    g.nf.inv_k = (float)(1.0 / (double)c.d_model); g.nf.eps = c.eps;
+    g.nf.bias = bias;
+    GemmExt ex;
+    if (act != 0) {
+        ex.group_rows = N; ex.lda = K; ex.out_n = ex.out_step = N / 2; ex.gate = act; ex.ldo = N / 2;
+        g.nf.out_hi = out_hi;
+        g.nf.out_lo = s->opt_split ? out_lo : nullptr;
+        g.ext = &ex;
+    }
+    mark(p);
+    return launch_gemm_tcgen05(g, p.st_hi);
+}
+
+// x += W a + bias; on the tensor cores the next norm's input is renewed in the epilogue.
+int32_t residual_product(StepPlan& p, RowPass& r, const DevTensor& W, const float* bias, const float* gamma_next) {
+    lumi_session* s = p.s;
+    RowBufs& b = *r.b;
+    const int N = (int)W.rows, K = (int)W.cols, ldx = s->m->cfg.x_ld();
+    mark(p);
+    if (!p.tc) {
+        GemvArgs g{b.y32, K, W.p, W.dtype, b.x, ldx, b.x, nullptr, r.rows(), N, K, s->m->cfg.eps, 0, &s->ctl->status};
+        g.bias = bias;
+        const cudaError_t e = launch_gemv(g, p.st_hi);
+        if (e == cudaErrorInvalidValue) return fail(LUMI_E_UNSUPPORTED, "a product over %d inputs is longer than the streaming kernel takes", K);
+        LUMI_CUDA(e);
+        return LUMI_OK;
+    }
+    GemmArgs g{b.ah, s->opt_split ? b.al : nullptr, (const __nv_bfloat16*)W.p, b.x, ldx, r.rows(), N, K, 1, &s->ctl->status, s->gemm_counters, kGemmCounters,
+               s->gemm_scratch, kGemmScratchFloats};
+    g.nf.bias = bias;
+    g.nf.gamma_next = gamma_next; g.nf.out_hi = b.xh; g.nf.out_lo = s->opt_split ? b.xl : nullptr;
+    g.nf.ssq_out = b.ssq; g.nf.ssq_stride = b.ssq_stride;
+    LUMI_TRY(launch_gemm_tcgen05(g, p.st_hi));
+    r.gamma_ready = gamma_next;
+    r.ssq_parts = (N + 31) / 32;
+    return LUMI_OK;
+}
+
+// Products of a pass's rows by groups of weight rows (blocks, heads): tensor cores from halves, or the few-rows kernel from fp32.
+struct GroupedProduct {
+    const DevTensor* W;
+    int groups, group_rows, K, n_out, out_step;           // K: true inputs per group (rows of W are padded)
+    const float* a32; int lda32, a_step;                  // fp32 rows
+    const __nv_bfloat16 *ah, *al;                         // halves, [rows][groups * W->cols]
+    const float* bias; const float* mul; int ldmul;
+    float* out32; int ld32; __nv_bfloat16 *oh, *ol; int ldo;
+};
+int32_t grouped_product(StepPlan& p, int rows, const GroupedProduct& q) {
+    lumi_session* s = p.s;
+    mark(p);
+    if (!p.tc) {
+        const BlockProductArgs a{q.a32, q.lda32, q.a_step, q.W->p, q.W->dtype, (int)q.W->cols, q.group_rows, q.bias, q.mul, q.ldmul, q.out32, q.ld32, q.out_step,
+                                 rows, q.groups, q.n_out, q.K};
+        LUMI_CUDA(launch_block_product(a, p.st_hi));
+        return LUMI_OK;
+    }
+    GemmExt ex;
+    ex.groups = q.groups; ex.group_rows = q.group_rows; ex.lda = q.groups * (int)q.W->cols; ex.out_step = q.out_step; ex.out_n = q.n_out;
+    ex.mul = q.mul; ex.ldmul = q.ldmul; ex.ldo = q.ldo;
+    GemmArgs g{q.ah, s->opt_split ? q.al : nullptr, (const __nv_bfloat16*)q.W->p, q.oh != nullptr ? nullptr : q.out32, q.ld32, rows, q.groups * q.group_rows,
+               (int)q.W->cols, 0, &s->ctl->status};
+    g.nf.bias = q.bias;
+    g.nf.out_hi = q.oh;
+    g.nf.out_lo = s->opt_split ? q.ol : nullptr;
+    g.ext = &ex;
+    return launch_gemm_tcgen05(g, p.st_hi);
+}
+
+int32_t retention_mixer(StepPlan& p, RowPass& r, const Layer& L, int li) {
+    lumi_session* s = p.s;
+    const MixerSpec& m = L.spec->mixer;
+    RowBufs& b = *r.b;
+    const LayerState& S = s->lstate[li];
+    RetentionArgs a{};
+    a.proj = b.proj; a.ldp = (int)L.s.in.rows;
+    a.off_q = L.s.off_q; a.off_k = L.s.off_k; a.off_v = L.s.off_v; a.off_g = L.s.off_g;
+    a.S = S.S; a.H = m.heads; a.dk = m.dim; a.dv = m.vdim; a.dvp = S.dvp;
+    a.rot = m.rot; a.freq = L.s.rot_freq; a.decay_pow = L.s.decay_pow;
+    a.k_scale = (float)(1.0 / std::sqrt((double)m.dim)); a.eps = s->m->cfg.eps;
+    a.pos = s->kv_pos; a.row_len = r.row_len; a.t_abs0 = r.t_abs0; a.ctl = s->ctl;
+    a.nseq = r.nseq; a.ts = r.ts; a.b0 = r.b0;
+    a.y32 = p.tc ? nullptr : b.y32; a.yhi = p.tc ? b.ah : nullptr; a.ylo = p.tc && s->opt_split ? b.al : nullptr; a.ldy = (int)L.s.out.cols;
+    a.o32 = b.mix;
+    p.fam = FAM_SSM;
+    mark(p);
+    int n = 0;
+    // short slices and fp32 models go token by token (the chunked form's products are tf32 terms)
+    const bool chunked = r.ts >= 16 && s->m->wdtype == LUMI_DTYPE_BF16 && retention_chunk_supported(m.dim, m.vdim);
+    const cudaError_t e = chunked ? launch_retention_chunk(a, p.st_lo, &n) : launch_retention_step(a, p.st_lo, &n);
+    if (e == cudaErrorInvalidValue) return fail(LUMI_E_UNSUPPORTED, "retention heads of %d x %d are not built", m.dim, m.vdim);
+    LUMI_CUDA(e);
+    p.n += n - 1;
+    return LUMI_OK;
+}
+
+int32_t rglru_mixer(StepPlan& p, RowPass& r, const Layer& L, int li) {
+    lumi_session* s = p.s;
+    const MixerSpec& m = L.spec->mixer;
+    RowBufs& b = *r.b;
+    const LayerState& S = s->lstate[li];
+    const int bs = m.channels / m.blocks, bp = (int)L.s.rg.cols;
+    RglruArgs a{};
+    a.proj = b.proj; a.ldp = (int)L.s.in.rows; a.off_x = L.s.off_x; a.off_y = L.s.off_y;
+    a.conv_w = L.s.conv_q; a.conv_b = L.s.conv_b; a.lam = L.s.lam;
+    a.rg = L.s.rg.p; a.rg_dtype = L.s.rg.dtype; a.rg_b = L.s.rg_b;
+    a.channels = m.channels; a.blocks = m.blocks; a.bp = bp; a.taps = m.taps; a.rate = m.decay_rate;
+    a.S = S.S; a.conv = S.conv;
+    a.pos = s->kv_pos; a.row_len = r.row_len; a.t_abs0 = r.t_abs0; a.ctl = s->ctl;
+    a.nseq = r.nseq; a.ts = r.ts; a.b0 = r.b0;
+    a.u32 = b.qkv; a.gates = b.gates;
+    a.y32 = p.tc ? nullptr : b.y32; a.yhi = p.tc ? b.ah : nullptr; a.ylo = p.tc && s->opt_split ? b.al : nullptr; a.ldy = (int)L.s.out.cols;
+    p.fam = FAM_SSM;
+    if (r.ts == 1 && r.rows() <= kRglruStepRows && rglru_step_supported(a)) {
+        mark(p);
+        LUMI_CUDA(launch_rglru_step(a, p.st_lo));
+        return LUMI_OK;
+    }
+    if (p.tc) { a.uh = b.bh; a.ul = s->opt_split ? b.bl : nullptr; }
+    mark(p);
+    LUMI_CUDA(launch_rglru_conv(a, p.st_lo));
+    const GroupedProduct q{&L.s.rg, m.blocks, 2 * bp, bs, 2 * bp, 2 * bp, b.qkv, m.channels, bs, b.bh, b.bl, L.s.rg_b, nullptr, 0, b.gates, m.blocks * 2 * bp,
+                           nullptr, nullptr, 0};
+    LUMI_TRY(grouped_product(p, r.rows(), q));
+    mark(p);
+    LUMI_CUDA(launch_rglru_scan(a, p.st_lo));
+    if (m.taps > 1) {
+        mark(p);
+        LUMI_CUDA(launch_rglru_tail(a, p.st_lo));
+    }
+    return LUMI_OK;
+}
+
+// Slices of at least this many tokens expand keys and values per head (bf16 caches).
+constexpr int kLatentExpandMin = 16;
+constexpr size_t kLatentExpandBytes = (size_t)2 << 30;    // of expanded keys and values at a time
+// Sequences whose rings are expanded together.
+int latent_expand_seqs(const lumi_session* s, const MixerSpec& m, int nseq) {
+    const LatentShape ls(m);
+    const size_t per = (size_t)s->pages_per_seq * kPageTokens * m.heads * (ls.dk_pad + ls.dv_pad) * sizeof(__nv_bfloat16);
+    return (int)std::min<size_t>(nseq, std::max<size_t>(1, kLatentExpandBytes / per));
+}
+
+int32_t latent_mixer(StepPlan& p, RowPass& r, const Layer& L, int li) {
+    lumi_session* s = p.s;
+    const MixerSpec& m = L.spec->mixer;
+    const LatentShape ls(m);
+    RowBufs& b = *r.b;
+    const int rows = r.rows(), ldp = (int)L.s.in.rows;
+    const bool expand = r.ts >= kLatentExpandMin && p.tc && L.s.ukv.p != nullptr && ls.dk_pad <= 256 && ls.dv_pad <= 256;
+    LatentArgs a{};
+    a.proj = b.proj; a.ldp = ldp; a.off_q = L.s.off_q; a.off_c = L.s.off_c;
+    a.kv = s->lstate[li].kv; a.kv_is_f32 = s->m->wdtype == LUMI_DTYPE_BF16 ? 0 : 1;
+    a.page_table = s->page_table; a.pages_per_seq = s->pages_per_seq; a.pos = s->kv_pos;
+    a.m = m; a.freq = L.s.rot_freq; a.c_norm = L.s.c_norm; a.eps = s->m->cfg.eps;
+    a.row_len = r.row_len; a.t_abs0 = r.t_abs0; a.ctl = s->ctl;
+    a.nseq = r.nseq; a.ts = r.ts; a.b0 = r.b0; a.limit = s->kv_limit;
+    if (!expand) {
+        if ((size_t)rows > b.lat_rows) return fail(LUMI_E_INVALID, "%d rows of latent attention, buffers for %zu", rows, b.lat_rows);
+        a.qlat = b.qlat;
+        if (p.tc) { a.qh = b.lh; a.ql = s->opt_split ? b.ll : nullptr; a.ch = b.lh; a.cl = s->opt_split ? b.ll : nullptr; }
+        else a.ctx = b.ctx;
+        a.part = s->attn_part; a.part_count = s->attn_part_count;
+    }
+    mark(p);
+    LUMI_CUDA(launch_latent_prep(a, p.st_hi));
+    if (!expand) {
+        const GroupedProduct uk{&L.s.uk, m.heads, ls.lp, m.dim, ls.lp, ls.row, b.proj + L.s.off_q, ldp, ls.dk, b.lh, b.ll, nullptr, nullptr, 0, b.qlat, m.heads * ls.row,
+                                nullptr, nullptr, 0};
+        LUMI_TRY(grouped_product(p, rows, uk));
+        mark(p);
+        LUMI_CUDA(launch_latent_attention(a, p.st_hi));
+        const GroupedProduct uv{&L.s.uv, m.heads, (int)(L.s.uv.rows / m.heads), m.kv_rank, m.vdim, m.vdim, b.ctx, m.heads * ls.lp, ls.lp, b.lh, b.ll, nullptr,
+                                b.proj + L.s.off_g, ldp, b.y32, (int)L.s.out.cols, p.tc ? b.ah : nullptr, p.tc ? b.al : nullptr, (int)L.s.out.cols};
+        return grouped_product(p, rows, uv);
+    }
+    // keys and values per head for a few sequences' rings at a time, then attention over them (pages of a slot lie together)
+    const int ring = s->pages_per_seq * kPageTokens, hw = ls.dk_pad + ls.dv_pad, ld = m.heads * hw, chunk = latent_expand_seqs(s, m, r.nseq);
+    for (int q0 = 0; q0 < r.nseq; q0 += chunk) {
+        const int nq = std::min(chunk, r.nseq - q0);
+        GemmArgs g{(const __nv_bfloat16*)a.kv + (size_t)(r.b0 + q0) * ring * ls.row, nullptr, (const __nv_bfloat16*)L.s.ukv.p, nullptr, ld, nq * ring, ld, ls.row, 0,
+                   &s->ctl->status};
+        g.nf.out_hi = s->lat_kv;
+        mark(p);
+        LUMI_TRY(launch_gemm_tcgen05(g, p.st_hi));
+        WinAttnArgs w{};
+        w.proj = b.proj + (size_t)q0 * r.ts * ldp; w.ldp = ldp; w.off_q = L.s.off_q;
+        w.kv = (void*)((uintptr_t)s->lat_kv - (uintptr_t)(r.b0 + q0) * ring * ld * sizeof(__nv_bfloat16));      // page numbers count from slot 0
+        w.kv_is_f32 = 0; w.dk_pad = ls.dk_pad; w.dv_pad = ls.dv_pad;
+        w.page_table = s->page_table; w.pages_per_seq = s->pages_per_seq; w.pos = s->kv_pos;
+        w.H = m.heads; w.G = m.heads; w.dk = ls.dk; w.dv = m.vdim;
+        w.m = m; w.m.kv_heads = m.heads; w.m.dim = ls.dk;
+        w.append = 0; w.eps = a.eps;
+        w.row_len = r.row_len; w.t_abs0 = r.t_abs0; w.ctl = s->ctl;
+        w.nseq = nq; w.ts = r.ts; w.b0 = r.b0 + q0; w.limit = s->kv_limit;
+        const size_t yo = (size_t)q0 * r.ts * L.s.out.cols;
+        w.yhi = b.ah + yo; w.ylo = s->opt_split ? b.al + yo : nullptr; w.ldy = (int)L.s.out.cols;
+        w.page_elems = (long)kPageTokens * ld; w.head_step = hw; w.k_ld = w.v_ld = ld; w.v_off = ls.dk_pad;
+        w.gate = b.proj + (size_t)q0 * r.ts * ldp + L.s.off_g; w.ldg = ldp;
+        int n = 0;
+        mark(p);
+        const cudaError_t e = launch_window_attention(w, p.st_hi, &n);
+        if (e == cudaErrorInvalidValue) return fail(LUMI_E_UNSUPPORTED, "attention heads of %d / %d elements are not built", ls.dk, m.vdim);
+        LUMI_CUDA(e);
+    }
+    return LUMI_OK;
+}
+
+// x += experts(norm(x)), a block of rows at a time.
+int32_t experts_ff(StepPlan& p, RowPass& r, const Layer& L, const float* gamma_next) {
+    lumi_session* s = p.s;
+    const Config& c = s->m->cfg;
+    const FfSpec& f = L.spec->ff;
+    RowBufs& b = *r.b;
+    MoeBufs& e = b.moe;
+    const int ldx = c.x_ld(), ffp = (int)L.s.down.cols, E_max = row_widths(s->m).experts, rows = r.rows();
+    for (int r0 = 0; r0 < rows; r0 += e.rows) {
+        RowBufs part = b;                                 // the block's rows
+        part.x = b.x + (size_t)r0 * ldx;
+        if (p.tc) { part.xh = b.xh + (size_t)r0 * ldx; part.xl = b.xl + (size_t)r0 * ldx; part.ssq = b.ssq + (size_t)r0 * b.ssq_stride; }
+        RowPass rp{&part, std::min(e.rows, rows - r0), 1, 0, nullptr, -1};
+        rp.gamma_ready = r.gamma_ready;
+        rp.ssq_parts = r.ssq_parts;
+        LUMI_TRY(norm_product(p, rp, L.s.router, L.s.norm2, nullptr, e.logits, (int)L.s.router.rows));
+        MoeArgs a{};
+        a.logits = e.logits; a.ldl = (int)L.s.router.rows;
+        a.rows = rp.rows(); a.E = f.experts; a.E_max = E_max; a.top = f.top; a.D = c.d_model; a.ldx = ldx; a.ff = f.ff; a.ffp = ffp;
+        a.x = part.x; a.gamma = L.s.norm2; a.eps = c.eps;
+        a.plan = e.plan;
+        if (!p.tc) {
+            a.h32 = e.h32; a.w_up = L.s.up.p; a.w_down = L.s.down.p; a.w_dtype = L.s.up.dtype; a.act = f.act;
+            mark(p);
+            mark(p);
+            LUMI_CUDA(launch_moe_few(a, p.st_hi));
+            continue;
+        }
+        a.gh = e.gh; a.gl = s->opt_split ? e.gl : nullptr; a.y = e.y;
+        a.gamma_next = gamma_next; a.xh = part.xh; a.xl = s->opt_split ? part.xl : nullptr; a.ssq = part.ssq; a.ssq_stride = b.ssq_stride;
+        mark(p);
+        LUMI_CUDA(launch_moe_route(a, p.st_hi));
+        mark(p);
+        LUMI_CUDA(launch_moe_gather(a, p.st_hi));
+        const int pairs = a.rows * f.top;
+        GemmExt ex;
+        ex.groups = f.experts; ex.group_rows = 2 * ffp; ex.lda = ldx; ex.out_step = 0; ex.out_n = ffp; ex.gate = f.act; ex.ldo = ffp;
+        ex.tiles = moe_tiles(a); ex.n_tiles = e.plan; ex.max_tiles = moe_max_tiles(a.rows, f.top, f.experts);
+        GemmArgs g{e.gh, a.gl, (const __nv_bfloat16*)L.s.up.p, nullptr, 0, pairs, f.experts * 2 * ffp, ldx, 0, &s->ctl->status};
+        g.nf.out_hi = e.hh; g.nf.out_lo = s->opt_split ? e.hl : nullptr;
+        g.ext = &ex;
+        mark(p);
+        LUMI_TRY(launch_gemm_tcgen05(g, p.st_hi));
+        ex.group_rows = ldx; ex.lda = ffp; ex.out_n = ldx; ex.gate = 0; ex.ldo = 0;
+        GemmArgs d{e.hh, s->opt_split ? e.hl : nullptr, (const __nv_bfloat16*)L.s.down.p, e.y, ldx, pairs, f.experts * ldx, ffp, 0, &s->ctl->status};
+        d.ext = &ex;
+        mark(p);
+        LUMI_TRY(launch_gemm_tcgen05(d, p.st_hi));
+        mark(p);
+        LUMI_CUDA(launch_moe_combine(a, p.st_hi));
+    }
+    if (p.tc) { r.gamma_ready = gamma_next; r.ssq_parts = 1; }
+    return LUMI_OK;
+}
+
+int32_t pre_norm_layer(StepPlan& p, RowPass& r, const Layer& L) {
+    lumi_session* s = p.s;
+    const MixerSpec& m = L.spec->mixer;
+    const FfSpec& f = L.spec->ff;
+    RowBufs& b = *r.b;
+    const int li = (int)(&L - s->m->layers.data());
+    const float* after = li + 1 < (int)s->m->layers.size() ? s->m->layers[li + 1].s.norm1 : s->m->final_norm_g;      // the norm behind this layer
+    p.fam = m.recurrent() ? FAM_IN_PROJ : FAM_ATTN;
+    LUMI_TRY(norm_product(p, r, L.s.in, L.s.norm1, L.s.in_b, b.proj, (int)L.s.in.rows));
+    if (m.kind == MIXER_RETENTION) LUMI_TRY(retention_mixer(p, r, L, li));
+    else if (m.kind == MIXER_RGLRU) LUMI_TRY(rglru_mixer(p, r, L, li));
+    else LUMI_TRY(latent_mixer(p, r, L, li));
+    p.fam = m.recurrent() ? FAM_OUT_PROJ : FAM_ATTN;
+    LUMI_TRY(residual_product(p, r, L.s.out, nullptr, f.ff > 0 ? L.s.norm2 : after));
+    if (f.ff == 0) return LUMI_OK;
+    p.fam = FAM_ATTN;
+    if (f.experts > 0) return experts_ff(p, r, L, after);
+    LUMI_TRY(norm_product(p, r, L.s.up, L.s.norm2, L.s.up_b, b.y32, (int)L.s.down.cols, f.act, b.ah, b.al));
+    return residual_product(p, r, L.s.down, L.s.down_b, after);
+}
+
+int32_t listed_layer(StepPlan& p, RowPass& r, const Layer& L) { return L.spec->pre_norm ? pre_norm_layer(p, r, L) : post_norm_layer(p, r, L); }
 
 // What is still pending joins the residual stream in a kernel of its own; the stream ends up in `x`, one of the two buffers.
 int32_t settle(StepPlan& p, RowPass& r, float* x) {
@@ -1155,7 +1736,7 @@ int32_t settle(StepPlan& p, RowPass& r, float* x) {
     return LUMI_OK;
 }
 
-// Final norm and tied head over `rows` rows of b.x (row_idx, device, picks them; null = the first `rows`).
+// Final norm and head over `rows` rows of b.x (row_idx, device, picks them; null = the first `rows`).
 int32_t listed_head(StepPlan& p, RowBufs& b, const int32_t* row_idx, int rows, float* out) {
     lumi_session* s = p.s;
     const Config& c = s->m->cfg;
@@ -1164,7 +1745,7 @@ int32_t listed_head(StepPlan& p, RowBufs& b, const int32_t* row_idx, int rows, f
                   c.d_model, c.x_ld(), c.eps, nullptr};
     p.fam = FAM_HEAD;
     if (!tc && row_idx == nullptr && c.d_model == c.x_ld()) {           // the norm rides in the product's prologue
-        GemvArgs g{b.x, c.d_model, s->m->embedding.p, s->m->embedding.dtype, out, c.vocab, nullptr, s->m->final_norm_g, rows, c.vocab, c.d_model,
+        GemvArgs g{b.x, c.d_model, s->m->head.p, s->m->head.dtype, out, c.vocab, nullptr, s->m->final_norm_g, rows, c.vocab, c.d_model,
                    c.eps, 0, &s->ctl->status};
         mark(p);
         LUMI_CUDA(launch_gemv(g, p.st_hi));
@@ -1174,7 +1755,7 @@ int32_t listed_head(StepPlan& p, RowBufs& b, const int32_t* row_idx, int rows, f
     LUMI_CUDA(launch_row_norm(a, p.st_hi));
     const bool keep = p.tc;
     p.tc = tc;
-    const int32_t rc = product(p, rows, s->m->embedding, b.y32, b.xh, b.xl, out, c.vocab, 0);
+    const int32_t rc = product(p, rows, s->m->head, b.y32, b.xh, b.xl, out, c.vocab, 0);
     p.tc = keep;
     return rc;
 }
@@ -1273,7 +1854,8 @@ int32_t enqueue_step(lumi_session* s, int B, bool with_head, int64_t* launches,
     if (fused) {
         p.fam = FAM_HEAD;
         int nparts = 0;
-        GemvArgs g{s->x, c.x_ld(), s->m->embedding.p, s->m->embedding.dtype, nullptr, c.vocab, nullptr, s->m->final_norm_g, B, c.vocab,
+        const DevTensor& head = c.stacked() ? s->m->head : s->m->embedding;
+        GemvArgs g{s->x, c.x_ld(), head.p, head.dtype, nullptr, c.vocab, nullptr, s->m->final_norm_g, B, c.vocab,
                    c.x_ld(), c.eps, 0, &s->ctl->status};
         if (c.x_ld() != c.d_model) {                      // padded rows: the mean runs over the true width, in a kernel of its own
             RowNormArgs rn{s->x, nullptr, s->m->final_norm_g, s->dec.y32, nullptr, nullptr, nullptr, B, c.d_model, c.x_ld(), c.eps, nullptr};
@@ -1485,6 +2067,19 @@ int32_t prefill_listed(lumi_session* s, int batch, int T, bool with_head, float*
         LUMI_TRY(alloc_rows(s, s->pre, rows_max, true));
     }
     RowBufs& b = s->pre;
+    // latent attention: slices that do not expand keys and values need queries in the latent space; the others the expanded rows
+    const bool half = s->m->wdtype == LUMI_DTYPE_BF16;
+    const int last_ts = T % TS == 0 ? TS : T % TS;
+    LUMI_TRY(ensure_latent_rows(s, b, !half ? rows_max : std::min(TS, last_ts) < kLatentExpandMin || s->opt_gemm == 1 ? (size_t)nb_max * std::min(TS, kLatentExpandMin) : 0));
+    for (const LayerSpec& L : c.specs) {
+        if (L.mixer.kind != MIXER_LATENT || !half || TS < kLatentExpandMin) continue;
+        const LatentShape ls(L.mixer);
+        const size_t need = (size_t)latent_expand_seqs(s, L.mixer, nb_max) * s->pages_per_seq * kPageTokens * L.mixer.heads * (ls.dk_pad + ls.dv_pad);
+        if (need > s->lat_kv_cap) {
+            LUMI_CUDA(cudaStreamSynchronize(s->stream));
+            LUMI_TRY(grow(s->lat_kv, s->lat_kv_cap, need));
+        }
+    }
     if (want != nullptr && want->size() > s->want_cap) LUMI_TRY(grow(s->want_idx, s->want_cap, want->size()));
     size_t wanted = 0;
     std::vector<int32_t> local;                           // outlives the copies below (synchronised before it changes)
@@ -2006,7 +2601,8 @@ extern "C" int32_t lumi_generate(lumi_session* s, const uint32_t* prompts, int32
             const LayerState& L = s->lstate[i];
             const MixerSpec& m = cf.specs[i].mixer;
             const int64_t esz = s->m->wdtype == LUMI_DTYPE_BF16 ? 2 : 4;
-            if (m.kind == MIXER_DELTA) listed += 2 * 4 * (int64_t)L.s_seq + 4 * (int64_t)L.conv_seq;
+            if (m.recurrent()) listed += 2 * 4 * (int64_t)L.s_seq + 4 * (int64_t)L.conv_seq;
+            else if (m.kind == MIXER_LATENT) listed += esz * LatentShape(m).row * (int64_t)std::min(m.window > 0 ? m.window : T + n_new / 2, T + n_new / 2);
             else listed += esz * m.kv_heads * (L.dk_pad + L.dv_pad) * (int64_t)std::min(m.window > 0 ? m.window : T + n_new / 2, T + n_new / 2);
         }
         stats->bytes_per_step = s->m->weight_bytes + (int64_t)batch * (per_seq + listed);
@@ -2139,7 +2735,7 @@ static int32_t snap_copy(lumi_session* s, int32_t slot, char* buf, bool save) {
     for (const LayerState& S : s->lstate) {
         if (S.S != nullptr) {
             LUMI_CUDA(xfer(S.S + slot * S.s_seq, S.s_seq * sizeof(float)));
-            LUMI_CUDA(xfer(S.conv + slot * S.conv_seq, S.conv_seq * sizeof(float)));
+            if (S.conv_seq > 0) LUMI_CUDA(xfer(S.conv + slot * S.conv_seq, S.conv_seq * sizeof(float)));
         }
         if (S.kv != nullptr) LUMI_CUDA(xfer((char*)S.kv + (size_t)slot * (S.kv_bytes / B), S.kv_bytes / B));
     }
@@ -2153,7 +2749,7 @@ extern "C" int32_t lumi_session_save_state(lumi_session* s, int32_t slot, void* 
     if (nbytes < (int64_t)(sizeof(SnapHeader) + L.payload))
         return fail(LUMI_E_INVALID, "snapshot buffer of %lld bytes, %zu needed", (long long)nbytes, sizeof(SnapHeader) + L.payload);
     LUMI_CUDA(cudaSetDevice(s->m->device));
-    SnapHeader hd{kSnapMagic, 1u, (uint32_t)(s->m->n_mamba + s->m->n_delta), (uint32_t)(s->m->n_attn + s->m->n_wattn), (uint64_t)L.payload, 0, 0u};
+    SnapHeader hd{kSnapMagic, 1u, (uint32_t)(s->m->n_mamba + s->m->n_recur), (uint32_t)(s->m->n_attn + s->m->n_wattn), (uint64_t)L.payload, 0, 0u};
     LUMI_CUDA(cudaMemcpyAsync(&hd.kv_pos, s->kv_pos + slot, sizeof(int32_t), cudaMemcpyDeviceToHost, s->stream));
     LUMI_TRY(snap_copy(s, slot, (char*)host_buf + sizeof(SnapHeader), true));
     LUMI_CUDA(cudaStreamSynchronize(s->stream));
@@ -2169,9 +2765,9 @@ extern "C" int32_t lumi_session_load_state(lumi_session* s, int32_t slot, const 
     if (nbytes < (int64_t)sizeof(hd)) return fail(LUMI_E_INVALID, "snapshot shorter than its header");
     memcpy(&hd, host_buf, sizeof(hd));
     if (hd.magic != kSnapMagic || hd.version != 1u) return fail(LUMI_E_INVALID, "not a sequence snapshot");
-    if (hd.n_mamba != (uint32_t)(s->m->n_mamba + s->m->n_delta) || hd.n_attn != (uint32_t)(s->m->n_attn + s->m->n_wattn) || hd.payload_bytes != (uint64_t)L.payload)
+    if (hd.n_mamba != (uint32_t)(s->m->n_mamba + s->m->n_recur) || hd.n_attn != (uint32_t)(s->m->n_attn + s->m->n_wattn) || hd.payload_bytes != (uint64_t)L.payload)
         return fail(LUMI_E_TENSOR, "snapshot of another model or cache size (%u Mamba + %u attention layers, %llu bytes; this session: %d + %d, %zu)",
-                    hd.n_mamba, hd.n_attn, (unsigned long long)hd.payload_bytes, s->m->n_mamba + s->m->n_delta, s->m->n_attn + s->m->n_wattn, L.payload);
+                    hd.n_mamba, hd.n_attn, (unsigned long long)hd.payload_bytes, s->m->n_mamba + s->m->n_recur, s->m->n_attn + s->m->n_wattn, L.payload);
     if (nbytes < (int64_t)(sizeof(hd) + L.payload)) return fail(LUMI_E_INVALID, "snapshot truncated");
     // the position indexes the page table and the cache: a value outside what this session can hold is refused here
     // (with a sliding window on every attention layer positions may run past the capacity: the ring wraps)

@@ -17,13 +17,12 @@
 // Raw convolution inputs live in a ring over positions (slot = position % taps): a step writes the slot of its own position
 // and reads the others, so the CTAs of one launch never touch a slot that another one writes.
 #include "rows.cuh"
+#include "tf32.cuh"
 
 #include <cmath>
 
 namespace lumi {
 namespace {
-
-__device__ __forceinline__ float softplus_f(float x) { return x > 20.f ? x : log1pf(expf(x)); }
 
 // Convolution output (before silu) of one channel at token t of the pass: inputs of this pass from the projection rows,
 // earlier ones from the ring, none before position 0.
@@ -415,98 +414,6 @@ __global__ void __launch_bounds__(256) delta_prep_rows_kernel(DeltaArgs a, int d
     }
 }
 
-// One warp per (row, head): RMS norm of the read-out, weight, gate.
-__global__ void __launch_bounds__(256) delta_out_kernel(DeltaArgs a) {
-    const long w = ((long)blockIdx.x * 256 + threadIdx.x) >> 5;
-    const int lane = threadIdx.x & 31;
-    if (w >= (long)a.nseq * a.ts * a.H) return;
-    const int row = (int)(w / a.H), h = (int)(w % a.H), sl = row / a.ts, t = row % a.ts;
-    const bool live = t < pass_tokens(a.row_len, a.ctl, a.b0 + sl, a.ts, a.t_abs0);
-    const float* o = a.o32 + ((size_t)row * a.H + h) * a.dvp;
-    const float* gate = a.proj + (size_t)row * a.ldp + a.off_g + h * a.dv;
-    const size_t oo = (size_t)row * a.ldy + h * a.dv;
-    if ((a.dv & 3) == 0 && a.dv <= 512 && ((a.ldp | a.off_g | a.ldy) & 3) == 0) {      // four neighbouring elements per lane
-        float4 v[4];
-        float s = 0.f;
-#pragma unroll
-        for (int i = 0; i < 4; ++i) {
-            const int c = 4 * (lane + 32 * i);
-            v[i] = live && c < a.dv ? *reinterpret_cast<const float4*>(o + c) : make_float4(0.f, 0.f, 0.f, 0.f);
-            s = fmaf(v[i].x, v[i].x, fmaf(v[i].y, v[i].y, fmaf(v[i].z, v[i].z, fmaf(v[i].w, v[i].w, s))));
-        }
-        const float rs = __frcp_rn(__fsqrt_rn(__fdiv_rn(warp_total(s), (float)a.dv) + a.eps));
-#pragma unroll
-        for (int i = 0; i < 4; ++i) {
-            const int c = 4 * (lane + 32 * i);
-            if (c >= a.dv) break;
-            float y[4] = {0.f, 0.f, 0.f, 0.f};
-            if (live) {
-                const float4 gt = *reinterpret_cast<const float4*>(gate + c);
-                const float ov[4] = {v[i].x, v[i].y, v[i].z, v[i].w}, gv[4] = {gt.x, gt.y, gt.z, gt.w};
-#pragma unroll
-                for (int e = 0; e < 4; ++e) y[e] = ov[e] * rs * a.o_norm[c + e] * __fdividef(gv[e], 1.0f + __expf(-gv[e]));
-            }
-            if (a.y32 != nullptr) *reinterpret_cast<float4*>(a.y32 + oo + c) = make_float4(y[0], y[1], y[2], y[3]);
-            if (a.yhi != nullptr) {
-                const __nv_bfloat162 h0 = __floats2bfloat162_rn(y[0], y[1]), h1 = __floats2bfloat162_rn(y[2], y[3]);
-                uint2 u;
-                u.x = *reinterpret_cast<const uint32_t*>(&h0); u.y = *reinterpret_cast<const uint32_t*>(&h1);
-                *reinterpret_cast<uint2*>(a.yhi + oo + c) = u;
-                if (a.ylo != nullptr) {
-                    const float2 f0 = __bfloat1622float2(h0), f1 = __bfloat1622float2(h1);
-                    const __nv_bfloat162 l0 = __floats2bfloat162_rn(y[0] - f0.x, y[1] - f0.y), l1 = __floats2bfloat162_rn(y[2] - f1.x, y[3] - f1.y);
-                    u.x = *reinterpret_cast<const uint32_t*>(&l0); u.y = *reinterpret_cast<const uint32_t*>(&l1);
-                    *reinterpret_cast<uint2*>(a.ylo + oo + c) = u;
-                }
-            }
-        }
-        return;
-    }
-    float s = 0.f;
-    if (live) for (int c = lane; c < a.dv; c += 32) s = fmaf(o[c], o[c], s);
-    s = warp_total(s);
-    const float rs = __frcp_rn(__fsqrt_rn(__fdiv_rn(s, (float)a.dv) + a.eps));
-    for (int c = lane; c < a.dv; c += 32)
-        put_row(a.y32, a.yhi, a.ylo, oo + c, live ? o[c] * rs * a.o_norm[c] * silu_f(gate[c]) : 0.f);
-}
-
-struct Tf2 { uint32_t hi, lo; };
-__device__ __forceinline__ Tf2 split_tf32(float x) {
-    Tf2 r;
-    asm("cvt.rna.tf32.f32 %0, %1;" : "=r"(r.hi) : "f"(x));
-    r.lo = __float_as_uint(x - __uint_as_float(r.hi));
-    return r;
-}
-__device__ __forceinline__ void mma_tf32(float (&d)[4], uint32_t a0, uint32_t a1, uint32_t a2, uint32_t a3, uint32_t b0, uint32_t b1) {
-    asm("mma.sync.aligned.m16n8k8.row.col.f32.tf32.tf32.f32 {%0, %1, %2, %3}, {%4, %5, %6, %7}, {%8, %9}, {%0, %1, %2, %3};"
-        : "+f"(d[0]), "+f"(d[1]), "+f"(d[2]), "+f"(d[3]) : "r"(a0), "r"(a1), "r"(a2), "r"(a3), "r"(b0), "r"(b1));
-}
-struct FragA { Tf2 v[4]; };
-struct FragB { Tf2 v[2]; };
-// A[m][k] = p[m * ld + k] at (m, k) of the fragment's corner
-__device__ __forceinline__ FragA frag_a(const float* p, int ld, int g, int tq) {
-    FragA f;
-    f.v[0] = split_tf32(p[g * ld + tq]); f.v[1] = split_tf32(p[(g + 8) * ld + tq]);
-    f.v[2] = split_tf32(p[g * ld + tq + 4]); f.v[3] = split_tf32(p[(g + 8) * ld + tq + 4]);
-    return f;
-}
-// B[k][n] = p[k * ld + n]
-__device__ __forceinline__ FragB frag_b(const float* p, int ld, int g, int tq) {
-    FragB f;
-    f.v[0] = split_tf32(p[tq * ld + g]); f.v[1] = split_tf32(p[(tq + 4) * ld + g]);
-    return f;
-}
-__device__ __forceinline__ void mma3(float (&d)[4], const FragA& a, const FragB& b) {
-    mma_tf32(d, a.v[0].lo, a.v[1].lo, a.v[2].lo, a.v[3].lo, b.v[0].hi, b.v[1].hi);
-    mma_tf32(d, a.v[0].hi, a.v[1].hi, a.v[2].hi, a.v[3].hi, b.v[0].lo, b.v[1].lo);
-    mma_tf32(d, a.v[0].hi, a.v[1].hi, a.v[2].hi, a.v[3].hi, b.v[0].hi, b.v[1].hi);
-}
-__device__ __forceinline__ void cp16(float* dst, const float* src, bool ok) {
-    const uint32_t d = (uint32_t)__cvta_generic_to_shared(dst);
-    const int bytes = ok ? 16 : 0;                        // 0: the 16 bytes are filled with zeros
-    asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(d), "l"(src), "r"(bytes) : "memory");
-}
-
 constexpr int SA = CH + 4;
 __host__ __device__ constexpr int chunk_sk(int dk16) { return dk16 + 4; }
 __host__ __device__ constexpr int chunk_ss(int dvb) { return dvb + 8; }
@@ -836,7 +743,6 @@ cudaError_t launch_delta_chunk(const DeltaArgs& a, cudaStream_t st, int* launche
     if (!chunk_shape(a.dk, a.dv, (long)a.nseq * a.H, &nw, &ntw)) return cudaErrorInvalidValue;
     const int dk4 = (a.dk + 3) / 4 * 4, dk16 = (a.dk + 15) / 16 * 16, dvb = nw * ntw * 8;
     const size_t smem = chunk_smem(dk16, dvb);
-    const long ow = (long)a.nseq * a.ts * a.H;
     const int bps = (a.ts + kPrepRows - 1) / kPrepRows;
     const unsigned pg = (unsigned)(((long)a.nseq * bps * (2 * a.G + a.H + 1) + 7) / 8);
     bool prepared = false;
@@ -863,8 +769,8 @@ cudaError_t launch_delta_chunk(const DeltaArgs& a, cudaStream_t st, int* launche
         delta_chunk_kernel<1><<<grid, nw * 64, smem, st>>>(a, dk4, dk16);
     }
     if ((e = cudaGetLastError()) != cudaSuccess) return e;
-    delta_out_kernel<<<(unsigned)((ow + 7) / 8), 256, 0, st>>>(a);
-    if ((e = cudaGetLastError()) != cudaSuccess) return e;
+    const HeadGateArgs hg{a.o32, a.H, a.dv, a.dvp, a.proj + a.off_g, a.ldp, a.o_norm, a.eps, a.row_len, a.t_abs0, a.ctl, a.nseq, a.ts, a.b0, a.y32, a.yhi, a.ylo, a.ldy};
+    if ((e = launch_head_gate(hg, st)) != cudaSuccess) return e;
     *launches = 4;
     return launch_tail(a, st);
 }

@@ -272,12 +272,98 @@ __device__ __forceinline__ float4 gamma4(const float* gamma, int col) {
     return gamma != nullptr ? __ldg(reinterpret_cast<const float4*>(gamma + col)) : make_float4(1.f, 1.f, 1.f, 1.f);
 }
 
-template <int BN, bool SPLIT>
+// what the accumulator is added to: the output's old values and / or the bias
+__device__ __forceinline__ float4 start4(const float* old, const float* bias, int col) {
+    float4 o = old != nullptr ? __ldcg(reinterpret_cast<const float4*>(old)) : make_float4(0.f, 0.f, 0.f, 0.f);
+    if (bias != nullptr) {
+        const float4 b = __ldg(reinterpret_cast<const float4*>(bias + col));
+        o.x += b.x; o.y += b.y; o.z += b.z; o.w += b.w;
+    }
+    return o;
+}
+__device__ __forceinline__ float sigmoid_f(float v) { return __frcp_rn(1.0f + __expf(-v)); }
+
+// Epilogue of a product in groups or with gated results for 32 columns of W that start at n within the group (GemmExt): row `row` of
+// the output, accumulators r times rs.
+__device__ __forceinline__ void ext_strip(const uint32_t (&r)[32], float rs, int row, int group, int n, float* D, int ldd, const NormFuse& nf,
+                                          const GemmExt& ex) {
+    float v[32];
+#pragma unroll
+    for (int j = 0; j < 32; ++j) v[j] = __uint_as_float(r[j]) * rs;
+    if (nf.bias != nullptr) {
+        const float* b = nf.bias + (size_t)group * ex.group_rows + n;
+#pragma unroll
+        for (int j = 0; j < 8; ++j) {
+            const float4 t = __ldg(reinterpret_cast<const float4*>(b + 4 * j));
+            v[4 * j] += t.x; v[4 * j + 1] += t.y; v[4 * j + 2] += t.z; v[4 * j + 3] += t.w;
+        }
+    }
+    int n0 = n, cnt = 32;
+    if (ex.gate != 0) {
+#pragma unroll
+        for (int j = 0; j < 16; ++j) {
+            const float g = v[j], u = v[16 + j];
+            v[j] = (ex.gate == ACT_RELU_GATE ? fmaxf(g, 0.f) : g * sigmoid_f(g)) * u;
+        }
+        n0 >>= 1;
+        cnt = 16;
+    }
+    cnt = min(cnt, ex.out_n - n0);
+    if (cnt <= 0) return;
+    const int col = group * ex.out_step + n0;
+    if (ex.mul != nullptr) {
+        const float* m = ex.mul + (size_t)row * ex.ldmul + col;
+#pragma unroll
+        for (int j = 0; j < 32; ++j) if (j < cnt) v[j] *= sigmoid_f(m[j]);
+    }
+    const bool whole = (cnt & 7) == 0 && ((col | ldd | ex.ldo) & 7) == 0;
+#pragma unroll
+    for (int j8 = 0; j8 < 4; ++j8) {
+        if (whole) {
+            if (8 * j8 >= cnt) break;
+            if (D != nullptr) {
+                float* dp = D + (size_t)row * ldd + col + 8 * j8;
+                *reinterpret_cast<float4*>(dp) = make_float4(v[8 * j8], v[8 * j8 + 1], v[8 * j8 + 2], v[8 * j8 + 3]);
+                *reinterpret_cast<float4*>(dp + 4) = make_float4(v[8 * j8 + 4], v[8 * j8 + 5], v[8 * j8 + 6], v[8 * j8 + 7]);
+            }
+            if (nf.out_hi != nullptr) {
+                uint32_t hw[4], lw[4];
+#pragma unroll
+                for (int e = 0; e < 4; ++e) {
+                    const float w0 = v[8 * j8 + 2 * e], w1 = v[8 * j8 + 2 * e + 1];
+                    const __nv_bfloat162 h = __floats2bfloat162_rn(w0, w1);
+                    const float2 f = __bfloat1622float2(h);
+                    const __nv_bfloat162 l = __floats2bfloat162_rn(w0 - f.x, w1 - f.y);
+                    hw[e] = *reinterpret_cast<const uint32_t*>(&h);
+                    lw[e] = *reinterpret_cast<const uint32_t*>(&l);
+                }
+                const size_t oo = (size_t)row * ex.ldo + col + 8 * j8;
+                *reinterpret_cast<uint4*>(nf.out_hi + oo) = make_uint4(hw[0], hw[1], hw[2], hw[3]);
+                if (nf.out_lo != nullptr) *reinterpret_cast<uint4*>(nf.out_lo + oo) = make_uint4(lw[0], lw[1], lw[2], lw[3]);
+            }
+        } else {
+#pragma unroll
+            for (int e = 0; e < 8; ++e) {
+                const int j = 8 * j8 + e;
+                if (j < cnt) {
+                    if (D != nullptr) D[(size_t)row * ldd + col + j] = v[j];
+                    if (nf.out_hi != nullptr) {
+                        const __nv_bfloat16 h = __float2bfloat16_rn(v[j]);
+                        nf.out_hi[(size_t)row * ex.ldo + col + j] = h;
+                        if (nf.out_lo != nullptr) nf.out_lo[(size_t)row * ex.ldo + col + j] = __float2bfloat16_rn(v[j] - __bfloat162float(h));
+                    }
+                }
+            }
+        }
+    }
+}
+
+template <int BN, bool SPLIT, bool EXT>
 __global__ void __launch_bounds__(192, 1)
 gemm_persistent_kernel(const __grid_constant__ CUtensorMap map_ahi, const __grid_constant__ CUtensorMap map_alo,
                        const __grid_constant__ CUtensorMap map_w, float* D, int ldd, int M, int N, int K,
                        int accumulate, int tiles_m, int ntiles, int splits, int32_t* tile_counters, float* scratch, int32_t* status,
-                       uint64_t wait_ns, int skip_unit, NormFuse nf) {
+                       uint64_t wait_ns, int skip_unit, NormFuse nf, GemmExt ex) {
     using T = Tile<BN, SPLIT, 1>;
     constexpr int S = T::STAGES;
     extern __shared__ uint8_t smem_raw[];
@@ -319,9 +405,28 @@ gemm_persistent_kernel(const __grid_constant__ CUtensorMap map_ahi, const __grid
     // The weights do not depend on any predecessor: the producer requests the weight tiles of its first stages before the
     // wait, so that they stream from HBM under the predecessor's tail (at 64-128 rows the weights are most of the bytes).
     uint32_t pre = 0;                            // stages whose weight tile is already on its way (and whose bytes are expected)
-    if (warp == 0 && lane == 0 && (int)blockIdx.x < ntiles * splits && (int)blockIdx.x != skip_unit) {
+    // where a tile lies: first row of A and of W, first element of K in A, and (EXT) its group, its first row of W in the group and
+    // the rows of A behind it
+    struct Place { int m0, n0, k0, group, n, m_end; };
+    const int tiles_pg = EXT ? (ex.group_rows + BN - 1) / BN : 0;       // column tiles per group
+    auto place = [&](int t) {
+        Place p;
+        if constexpr (!EXT) {
+            p.m0 = (t % tiles_m) * BM; p.n0 = (t / tiles_m) * BN; p.k0 = 0; p.group = 0; p.n = p.n0; p.m_end = M;
+        } else if (ex.tiles != nullptr) {
+            const int4 rt = __ldg(ex.tiles + t / tiles_pg);
+            p.m0 = rt.x; p.m_end = rt.x + rt.y; p.group = rt.z; p.n = (t % tiles_pg) * BN; p.n0 = p.group * ex.group_rows + p.n; p.k0 = 0;
+        } else {
+            const int tn = t / tiles_m;
+            p.m0 = (t % tiles_m) * BM; p.m_end = M; p.group = tn / tiles_pg; p.n = (tn % tiles_pg) * BN; p.n0 = p.group * ex.group_rows + p.n;
+            p.k0 = p.group * K;
+        }
+        return p;
+    };
+    const bool by_rows = EXT && ex.tiles != nullptr;      // the tiles are known only behind the dependency wait
+    if (!by_rows && warp == 0 && lane == 0 && (int)blockIdx.x < ntiles * splits && (int)blockIdx.x != skip_unit) {
         const int t = blockIdx.x / splits, sp = blockIdx.x - t * splits;
-        const int n0 = (t / tiles_m) * BN;
+        const int n0 = place(t).n0;
         const int kb0 = sp * num_kb / splits, kb1 = (sp + 1) * num_kb / splits;
         pre = (uint32_t)min(S, kb1 - kb0);
         for (uint32_t i = 0; i < pre; ++i) {
@@ -330,6 +435,7 @@ gemm_persistent_kernel(const __grid_constant__ CUtensorMap map_ahi, const __grid
         }
     }
     asm volatile("griddepcontrol.wait;" ::: "memory");
+    if (by_rows) ntiles = __ldcg(ex.n_tiles) * tiles_pg;
 
     bool timed_out = false;
     if (warp == 0) {
@@ -338,7 +444,8 @@ gemm_persistent_kernel(const __grid_constant__ CUtensorMap map_ahi, const __grid
             for (int u = blockIdx.x; u < ntiles * splits && !timed_out; u += gridDim.x) {
                 if (u == skip_unit) break;       // test hook: this unit's operands never arrive, so the waits below it run out
                 const int t = u / splits, sp = u - t * splits;
-                const int m0 = (t % tiles_m) * BM, n0 = (t / tiles_m) * BN;
+                const Place pl = place(t);
+                const int m0 = pl.m0, n0 = pl.n0;
                 const int kb0 = sp * num_kb / splits, kb1 = (sp + 1) * num_kb / splits;
                 for (int kb = kb0; kb < kb1; ++kb, ++kbg) {
                     const int s = kbg % S;
@@ -346,8 +453,8 @@ gemm_persistent_kernel(const __grid_constant__ CUtensorMap map_ahi, const __grid
                     if (!mbar_wait(&empty_bar[s], ph ^ 1u, wait_ns)) { timed_out = true; break; }
                     uint8_t* st = base + s * T::STAGE;
                     if (kbg >= pre) mbar_expect_tx(&full_bar[s], (uint32_t)T::STAGE);
-                    tma_load_2d(st, &map_ahi, &full_bar[s], kb * BK, m0);
-                    if (SPLIT) tma_load_2d(st + T::A_BYTES, &map_alo, &full_bar[s], kb * BK, m0);
+                    tma_load_2d(st, &map_ahi, &full_bar[s], pl.k0 + kb * BK, m0);
+                    if (SPLIT) tma_load_2d(st + T::A_BYTES, &map_alo, &full_bar[s], pl.k0 + kb * BK, m0);
                     if (kbg >= pre) tma_load_2d(st + T::A_BYTES * (SPLIT ? 2 : 1), &map_w, &full_bar[s], kb * BK, n0);
                 }
             }
@@ -399,7 +506,8 @@ gemm_persistent_kernel(const __grid_constant__ CUtensorMap map_ahi, const __grid
         for (int u = blockIdx.x; u < ntiles * splits; u += gridDim.x, ++it) {
             const uint32_t as = it & 1u, aph = (it >> 1) & 1u;
             const int t = u / splits, sp = u - t * splits;
-            const int m0 = (t % tiles_m) * BM, n0 = (t / tiles_m) * BN;
+            const Place pl = place(t);
+            const int m0 = pl.m0, n0 = pl.n0;
             // RMSNorm folded around the product (inference/src/model.rs:100-106 with the per-row scale moved behind the
             // contraction): the rows of A were written as x * gamma WITHOUT the scale 1 / sqrt(mean(x^2) + eps); the
             // sums of squares arrive as `ssq_parts` partial sums per row (one per 32 columns of x, added in column order,
@@ -471,7 +579,7 @@ gemm_persistent_kernel(const __grid_constant__ CUtensorMap map_ahi, const __grid
                             if (vec) {
                                 float4 o[4], pv[kMaxSplits][4];
 #pragma unroll
-                                for (int j = 0; j < 4; ++j) o[j] = acc_in ? __ldcg(reinterpret_cast<const float4*>(dp + 4 * j)) : make_float4(0.f, 0.f, 0.f, 0.f);
+                                for (int j = 0; j < 4; ++j) o[j] = start4(acc_in ? dp + 4 * j : nullptr, nf.bias, col + 4 * j);
 #pragma unroll
                                 for (int s2 = 0; s2 < kMaxSplits; ++s2)
 #pragma unroll
@@ -496,7 +604,7 @@ gemm_persistent_kernel(const __grid_constant__ CUtensorMap map_ahi, const __grid
                                     if (col + e < nlim) {
                                         float sum = 0.f;
                                         for (int s2 = 0; s2 < splits; ++s2) sum += __ldcg(scratch + ((size_t)(s2 * ntiles + t) * BM + row_l) * BN + c16 + e);
-                                        v[e] = epi_act(fmaf(sum, rs, acc_in ? __ldcg(dp + e) : 0.f), nf.act);
+                                        v[e] = epi_act(fmaf(sum, rs, (acc_in ? __ldcg(dp + e) : 0.f) + (nf.bias != nullptr ? nf.bias[col + e] : 0.f)), nf.act);
                                         if (D != nullptr) dp[e] = v[e];
                                     }
                                 }
@@ -534,6 +642,14 @@ gemm_persistent_kernel(const __grid_constant__ CUtensorMap map_ahi, const __grid
                 continue;
             }
             const int row = m0 + q * 32 + lane;
+            if constexpr (EXT) {
+#pragma unroll 1
+                for (int cb = 0; cb < BN / 32; ++cb) {
+                    uint32_t r[32];
+                    tmem_ld32(tmem_base + ((uint32_t)(q * 32) << 16) + as * ACC_COLS + (uint32_t)(cb * 32), r);
+                    if (row < pl.m_end && pl.n + cb * 32 < ex.group_rows) ext_strip(r, rs, row, pl.group, pl.n + cb * 32, D, ldd, nf, ex);
+                }
+            } else
 #pragma unroll 1
             for (int cb = 0; cb < (BN + 31) / 32; ++cb) {
                 uint32_t r[32];
@@ -548,7 +664,7 @@ gemm_persistent_kernel(const __grid_constant__ CUtensorMap map_ahi, const __grid
                         // as far as the compiler can tell, and a load behind a store would wait a whole L2 round trip
                         float4 o[8];
 #pragma unroll
-                        for (int j = 0; j < 8; ++j) o[j] = acc_in ? __ldcg(reinterpret_cast<const float4*>(dp + 4 * j)) : make_float4(0.f, 0.f, 0.f, 0.f);
+                        for (int j = 0; j < 8; ++j) o[j] = start4(acc_in ? dp + 4 * j : nullptr, nf.bias, col0 + 4 * j);
                         float4 v[8];
 #pragma unroll
                         for (int j = 0; j < 8; ++j)
@@ -590,6 +706,7 @@ gemm_persistent_kernel(const __grid_constant__ CUtensorMap map_ahi, const __grid
                             if (col0 + j < nlim) {
                                 float v = __uint_as_float(r[j]) * rs;
                                 if (acc_in) v += __ldcg(dp + j);
+                                if (nf.bias != nullptr) v += nf.bias[col0 + j];
                                 v = epi_act(v, nf.act);
                                 if (D != nullptr) dp[j] = v;
                                 if (nf.out_hi != nullptr) {
@@ -663,17 +780,19 @@ int sm_count_gemm() {
     return n;
 }
 
-template <int BN, bool SPLIT>
+template <int BN, bool SPLIT, bool EXT = false>
 int32_t launch_persistent(const GemmArgs& a, int splits, cudaStream_t st) {
     using T = Tile<BN, SPLIT, 1>;
     CUtensorMap mh, ml, mw;
-    LUMI_TRY(make_map(&mh, a.a_hi, a.M, a.K, BM));
-    LUMI_TRY(make_map(&ml, SPLIT ? a.a_lo : a.a_hi, a.M, a.K, BM));
+    const int lda = EXT ? a.ext->lda : a.K;
+    LUMI_TRY(make_map(&mh, a.a_hi, a.M, lda, BM));
+    LUMI_TRY(make_map(&ml, SPLIT ? a.a_lo : a.a_hi, a.M, lda, BM));
     LUMI_TRY(make_map(&mw, a.w, a.N, a.K, BN));
-    auto kern = gemm_persistent_kernel<BN, SPLIT>;
+    auto kern = gemm_persistent_kernel<BN, SPLIT, EXT>;
     LUMI_CUDA(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, T::SMEM));
-    const int tiles_m = (a.M + BM - 1) / BM, tiles_n = (a.N + BN - 1) / BN;
-    const int ntiles = tiles_m * tiles_n;
+    const int tiles_m = (a.M + BM - 1) / BM;
+    const int tiles_n = EXT ? (a.ext->group_rows + BN - 1) / BN * (a.ext->tiles != nullptr ? 1 : a.ext->groups) : (a.N + BN - 1) / BN;
+    const int ntiles = (EXT && a.ext->tiles != nullptr ? a.ext->max_tiles : tiles_m) * tiles_n;      // by rows: as many as there can be
     const int units = ntiles * splits;
     const int grid = units < sm_count_gemm() ? units : sm_count_gemm();
     cudaLaunchConfig_t cfg = {};
@@ -687,7 +806,7 @@ int32_t launch_persistent(const GemmArgs& a, int splits, cudaStream_t st) {
     cfg.attrs = attr;
     cfg.numAttrs = launch_pdl_gemm_on() ? 1 : 0;   // the set-up overlaps the predecessor's tail
     LUMI_CUDA(cudaLaunchKernelEx(&cfg, kern, mh, ml, mw, a.d, a.ldd, a.M, a.N, a.K, a.accumulate, tiles_m, ntiles, splits, a.tile_counters,
-                                 a.scratch, a.status_word, a.wait_limit_ns ? a.wait_limit_ns : kWaitLimitNs, a.debug_skip_unit, a.nf));
+                                 a.scratch, a.status_word, a.wait_limit_ns ? a.wait_limit_ns : kWaitLimitNs, a.debug_skip_unit, a.nf, EXT ? *a.ext : GemmExt()));
     return LUMI_OK;
 }
 
@@ -783,14 +902,40 @@ static void pick_tile(const GemmArgs& a, int* width, int* splits) {
 // The tile width and K split launch_gemm_tcgen05 would take for these arguments (host-side choice only; nothing is launched).
 void gemm_tcgen05_plan(const GemmArgs& a, int* width, int* splits) { pick_tile(a, width, splits); }
 
+// Products in groups and gated results.
+static int32_t launch_ext(const GemmArgs& a, cudaStream_t st) {
+    const GemmExt& e = *a.ext;
+    const bool by_rows = e.tiles != nullptr;
+    if (e.group_rows <= 0 || e.group_rows % 32 || e.groups <= 0 || e.groups * e.group_rows != a.N || e.lda % 64 || e.lda < (by_rows ? a.K : e.groups * a.K) ||
+        e.out_n <= 0 || a.accumulate || a.nf.ssq_out != nullptr || (by_rows && (e.n_tiles == nullptr || e.max_tiles <= 0)) ||
+        (a.nf.out_hi != nullptr && e.ldo <= 0) || (a.d == nullptr && a.nf.out_hi == nullptr))
+        return fail(LUMI_E_INVALID, "tcgen05 GEMM in groups: %d groups of %d rows of W, N %d, rows of A of %d elements", e.groups, e.group_rows, a.N, e.lda);
+    LUMI_TRY(gemm_tcgen05_init());
+    const long tiles_m = by_rows ? e.max_tiles : (a.M + BM - 1) / BM;
+    int best = 256;
+    long best_cost = -1;
+    for (int w : {256, 128, 64, 32}) {
+        const long tiles = tiles_m * ((e.group_rows + w - 1) / w) * (by_rows ? 1 : e.groups);
+        const long rounds = (tiles + sm_count_gemm() - 1) / sm_count_gemm();
+        const long cost = rounds * (w + 32);
+        if (best_cost < 0 || cost < best_cost) { best = w; best_cost = cost; }
+    }
+    const bool split = a.a_lo != nullptr;
+#define LUMI_EXT_CASE(W) if (best == W) return split ? launch_persistent<W, true, true>(a, 1, st) : launch_persistent<W, false, true>(a, 1, st);
+    LUMI_EXT_CASE(256) LUMI_EXT_CASE(128) LUMI_EXT_CASE(64) LUMI_EXT_CASE(32)
+#undef LUMI_EXT_CASE
+    return LUMI_OK;
+}
+
 int32_t launch_gemm_tcgen05(const GemmArgs& a, cudaStream_t st) {
     if (a.M <= 0 || a.N <= 0 || a.K <= 0 || (a.K % BK) != 0)
         return fail(LUMI_E_UNSUPPORTED, "tcgen05 GEMM needs K %% 64 == 0 (M %d N %d K %d)", a.M, a.N, a.K);
     if ((reinterpret_cast<uintptr_t>(a.a_hi) | reinterpret_cast<uintptr_t>(a.w) | reinterpret_cast<uintptr_t>(a.a_lo)) & 15)
         return fail(LUMI_E_INVALID, "tcgen05 GEMM operands must be 16-byte aligned");
+    if (a.ext != nullptr) return launch_ext(a, st);
     LUMI_TRY(gemm_tcgen05_init());
     const bool split = a.a_lo != nullptr;
-    const bool fused = a.nf.ssq_in != nullptr || a.nf.out_hi != nullptr || a.nf.act != 0;
+    const bool fused = a.nf.ssq_in != nullptr || a.nf.out_hi != nullptr || a.nf.act != 0 || a.nf.bias != nullptr;
     if (a.nf.out_hi != nullptr && a.nf.gamma_next == nullptr && a.nf.ssq_out == nullptr) {
         if ((a.N & 7) != 0) return fail(LUMI_E_INVALID, "a result in bf16 halves needs N %% 8 == 0");
     } else if (a.nf.out_hi != nullptr && ((a.N & 7) != 0 || a.nf.gamma_next == nullptr || a.nf.ssq_out == nullptr || a.nf.ssq_stride * 32 < a.N))

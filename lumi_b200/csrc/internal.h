@@ -31,13 +31,19 @@ int32_t fail(int32_t code, const char* fmt, ...);
 
 // ---- configuration (ModelConfig of the reference, inference/src/model.rs:20-86) -----------------
 // One layer of a model whose config lists its layers one by one: a mixer and, behind it, an optional feed-forward, each
-// followed by a norm of its OUTPUT before it joins the residual stream.  Every mixer constant is a field here, so that
-// another design can combine them differently.
-enum MixerKind { MIXER_NONE = 0, MIXER_DELTA, MIXER_ATTENTION };
+// either behind a norm of the residual stream (pre_norm) or followed by a norm of its OUTPUT before it joins the stream.
+// Every mixer constant is a field here, so that another design can combine them differently.
+enum MixerKind { MIXER_NONE = 0, MIXER_DELTA, MIXER_ATTENTION, MIXER_RETENTION, MIXER_RGLRU, MIXER_LATENT };
+// Rotary positions: `dims` of a head's dimensions turn by p * base^(-2i/dims), dimension i with i + dims/2, or (pairs) 2i with 2i + 1.
+struct RotSpec {
+    int dims = 0;
+    bool pairs = false;
+    double base = 10000.0;
+};
 struct MixerSpec {
     MixerKind kind = MIXER_NONE;
     int heads = 0, kv_heads = 0, dim = 0, vdim = 0;
-    int taps = 1;              // delta rule: length of the short convolutions
+    int taps = 1;              // delta rule, gated linear recurrence: length of the short convolutions
     float unit_eps = 1e-6f;    // delta rule: epsilon inside the root of the unit vectors
     float scale = 1.f;         // attention: factor of the scores
     int window = 0;            // attention: tokens a position sees, itself included (0 = all)
@@ -45,10 +51,31 @@ struct MixerSpec {
     bool qk_norm = false;      // attention: q and k over their root mean square
     bool sink = false;         // attention: one score of `sink_score` without a value joins the softmax
     float sink_score = 0.f;
+    RotSpec rot;               // retention (first dimensions of q and k), latent attention (the rot_dim part of q and k)
+    int kv_rank = 0;           // latent attention: size of the cached latent
+    int rot_dim = 0;           // latent attention: rotated dimensions per query head and of the shared key part
+    int channels = 0;          // gated linear recurrence: width of its two branches
+    int blocks = 0;            // gated linear recurrence: blocks of the gates' matrices
+    float decay_rate = 8.f;    // gated linear recurrence: log a = -decay_rate * r * softplus(lam)
+    bool recurrent() const { return kind == MIXER_DELTA || kind == MIXER_RETENTION || kind == MIXER_RGLRU; }
+    bool cached() const { return kind == MIXER_ATTENTION || kind == MIXER_LATENT; }
+};
+// Activations of a product.  Gated ones take the rows of W in groups of 16 gate rows and the 16 up rows that belong to them:
+// result n = act(gate n) * up n.  ACT_SIGMOID_GATE is the hybrid's form (gate rows first, then the up rows).
+enum Act { ACT_NONE = 0, ACT_SIGMOID_GATE = 1, ACT_RELU2 = 2, ACT_RELU_GATE = 3, ACT_SILU_GATE = 4 };
+struct FfSpec {
+    int ff = 0;                // width (0 = no feed-forward)
+    int act = ACT_RELU2;       // gated kinds have a gate matrix beside the up matrix
+    bool bias = false;
+    int experts = 0, top = 0;  // mixture of experts (0 = dense): sigmoid scores, the weight multiplies the expert's input
+    bool gated() const { return act == ACT_RELU_GATE || act == ACT_SILU_GATE; }
 };
 struct LayerSpec {
     MixerSpec mixer;
-    int ff = 0;                // width of the squared-ReLU feed-forward (0 = none)
+    FfSpec ff;
+    bool pre_norm = false;
+    int weights_of = -1;       // layer whose weights are used (-1 = its own); cache and state are always its own
+    std::vector<float> decay;  // retention: decay per head
 };
 
 struct Config;
@@ -61,7 +88,7 @@ struct Architecture {
     int32_t (*parse)(const JsonValue& root, Config& out);
     // shape of a tensor by its name (prefix removed); rank 0 = not a tensor of this model.  `wide` is set for tensors
     // that are kept in fp32 whatever their rank
-    int (*expected_shape)(const Config& c, const std::string& name, int64_t shp[2], bool& wide);
+    int (*expected_shape)(const Config& c, const std::string& name, int64_t shp[3], bool& wide);
 };
 const Architecture* find_architecture(const char* name);  // null if there is none of that name
 
@@ -77,6 +104,8 @@ struct Config {
     std::vector<LayerSpec> specs;          // one entry per layer for designs that list them; empty for the hybrid
     float embed_scale = 1.f;
     bool embed_positions = false;          // sinusoidal position vectors are added to the embedding
+    bool own_head = false;                 // the output matrix is a tensor of its own, not the embedding
+    bool norm_offset = true;               // norm weights of listed designs are stored as offsets from one
 
     bool stacked() const { return !specs.empty(); }
     // elements per row of the residual stream on the device: rows of listed designs are padded with zeros to whole
@@ -84,7 +113,7 @@ struct Config {
     int x_ld() const { return stacked() ? (d_model + 63) / 64 * 64 : d_model; }
     int max_window() const {               // most tokens an attention layer looks back over; 0 = one of them sees all
         int w = 1;
-        for (const LayerSpec& l : specs) if (l.mixer.kind == MIXER_ATTENTION) { if (l.mixer.window <= 0) return 0; if (l.mixer.window > w) w = l.mixer.window; }
+        for (const LayerSpec& l : specs) if (l.mixer.cached()) { if (l.mixer.window <= 0) return 0; if (l.mixer.window > w) w = l.mixer.window; }
         return w;
     }
 
@@ -129,6 +158,26 @@ struct SubW {
     const float *conv_q = nullptr, *conv_k = nullptr, *conv_v = nullptr;      // [channels][taps]
     const float *a_log = nullptr, *dt_bias = nullptr, *o_norm = nullptr;
     const float *norm1 = nullptr, *norm2 = nullptr;                           // [x_ld]
+    const float *in_b = nullptr, *up_b = nullptr, *down_b = nullptr;          // biases by weight row (may be null)
+    const double* rot_freq = nullptr;                                         // [rot.dims / 2] frequencies in half turns per position
+    const float* decay_pow = nullptr;                                         // retention: [heads][kDecayPowers] powers 0, 1, ... of the decay
+    // gated linear recurrence: [block][2 bp][bp], rows in groups of 16 of the decay gate and 16 of the input gate (bp: block size
+    // padded to 64), biases in the same order; conv_q holds the filter
+    DevTensor rg; const float *rg_b = nullptr, *conv_b = nullptr, *lam = nullptr;
+    int off_x = 0, off_y = 0, off_c = 0;
+    // latent attention: key up-projection per head transposed [head][lp][dp], value up-projection [head][vdim][lp], and both as one
+    // matrix over a cache row for prompts [head][dk_pad + dv_pad][row]; norm weight of the latent
+    DevTensor uk, uv, ukv; const float* c_norm = nullptr;
+    // experts: up [expert][2 ffp][x_ld] (gate and up rows in groups of 16), down [expert][x_ld][ffp]
+    DevTensor router;
+};
+constexpr int kDecayPowers = 65;
+// Padded sizes of a latent attention layer: latent, unrotated query part, cache row.
+struct LatentShape {
+    int lp, dp, row, dk, dk_pad, dv_pad;
+    __host__ __device__ explicit LatentShape(const MixerSpec& m)
+        : lp((m.kv_rank + 63) / 64 * 64), dp((m.dim + 63) / 64 * 64), row((lp + m.rot_dim + 63) / 64 * 64), dk(m.dim + m.rot_dim),
+          dk_pad((dk + 15) / 16 * 16), dv_pad((m.vdim + 15) / 16 * 16) {}
 };
 struct Layer {
     bool is_attn = false;
@@ -153,9 +202,10 @@ struct lumi_model {
     std::vector<void*> owned;                         // extra device allocations made at finalize
     std::vector<lumi::Layer> layers;
     lumi::DevTensor embedding;
+    lumi::DevTensor head;                             // listed designs: the embedding, or a matrix of its own
     const float* final_norm_g = nullptr;
     int n_mamba = 0, n_attn = 0;
-    int n_delta = 0, n_wattn = 0;                     // listed layers by mixer
+    int n_recur = 0, n_wattn = 0;                     // listed layers with a recurrent state, and with a cache
     int64_t weight_bytes = 0;                         // bytes of weights one decode step reads
 };
 
@@ -197,10 +247,18 @@ struct LayerState {
     void* kv = nullptr;         // attention: page pool [slot pages][kv_head][K rows | V rows of 64 tokens], rows padded to dk_pad / dv_pad
     size_t kv_bytes = 0;
     int dk_pad = 0, dv_pad = 0;
-    float* S = nullptr;         // delta rule: [slot][head][dim][dv_pad]
-    float* conv = nullptr;      // delta rule: [slot][taps][channels] raw inputs of the short convolutions, ring over positions
+    float* S = nullptr;         // delta rule, retention: [slot][head][dim][dv_pad]; gated linear recurrence: [slot][channels]
+    float* conv = nullptr;      // [slot][taps][channels] raw inputs of the short convolutions, ring over positions
     int dvp = 0, channels = 0;
     size_t s_seq = 0, conv_seq = 0;      // floats per sequence
+};
+// Buffers of a mixture of experts over `rows` token rows at a time: the (row, expert) pairs sorted by expert, operand halves, hidden
+// halves and results; fp32 hidden rows where no tensor cores are used.
+struct MoeBufs {
+    int rows = 0;
+    float *logits = nullptr, *y = nullptr, *h32 = nullptr;
+    __nv_bfloat16 *gh = nullptr, *gl = nullptr, *hh = nullptr, *hl = nullptr;
+    int32_t* plan = nullptr;                         // see MoeArgs
 };
 // Row buffers of a pass over listed layers (one set for decode steps, one for prompt slices).
 struct RowBufs {
@@ -209,6 +267,13 @@ struct RowBufs {
     float *x2 = nullptr;                             // where x goes when a product's prologue adds to it (few rows)
     float *proj = nullptr, *mix = nullptr, *qkv = nullptr, *gates = nullptr, *y32 = nullptr;
     __nv_bfloat16 *xh = nullptr, *xl = nullptr, *ah = nullptr, *al = nullptr;
+    float* ssq = nullptr; int ssq_stride = 0;        // pre-norm layers: sums of squares beside xh / xl
+    __nv_bfloat16 *bh = nullptr, *bl = nullptr;      // operand rows of products by blocks (gated linear recurrence)
+    // latent attention with queries in the latent space: queries, contexts, and either as halves
+    size_t lat_rows = 0;
+    float *qlat = nullptr, *ctx = nullptr;
+    __nv_bfloat16 *lh = nullptr, *ll = nullptr;
+    lumi::MoeBufs moe;
 };
 }
 
@@ -261,6 +326,8 @@ struct lumi_session {
     int pages_per_seq = 0;
     // designs that list their layers
     std::vector<lumi::LayerState> lstate;
+    __nv_bfloat16* lat_kv = nullptr;   // latent attention, prompt slices: keys and values per head of a few sequences' rings
+    size_t lat_kv_cap = 0;
     lumi::RowBufs dec, pre;
     int kv_limit = 0;                  // positions at or past it are refused (0 = the ring takes any)
     int slice_max = 0;                 // most tokens of a sequence per pass (what the ring leaves beside the widest window)
@@ -313,7 +380,7 @@ struct GemvArgs {
     const float* gamma;              // RMSNorm weight applied to rows of A first, or null
     int M, N, K;
     float eps;
-    int act;                         // 0 none; 1: D = sigmoid(W_gate a) * (W_up a), W = [gate rows | up rows], N = rows of each; 2: D = max(0, W a)^2
+    int act;                         // Act; gated kinds: N = results (pairs of rows)
     int32_t* status = nullptr;       // device word that receives STATUS_TIMEOUT if a bounded wait gives up; may be null
     bool allow_preload = true;       // false: never the single-wave preloading kernel (the only GEMV with a device-side wait)
     // greedy head: per (batch row, CTA) the best (value, row) of the CTA's rows goes to amax_val / amax_idx
@@ -323,6 +390,8 @@ struct GemvArgs {
     int amax_stride = 0;
     int* amax_parts = nullptr;
     PostAdd post;                    // applied before gamma
+    int norm_width = 0;              // elements the norm under gamma runs over (0 = K; the others are zero padding)
+    const float* bias = nullptr;     // by weight row
 };
 cudaError_t launch_gemv(const GemvArgs& a, cudaStream_t st);
 cudaError_t launch_logprob(const float* logits, int B, int V, const uint32_t* targets, float* out, int out_stride, int out_col,
@@ -432,9 +501,26 @@ struct NormFuse {
     const float* gamma_next = nullptr;
     __nv_bfloat16 *out_hi = nullptr, *out_lo = nullptr;
     float* ssq_out = nullptr;
-    // activation before the result is stored: 0 none, 2 max(0, v)^2.  With gamma_next null, out_hi / out_lo receive the
-    // result itself (width N) and no sums of squares are written; D may then be null
+    // activation before the result is stored: ACT_NONE, ACT_RELU2 (the gated ones belong to GemmExt).  With gamma_next null,
+    // out_hi / out_lo receive the result itself (width N) and no sums of squares are written; D may then be null
     int act = 0;
+    const float* bias = nullptr;         // [N], added before the activation
+};
+
+// Products in groups, and gated results (persistent kernel, rows of W in `groups` blocks of group_rows each).
+//   by columns:  group g multiplies columns [g K, (g + 1) K) of A (rows of lda elements); its results go to columns g * out_step + n,
+//                n < out_n.  groups == 1 is an ordinary product.
+//   by rows (tiles given): rows of A are sorted by group; row tile i holds tiles[i] = (first row, rows, group, 0), *n_tiles of them.
+// gate: ACT_RELU_GATE / ACT_SILU_GATE (rows of W as Act says; out_n and out_step count results).  mul: the result is multiplied
+// by sigmoid(mul[row * ldmul + column]).  Results go to D (ldd) and / or out_hi / out_lo (ldo).
+struct GemmExt {
+    int groups = 1, group_rows = 0, lda = 0, out_step = 0, out_n = 0;
+    const int4* tiles = nullptr;
+    const int32_t* n_tiles = nullptr;
+    int max_tiles = 0;                   // row tiles there can be (bounds the launch)
+    int gate = 0;
+    const float* mul = nullptr; int ldmul = 0;
+    int ldo = 0;
 };
 
 struct GemmArgs {
@@ -451,6 +537,7 @@ struct GemmArgs {
     uint64_t wait_limit_ns = 0;         // limit of every device-side wait (0 = the default, 0.5 s)
     int debug_skip_unit = -1;           // test hook: the producer stops before this work unit, so the consumers' waits run out
     NormFuse nf;                        // RMSNorm folded around the product (persistent kernel only)
+    const GemmExt* ext = nullptr;       // products in groups, gated results
 };
 int32_t launch_gemm_tcgen05(const GemmArgs& a, cudaStream_t st);   // returns LUMI_* status
 void gemm_tcgen05_plan(const GemmArgs& a, int* width, int* splits);     // the tile width and K split that launch would take
@@ -519,6 +606,18 @@ struct RowNormArgs {
 };
 cudaError_t launch_row_norm(const RowNormArgs& a, cudaStream_t st);
 
+// Read-outs of a recurrence head by head: o / rms(o) * w * silu(gate), rows of the pass as in DeltaArgs (dead rows are zero).
+struct HeadGateArgs {
+    const float* o; int H, dv, dvp;                  // [rows][H][dvp]
+    const float* gate; int ldg;                      // [rows][ldg], H dv elements used
+    const float* w;                                  // [dv], or null
+    float eps;
+    const int32_t* row_len; int t_abs0; const StepCtl* ctl;
+    int nseq, ts, b0;
+    float* y32; __nv_bfloat16 *yhi, *ylo; int ldy;
+};
+cudaError_t launch_head_gate(const HeadGateArgs& a, cudaStream_t st);
+
 // ---- gated delta rule (delta_rule.cu) ----------------------------------------------------------------------
 // Rows of the stacked input projections; row r = sequence b0 + r / ts, token r % ts of this pass.
 struct DeltaArgs {
@@ -558,9 +657,115 @@ struct WinAttnArgs {
     int limit;                                       // positions at or past it are refused (0 = the ring takes any)
     float* y32; __nv_bfloat16 *yhi, *ylo; int ldy;
     float* part; int32_t* part_count;                // as in AttnArgs, decode only
+    // where the rows lie, if not as LayerState says (page_elems 0): elements per page, from one head's rows to the next one's,
+    // from a K row to the next, from a V row to the next, and from a head's first K row to its first V row
+    long page_elems = 0; int head_step = 0, k_ld = 0, v_ld = 0, v_off = 0;
+    bool plain = false;                              // always the plain form
+    const float* gate = nullptr; int ldg = 0;        // the contexts are multiplied by sigmoid(gate[row * ldg + h * dv + d])
 };
 cudaError_t launch_window_attention(const WinAttnArgs& a, cudaStream_t st, int* launches);
 size_t window_attention_part_floats(const MixerSpec& m);      // room for the partial results of one (row, head group)
+
+// ---- retention (retention.cu) ------------------------------------------------------------------------------
+// Linear attention with a fixed decay per head: S_t = decay S_{t-1} + k_t v_t^T, o_t = S_t^T q_t; q and k rotated, k times k_scale;
+// o over its root mean square, times silu of the gate rows.
+struct RetentionArgs {
+    const float* proj; int ldp; int off_q, off_k, off_v, off_g;
+    float* S;                                        // this layer's state, slot 0
+    int H, dk, dv, dvp;
+    RotSpec rot; const double* freq;
+    const float* decay_pow;                          // [H][kDecayPowers]
+    float k_scale, eps;
+    const int32_t* pos;
+    const int32_t* row_len; int t_abs0; const StepCtl* ctl;      // as in DeltaArgs
+    int nseq, ts, b0;
+    float* y32; __nv_bfloat16 *yhi, *ylo; int ldy;
+    float* o32;                                      // chunked form: read-out before its norm, [rows][H][dvp]
+};
+cudaError_t launch_retention_step(const RetentionArgs& a, cudaStream_t st, int* launches);
+bool retention_chunk_supported(int dk, int dv);
+cudaError_t launch_retention_chunk(const RetentionArgs& a, cudaStream_t st, int* launches);
+
+// ---- gated linear recurrence (rglru.cu) --------------------------------------------------------------------
+// u = conv(x) per channel; r, i = sigmoid of block-diagonal products of u; log a = -rate r softplus(lam);
+// S_t = a S_{t-1} + sqrt(1 - a^2) i u; output S * gelu(y).
+struct RglruArgs {
+    const float* proj; int ldp; int off_x, off_y;
+    const float *conv_w, *conv_b, *lam;
+    const void* rg; int rg_dtype; const float* rg_b; // as in SubW
+    int channels, blocks, bp, taps;                  // bp: block size padded to 64
+    float rate;
+    float *S, *conv;                                 // this layer's state, slot 0
+    const int32_t* pos;
+    const int32_t* row_len; int t_abs0; const StepCtl* ctl;
+    int nseq, ts, b0;
+    float* u32; __nv_bfloat16 *uh, *ul;              // convolution output: [rows][channels], halves [rows][blocks bp] (may be null)
+    const float* gates;                              // [rows][blocks][2 bp] gate rows before the sigmoid (SubW order, bias included)
+    float* y32; __nv_bfloat16 *yhi, *ylo; int ldy;
+};
+cudaError_t launch_rglru_conv(const RglruArgs& a, cudaStream_t st);
+cudaError_t launch_rglru_scan(const RglruArgs& a, cudaStream_t st);
+cudaError_t launch_rglru_tail(const RglruArgs& a, cudaStream_t st);
+constexpr int kRglruStepRows = 32;                    // rows up to which a decode token takes the one-launch form
+bool rglru_step_supported(const RglruArgs& a);
+cudaError_t launch_rglru_step(const RglruArgs& a, cudaStream_t st);      // a decode token, everything in one launch
+
+// ---- latent attention (latent_attention.cu) ----------------------------------------------------------------
+struct LatentArgs {
+    float* proj; int ldp; int off_q, off_c;          // q rows are rotated in place
+    void* kv; int kv_is_f32;                         // cache rows [latent lp | rotated key | 0] of `row` elements, pages of 64
+    const int32_t* page_table; int pages_per_seq;
+    const int32_t* pos;
+    MixerSpec m; const double* freq; const float* c_norm;
+    float eps;
+    const int32_t* row_len; int t_abs0; StepCtl* ctl;
+    int nseq, ts, b0, limit;
+    __nv_bfloat16 *qh, *ql;                          // unrotated query parts [rows][H][dp] as halves (may be null)
+    float* qlat;                                     // queries over a cache row [rows][H][row]; the prep kernel writes the rotated part and padding
+    float* ctx; __nv_bfloat16 *ch, *cl;              // contexts over the latent [rows][H][lp]
+    float* part; int32_t* part_count;
+};
+cudaError_t launch_latent_prep(const LatentArgs& a, cudaStream_t st);
+cudaError_t launch_latent_attention(const LatentArgs& a, cudaStream_t st);       // queries absorbed into the latent space
+size_t latent_part_floats(const MixerSpec& m);
+
+// ---- products of a few rows by groups (block_product.cu) ---------------------------------------------------
+// D[r][g * out_step + n] = (sum_k A[r][g * a_step + k] W[g][n][k] + bias[g][n]) * sigmoid(mul[r][g * out_step + n]), n < n_out <= group_rows, k < K
+// (K <= the padded row length ldw of W).  fp32 or bf16 weights, fp32 products.
+struct BlockProductArgs {
+    const float* A; int lda, a_step;
+    const void* W; int w_dtype; int ldw, group_rows;
+    const float* bias; const float* mul; int ldmul;
+    float* D; int ldd, out_step;
+    int rows, groups, n_out, K;
+};
+cudaError_t launch_block_product(const BlockProductArgs& a, cudaStream_t st);
+// dst[(r / rg * rs + r % rg + ro) * ld + co + c] = src[r][c]; transpose: dst[(r / rg * rs + c + ro) * ld + co + r % rg]
+cudaError_t launch_pack_rows(void* dst, long ld, const void* src, long rows, long cols, int esz, long rg, long rs, long ro, long co, bool transpose,
+                             cudaStream_t st);
+
+// ---- mixture of experts (moe.cu) -----------------------------------------------------------------------------
+// plan (int32): [0] row tiles, [1] ticket, [4 ...] counts [E_max] (zeros between launches), offsets [E_max], then per pair expert and
+// place [2 pairs], weights [pairs] (as float bits) and the row tiles (int4 each, 16-byte aligned).
+struct MoeArgs {
+    const float* logits; int ldl;                    // router logits [rows][ldl]
+    int rows, E, E_max, top, D, ldx, ff, ffp;        // E_max: most experts of any layer that uses the plan
+    float* x; const float* gamma; float eps;         // residual rows and the norm in front of the router and the experts
+    int32_t* plan;
+    __nv_bfloat16 *gh, *gl;                          // experts' inputs sorted by expert [pairs][ldx]
+    float* y;                                        // experts' results [pairs][ldx]
+    // few rows: hidden rows [pairs][ffp] fp32 and the experts' weights
+    float* h32; const void *w_up, *w_down; int w_dtype, act;
+    // what the next product takes (tensor-core path): x * gamma_next as halves and its sum of squares
+    const float* gamma_next; __nv_bfloat16 *xh, *xl; float* ssq; int ssq_stride;
+};
+size_t moe_plan_ints(int rows, int top, int E_max);
+int moe_max_tiles(int rows, int top, int E);
+const int4* moe_tiles(const MoeArgs& a);
+cudaError_t launch_moe_route(const MoeArgs& a, cudaStream_t st);
+cudaError_t launch_moe_gather(const MoeArgs& a, cudaStream_t st);
+cudaError_t launch_moe_combine(const MoeArgs& a, cudaStream_t st);
+cudaError_t launch_moe_few(const MoeArgs& a, cudaStream_t st);       // two launches: route + gate and up rows, then down rows into x
 
 cudaError_t launch_gate_mul(const float* gu, int ld, float* out32, __nv_bfloat16* hi, __nv_bfloat16* lo, int B, int mlp,
                             cudaStream_t st);

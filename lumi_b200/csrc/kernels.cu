@@ -195,12 +195,19 @@ template <typename WT, int NB, int RPW, int ACT>
 __global__ void __launch_bounds__(256) gemv_kernel(const float* A, int lda, const WT* __restrict__ W,
                                                    float* D, int ldd, const float* R,
                                                    const float* __restrict__ gamma, int M, int N, int K, float eps, int KS,
-                                                   float* amax_val, int* amax_idx, int amax_stride, PostAdd post) {
+                                                   float* amax_val, int* amax_idx, int amax_stride, PostAdd post, int norm_width,
+                                                   const float* __restrict__ bias) {
     extern __shared__ float4 gemv_smem4[];
     float* xs = reinterpret_cast<float*>(gemv_smem4);
     constexpr int E = WLoad<WT>::E;
     constexpr int U = kGemvU;
-    constexpr int NR = (ACT == 1) ? 2 * RPW : RPW;     // ACT == 1 pairs weight rows n (gate) and n + N (up)
+    constexpr bool PAIR = ACT == ACT_SIGMOID_GATE || ACT == ACT_RELU_GATE || ACT == ACT_SILU_GATE;
+    constexpr int NR = PAIR ? 2 * RPW : RPW;           // a gate row and an up row per result
+    // weight row of result n: ACT_SIGMOID_GATE keeps the up rows behind all gate rows, the others in groups of 16 and 16
+    auto weight_row = [&](int n, bool up) {
+        if (ACT == ACT_RELU_GATE || ACT == ACT_SILU_GATE) return (n >> 4) * 32 + (n & 15) + (up ? 16 : 0);
+        return n + (PAIR && up ? N : 0);
+    };
     __shared__ float part[8][NR][NB];
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const int m0 = blockIdx.y * NB;
@@ -216,7 +223,7 @@ __global__ void __launch_bounds__(256) gemv_kernel(const float* A, int lda, cons
     uint4 wreg[NR][U];
 #pragma unroll
     for (int r = 0; r < NR; ++r) {
-        const int row = min(row0 + (r % RPW), N - 1) + ((ACT == 1 && r >= RPW) ? N : 0);
+        const int row = weight_row(min(row0 + (r % RPW), N - 1), r >= RPW);
         const WT* wp = W + (size_t)row * K;
 #pragma unroll
         for (int u = 0; u < U; ++u) {
@@ -279,7 +286,7 @@ __global__ void __launch_bounds__(256) gemv_kernel(const float* A, int lda, cons
                 float t = 0.f;
 #pragma unroll
                 for (int w = 0; w < 8; ++w) t += nred[b][w];
-                const float r = rms_scale(t, K, eps);
+                const float r = rms_scale(t, norm_width, eps);
                 for (int k = threadIdx.x; k < K; k += 256) xs[b * K + k] = __fmul_rn(__fmul_rn(xs[b * K + k], r), gamma[k]);
             }
         }
@@ -349,8 +356,13 @@ __global__ void __launch_bounds__(256) gemv_kernel(const float* A, int lda, cons
             for (int b = 0; b < NB; ++b) {
                 if (b >= nb) break;
                 float v = acc[r][b];
-                if constexpr (ACT == 1) v = __fmul_rn(sigmoid_ref(v), acc[RPW + r][b]);     // model.rs:550-552
-                if constexpr (ACT == 2) { v = fmaxf(v, 0.f); v = __fmul_rn(v, v); }
+                if (bias != nullptr) v += bias[weight_row(row, false)];
+                if constexpr (ACT == ACT_SIGMOID_GATE) v = __fmul_rn(sigmoid_ref(v), acc[RPW + r][b]);     // model.rs:550-552
+                if constexpr (ACT == ACT_RELU_GATE || ACT == ACT_SILU_GATE) {
+                    const float up = acc[RPW + r][b] + (bias != nullptr ? bias[weight_row(row, true)] : 0.f);
+                    v = __fmul_rn(ACT == ACT_RELU_GATE ? fmaxf(v, 0.f) : silu_ref(v), up);
+                }
+                if constexpr (ACT == ACT_RELU2) { v = fmaxf(v, 0.f); v = __fmul_rn(v, v); }
                 size_t o = (size_t)(m0 + b) * ldd + row;
                 if (R != nullptr) v = __fadd_rn(v, R[o]);
                 if (D != nullptr) D[o] = v;
@@ -404,7 +416,8 @@ template <typename WT, int NB, int U, int RPW>
 __global__ void __launch_bounds__(256, 2) gemv_pre_kernel(const float* A, int lda, const WT* __restrict__ W,
                                                           float* D, int ldd, const float* R,
                                                           const float* __restrict__ gamma, int M, int N, int K, float eps,
-                                                          int rows_per_cta, int pace_ns, int pre_delay_ns, int32_t* status, PostAdd post) {
+                                                          int rows_per_cta, int pace_ns, int pre_delay_ns, int32_t* status, PostAdd post,
+                                                          int norm_width, const float* __restrict__ bias) {
     extern __shared__ float4 gemv_smem4[];
     constexpr int E = WLoad<WT>::E;
     constexpr int GN = (U * E + 7) / 8;                 // gamma values per thread: K / 256 rounded up
@@ -487,18 +500,21 @@ __global__ void __launch_bounds__(256, 2) gemv_pre_kernel(const float* A, int ld
 
     // residuals of the rows whose stores this lane owns (register rows, first shared-memory group)
     float rres_r[NB], rres_s[NB];
+    const bool has_add = R != nullptr || bias != nullptr;
+    const float bias_r = bias != nullptr && lane < RPW && warp + 8 * lane < nrows ? bias[row_base + warp + 8 * lane] : 0.f;
+    const float bias_s = bias != nullptr && lane < GR && warp + 8 * lane < ns ? bias[row_base + RR + warp + 8 * lane] : 0.f;
 #pragma unroll
-    for (int b = 0; b < NB; ++b) rres_r[b] = rres_s[b] = 0.f;
+    for (int b = 0; b < NB; ++b) { rres_r[b] = bias_r; rres_s[b] = bias_s; }
     if (R != nullptr) {
         if (lane < RPW && warp + 8 * lane < nrows) {
 #pragma unroll
             for (int b = 0; b < NB; ++b)
-                if (b < nb) rres_r[b] = R[(size_t)b * ldd + row_base + warp + 8 * lane];
+                if (b < nb) rres_r[b] += R[(size_t)b * ldd + row_base + warp + 8 * lane];
         }
         if (lane < GR && warp + 8 * lane < ns) {
 #pragma unroll
             for (int b = 0; b < NB; ++b)
-                if (b < nb) rres_s[b] = R[(size_t)b * ldd + row_base + RR + warp + 8 * lane];
+                if (b < nb) rres_s[b] += R[(size_t)b * ldd + row_base + RR + warp + 8 * lane];
         }
     }
 
@@ -550,7 +566,7 @@ __global__ void __launch_bounds__(256, 2) gemv_pre_kernel(const float* A, int ld
                 s2 = fmaf(xr[i + 2], xr[i + 2], s2); s3 = fmaf(xr[i + 3], xr[i + 3], s3);
             }
             const float tot = warp_sum(__fadd_rn(__fadd_rn(s0, s1), __fadd_rn(s2, s3)));
-            const float rs = rms_scale(tot, K, eps);
+            const float rs = rms_scale(tot, norm_width, eps);
 #pragma unroll
             for (int u = 0; u < U; ++u) {
                 const int c = lane + 32 * u;
@@ -616,7 +632,7 @@ __global__ void __launch_bounds__(256, 2) gemv_pre_kernel(const float* A, int ld
                     float t = 0.f;
 #pragma unroll
                     for (int w = 0; w < 8; ++w) t += nred[b][w];
-                    const float r = rms_scale(t, K, eps);
+                    const float r = rms_scale(t, norm_width, eps);
 #pragma unroll
                     for (int i = 0; i < GN; ++i) {
                         const int k = threadIdx.x + 256 * i;
@@ -675,7 +691,7 @@ __global__ void __launch_bounds__(256, 2) gemv_pre_kernel(const float* A, int ld
                 for (int b = 0; b < NB; ++b)
                     if (b < nb) {
                         float v = acc[r][0][b];
-                        if (R != nullptr) v = __fadd_rn(v, rres_r[b]);
+                        if (has_add) v = __fadd_rn(v, rres_r[b]);
                         D[(size_t)b * ldd + row_base + warp + 8 * r] = v;
                     }
             }
@@ -686,11 +702,11 @@ __global__ void __launch_bounds__(256, 2) gemv_pre_kernel(const float* A, int ld
     for (int j0 = warp; j0 < ns && !timed_out; j0 += 8 * GR) {
         if (j0 != warp) {            // later groups (rare): their residuals are fetched here
 #pragma unroll
-            for (int b = 0; b < NB; ++b) rres_s[b] = 0.f;
+            for (int b = 0; b < NB; ++b) rres_s[b] = bias != nullptr && lane < GR && j0 + 8 * lane < ns ? bias[row_base + RR + j0 + 8 * lane] : 0.f;
             if (R != nullptr && lane < GR && j0 + 8 * lane < ns) {
 #pragma unroll
                 for (int b = 0; b < NB; ++b)
-                    if (b < nb) rres_s[b] = R[(size_t)b * ldd + row_base + RR + j0 + 8 * lane];
+                    if (b < nb) rres_s[b] += R[(size_t)b * ldd + row_base + RR + j0 + 8 * lane];
             }
         }
         if (j0 == warp) {
@@ -740,7 +756,7 @@ __global__ void __launch_bounds__(256, 2) gemv_pre_kernel(const float* A, int ld
                     for (int b = 0; b < NB; ++b)
                         if (b < nb) {
                             float v = acc[g][0][b];
-                            if (R != nullptr) v = __fadd_rn(v, rres_s[b]);
+                            if (has_add) v = __fadd_rn(v, rres_s[b]);
                             D[(size_t)b * ldd + row_base + RR + j0 + 8 * g] = v;
                         }
                 }
@@ -1414,7 +1430,7 @@ static cudaError_t gemv_launch(const GemvArgs& a, int KS, cudaStream_t st) {
         if (a.amax_parts != nullptr) *a.amax_parts = (int)grid.x;
     }
     return launch_k(kern, grid, dim3(256), smem, st, a.A, a.lda, (const WT*)a.W, a.D, a.ldd, a.R, a.gamma, a.M, a.N, a.K, a.eps, KS,
-                    a.amax_val, a.amax_idx, a.amax_stride, a.post);
+                    a.amax_val, a.amax_idx, a.amax_stride, a.post, a.norm_width > 0 ? a.norm_width : a.K, a.bias);
 }
 
 template <typename WT, int NB, int ACT>
@@ -1434,12 +1450,22 @@ static cudaError_t gemv_by_batch(const GemvArgs& a, cudaStream_t st) {
     if (a.M > 1 && (size_t)a.K * sizeof(float) * (a.M > 4 ? 8 : 4) > 200 * 1024) {      // the staged rows have to fit: fewer of them per CTA
         if (a.act == 1) return gemv_dispatch<WT, 1, 1>(a, st);
         if (a.act == 2) return gemv_dispatch<WT, 1, 2>(a, st);
+        if (a.act == ACT_RELU_GATE) return gemv_dispatch<WT, 1, 3>(a, st);
+        if (a.act == ACT_SILU_GATE) return gemv_dispatch<WT, 1, 4>(a, st);
         return gemv_dispatch<WT, 1, 0>(a, st);
     }
     if (a.act == 1) {
         if (a.M <= 1) return gemv_dispatch<WT, 1, 1>(a, st);
         if (a.M <= 2) return gemv_dispatch<WT, 2, 1>(a, st);
         return gemv_dispatch<WT, 4, 1>(a, st);
+    }
+    if (a.act == ACT_RELU_GATE) {
+        if (a.M <= 1) return gemv_dispatch<WT, 1, 3>(a, st);
+        return gemv_dispatch<WT, 4, 3>(a, st);
+    }
+    if (a.act == ACT_SILU_GATE) {
+        if (a.M <= 1) return gemv_dispatch<WT, 1, 4>(a, st);
+        return gemv_dispatch<WT, 4, 4>(a, st);
     }
     if (a.act == 2) {
         if (a.M <= 1) return gemv_dispatch<WT, 1, 2>(a, st);
@@ -1503,7 +1529,8 @@ static cudaError_t gemv_pre_launch(const GemvArgs& a, int rows_per_cta, size_t s
     }
     dim3 grid((a.N + rows_per_cta - 1) / rows_per_cta);
     return launch_k(kern, grid, dim3(256), smem, st, a.A, a.lda, (const WT*)a.W, a.D, a.ldd, a.R, a.gamma, a.M, a.N, a.K, a.eps,
-                    rows_per_cta, gemv_pre_pace_ns(), smem > 64 * 1024 ? gemv_pre_delay_ns() : 0, a.status, a.post);
+                    rows_per_cta, gemv_pre_pace_ns(), smem > 64 * 1024 ? gemv_pre_delay_ns() : 0, a.status, a.post,
+                    a.norm_width > 0 ? a.norm_width : a.K, a.bias);
 }
 
 // Returns true (and the launch result in *err) when the product was given to the preloading kernel.

@@ -24,24 +24,31 @@ constexpr int kPadRow = 8;                                // extra bf16 per stag
 constexpr float kLog2e = 1.4426950408889634f;
 
 struct WinShape {
-    int ring, hpk, page_elems, v_off;                     // page_elems: elements per page; v_off: from a head's K block to its V block
+    int ring, hpk, head_step, k_ld, v_ld, v_off;          // as in WinAttnArgs
+    size_t page_elems;
 };
 __host__ __device__ inline WinShape shape_of(const WinAttnArgs& a) {
     WinShape s;
     s.ring = a.pages_per_seq * kPageTokens;
     s.hpk = a.H / a.G;
-    s.v_off = kPageTokens * a.dk_pad;
-    s.page_elems = a.G * kPageTokens * (a.dk_pad + a.dv_pad);
+    if (a.page_elems > 0) {
+        s.head_step = a.head_step; s.k_ld = a.k_ld; s.v_ld = a.v_ld; s.v_off = a.v_off;
+        s.page_elems = (size_t)a.page_elems;
+    } else {
+        s.head_step = kPageTokens * (a.dk_pad + a.dv_pad);
+        s.k_ld = a.dk_pad; s.v_ld = a.dv_pad; s.v_off = kPageTokens * a.dk_pad;
+        s.page_elems = (size_t)a.G * s.head_step;
+    }
     return s;
 }
 // element index of the K row of position p (kv head kvh); the V row of it starts at v_row()
 __device__ __forceinline__ size_t k_row(const WinAttnArgs& a, const WinShape& s, const int32_t* pt, int kvh, int p) {
     const int rs = p % s.ring;
-    return (size_t)pt[rs / kPageTokens] * s.page_elems + (size_t)kvh * kPageTokens * (a.dk_pad + a.dv_pad) + (size_t)(rs % kPageTokens) * a.dk_pad;
+    return (size_t)pt[rs / kPageTokens] * s.page_elems + (size_t)kvh * s.head_step + (size_t)(rs % kPageTokens) * s.k_ld;
 }
 __device__ __forceinline__ size_t v_row(const WinAttnArgs& a, const WinShape& s, const int32_t* pt, int kvh, int p) {
     const int rs = p % s.ring;
-    return (size_t)pt[rs / kPageTokens] * s.page_elems + (size_t)kvh * kPageTokens * (a.dk_pad + a.dv_pad) + s.v_off + (size_t)(rs % kPageTokens) * a.dv_pad;
+    return (size_t)pt[rs / kPageTokens] * s.page_elems + (size_t)kvh * s.head_step + s.v_off + (size_t)(rs % kPageTokens) * s.v_ld;
 }
 template <typename T> __device__ __forceinline__ T cache_elem(float v);
 template <> __device__ __forceinline__ float cache_elem<float>(float v) { return v; }
@@ -142,7 +149,10 @@ __global__ void __launch_bounds__(128) win_simple_kernel(WinAttnArgs a) {
         l = fmaf(l, f, (red[0] + red[1]) + (red[2] + red[3]));
         __syncthreads();
     }
-    for (int c = tid; c < a.dv; c += 128) put_row(a.y32, a.yhi, a.ylo, out + c, __fdiv_rn(cx[c], l));
+    for (int c = tid; c < a.dv; c += 128) {
+        const float v = __fdiv_rn(cx[c], l);
+        put_row(a.y32, a.yhi, a.ylo, out + c, a.gate != nullptr ? v * sigmoid_f(a.gate[(size_t)row * a.ldg + (size_t)h * a.dv + c]) : v);
+    }
 }
 
 // ---- tensor cores ----------------------------------------------------------------------------------------
@@ -232,17 +242,17 @@ __global__ void __launch_bounds__(128, NT <= 8 ? 4 : (NT <= 16 ? 3 : 2)) win_mma
         __nv_bfloat16* ks = stage + ((pg - pb) % kWinStages) * stage_elems;
         __nv_bfloat16* vs = ks + kPageTokens * KS;
         const int pidx = pt[pg % a.pages_per_seq];
-        const __nv_bfloat16* kp = pool + (size_t)pidx * s.page_elems + (size_t)kvh * kPageTokens * (DKP + DVP);
+        const __nv_bfloat16* kp = pool + (size_t)pidx * s.page_elems + (size_t)kvh * s.head_step;
         const __nv_bfloat16* vp = kp + s.v_off;
         for (int r = kr0, c = kc0; r < kPageTokens;) {
             const int p = pg * kPageTokens + r;
-            cp16b(ks + r * KS + c * 8, kp + r * DKP + c * 8, p >= lo && p <= hi && p != local);
+            cp16b(ks + r * KS + c * 8, kp + (size_t)r * s.k_ld + c * 8, p >= lo && p <= hi && p != local);
             r += kdr; c += kdc;
             if (c >= kc) { c -= kc; ++r; }
         }
         for (int r = vr0, c = vc0; r < kPageTokens;) {
             const int p = pg * kPageTokens + r;
-            cp16b(vs + r * VS + c * 8, vp + r * DVP + c * 8, p >= lo && p <= hi && p != local);
+            cp16b(vs + r * VS + c * 8, vp + (size_t)r * s.v_ld + c * 8, p >= lo && p <= hi && p != local);
             r += vdr; c += vdc;
             if (c >= vc) { c -= vc; ++r; }
         }
@@ -429,6 +439,7 @@ __global__ void __launch_bounds__(128, NT <= 8 ? 4 : (NT <= 16 ? 3 : 2)) win_mma
         ls[c] += __shfl_xor_sync(0xffffffffu, ls[c], 2);
     }
     auto emit = [&](int rr, int hh, int d, float v) {
+        if (a.gate != nullptr) v *= sigmoid_f(a.gate[(size_t)(sl * a.ts + i0 + rr) * a.ldg + (size_t)(kvh * s.hpk + h0 + hh) * a.dv + d]);
         put_row(a.y32, a.yhi, a.ylo, (size_t)(sl * a.ts + i0 + rr) * a.ldy + (size_t)(kvh * s.hpk + h0 + hh) * a.dv + d, v);
     };
     if constexpr (!DECODE) {
@@ -439,10 +450,15 @@ __global__ void __launch_bounds__(128, NT <= 8 ? 4 : (NT <= 16 ? 3 : 2)) win_mma
             const float inv = __frcp_rn(ls[c] + (a.m.sink ? exp2f(a.m.sink_score * kLog2e - mx[c]) : 0.f));
             const size_t oo = (size_t)(sl * a.ts + i0 + rr) * a.ldy + (size_t)(kvh * s.hpk + h0 + hh) * a.dv;
             const bool pairs = ((a.dv | a.ldy) & 1) == 0;
+            const float* gt = a.gate != nullptr ? a.gate + (size_t)(sl * a.ts + i0 + rr) * a.ldg + (size_t)(kvh * s.hpk + h0 + hh) * a.dv : nullptr;
 #pragma unroll
             for (int i = 0; i < NT; ++i) {
                 const int d = i * 8 + 2 * tq;
-                const float v0 = o[i][2 * c] * inv, v1 = o[i][2 * c + 1] * inv;
+                float v0 = o[i][2 * c] * inv, v1 = o[i][2 * c + 1] * inv;
+                if (pairs && gt != nullptr && d < a.dv) {
+                    v0 *= __frcp_rn(1.0f + __expf(-gt[d]));
+                    v1 *= __frcp_rn(1.0f + __expf(-gt[d + 1]));
+                }
                 if (pairs && d < a.dv) {
                     if (a.y32 != nullptr) *reinterpret_cast<float2*>(a.y32 + oo + d) = make_float2(v0, v1);
                     if (a.yhi != nullptr) {
@@ -525,21 +541,6 @@ __global__ void __launch_bounds__(128, NT <= 8 ? 4 : (NT <= 16 ? 3 : 2)) win_mma
     }
 }
 
-template <typename... KArgs, typename... Args>
-cudaError_t launch_dep(void (*kern)(KArgs...), dim3 grid, int threads, size_t smem, cudaStream_t st, Args... args) {
-    cudaLaunchConfig_t cfg = {};
-    cfg.gridDim = grid;
-    cfg.blockDim = dim3(threads);
-    cfg.dynamicSmemBytes = smem;
-    cfg.stream = st;
-    cudaLaunchAttribute attr[1];
-    attr[0].id = cudaLaunchAttributeProgrammaticStreamSerialization;
-    attr[0].val.programmaticStreamSerializationAllowed = 1;
-    cfg.attrs = attr;
-    cfg.numAttrs = launch_pdl_on() ? 1 : 0;
-    return cudaLaunchKernelEx(&cfg, kern, KArgs(args)...);
-}
-
 constexpr size_t kSmemMax = 227 * 1024 - 1024;
 int head_block(const MixerSpec& m) {                      // heads of a group that one CTA serves
     const int hpk = m.heads / m.kv_heads, subs = (hpk + 15) / 16;
@@ -568,19 +569,19 @@ cudaError_t launch_mma(const WinAttnArgs& a, cudaStream_t st) {
         auto kern = win_mma_kernel<NT, NK, true>;
         cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
         if (e != cudaSuccess) return e;
-        return launch_dep(kern, dim3(a.nseq, a.G * subs, nsplit), 128, smem, st, a, hb, 1, 1);
+        return launch_rows(kern, dim3(a.nseq, a.G * subs, nsplit), 128, smem, st, a, hb, 1, 1);
     }
     const int q_rows = 16 / hb, gps = (a.ts + 4 * q_rows - 1) / (4 * q_rows);
     auto kern = win_mma_kernel<NT, NK, false>;
     cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     if (e != cudaSuccess) return e;
-    return launch_dep(kern, dim3((unsigned)a.nseq * gps, a.G * subs, 1), 128, smem, st, a, hb, q_rows, gps);
+    return launch_rows(kern, dim3((unsigned)a.nseq * gps, a.G * subs, 1), 128, smem, st, a, hb, q_rows, gps);
 }
 
 template <typename KT>
 cudaError_t append(const WinAttnArgs& a, cudaStream_t st) {
     const long warps = (long)a.nseq * a.ts * a.G;
-    return launch_dep(win_append_kernel<KT>, dim3((unsigned)((warps + 7) / 8)), 256, 0, st, a);
+    return launch_rows(win_append_kernel<KT>, dim3((unsigned)((warps + 7) / 8)), 256, 0, st, a);
 }
 template <typename KT>
 cudaError_t simple(const WinAttnArgs& a, cudaStream_t st) {
@@ -591,7 +592,7 @@ cudaError_t simple(const WinAttnArgs& a, cudaStream_t st) {
         const cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
         if (e != cudaSuccess) return e;
     }
-    return launch_dep(kern, dim3((unsigned)(a.nseq * a.ts), a.H), 128, smem, st, a);
+    return launch_rows(kern, dim3((unsigned)(a.nseq * a.ts), a.H), 128, smem, st, a);
 }
 
 }  // namespace
@@ -600,7 +601,7 @@ size_t window_attention_part_floats(const MixerSpec& m) { return (size_t)kWinSli
 
 cudaError_t launch_window_attention(const WinAttnArgs& a, cudaStream_t st, int* launches) {
     *launches = 0;
-    const bool mma = !a.kv_is_f32 && a.dk_pad <= kMmaDim && a.dv_pad <= 256 && mma_smem(a, a.ts == 1) <= kSmemMax;
+    const bool mma = !a.kv_is_f32 && !a.plain && a.dk_pad <= kMmaDim && a.dv_pad <= 256 && mma_smem(a, a.ts == 1) <= kSmemMax;
     cudaError_t e;
     if (a.append && !(mma && a.ts == 1)) {
         e = a.kv_is_f32 ? append<float>(a, st) : append<__nv_bfloat16>(a, st);
@@ -614,6 +615,7 @@ cudaError_t launch_window_attention(const WinAttnArgs& a, cudaStream_t st, int* 
     if (nt == 8 && nk == 4) return launch_mma<8, 4>(a, st);
     if (nt == 12 && nk == 6) return launch_mma<12, 6>(a, st);
     if (nt == 16 && nk == 8) return launch_mma<16, 8>(a, st);
+    if (nt == 16 && nk == 12) return launch_mma<16, 12>(a, st);
     if (nt <= 4) return launch_mma<4, 0>(a, st);
     if (nt <= 8) return launch_mma<8, 0>(a, st);
     if (nt <= 12) return launch_mma<12, 0>(a, st);

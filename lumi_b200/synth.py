@@ -254,10 +254,12 @@ BENCH_CONFIGS = {
 
 def config_from_json(text: str):
     """The configuration class a config.json asks for: registered designs by their "architecture", else ModelConfig."""
-    from . import zozonex
+    from . import zozonex, zutazen
     name = json.loads(text).get("architecture")
     if name is None:
         return ModelConfig.from_json(text)
     if name == zozonex.ARCHITECTURE:
         return zozonex.ZozonexConfig.from_json(text)
+    if name == zutazen.ARCHITECTURE:
+        return zutazen.ZutazenConfig.from_json(text)
     raise ValueError(f"architecture {name!r} is not known")
