@@ -1448,6 +1448,7 @@ int32_t norm_product(StepPlan& p, RowPass& r, const DevTensor& W, const float* g
     GemmExt ex;
     if (act != 0) {
         ex.group_rows = N; ex.lda = K; ex.out_n = ex.out_step = N / 2; ex.gate = act; ex.ldo = N / 2;
+        g.d = nullptr;                                    // halves only
         g.nf.out_hi = out_hi;
         g.nf.out_lo = s->opt_split ? out_lo : nullptr;
         g.ext = &ex;
