@@ -181,7 +181,10 @@ def forward(cfg, W, tokens, dtype=np.float64):
     x = W["embed"][np.asarray(tokens)] * cfg["embedding"]["scale"]
     stream = []
     for i, L in enumerate(cfg["layers"]):
-        p = "l%d." % L.get("weights_of", i)
+        own = i
+        while "weights_of" in cfg["layers"][own]:
+            own = cfg["layers"][own]["weights_of"]
+        p = "l%d." % own
         h = rms(x, eps) * W[p + "norm1"]
         if L["type"] == "retention":
             x = x + retention_mixer(W, p + "mix.", L["mixer"], h, eps)
