@@ -308,9 +308,35 @@ def zozonex_pair(name):
     return (zcfg, zz.iter_tensors(zcfg, seed=0)), (hcfg, synth.iter_tensors(hcfg, seed=0, weights_dtype="bf16"))
 
 
-def run_zozonex(args, rank, local_rank, world):
-    """Prefill and decode throughput of the Zozonex design beside the Mamba-3 / attention hybrid of equal size: CUDA events inside
-    the library, random weights, greedy decode; device times by kernel family from one profiled step."""
+# --workload zutazen: (width, layers, (retention heads, dim), (recurrence blocks), (latent attention heads, dim, rotated, vdim, rank),
+# window, dense ff, (experts, top, expert ff), Zozonex: delta heads / dim / vdim, attention heads / kv heads / dim).  Layers go retention
+# (dense), gated recurrence (experts), retention, gated recurrence (dense), retention, latent attention; the Zozonex model beside it has
+# the same width, depth, state bytes per matrix-state layer, window and active feed-forward parameters per layer.
+ZUTAZEN_SIZES = {
+    "w1024": (1024, 12, (8, 128), 8, (16, 64, 32, 64, 256), 1024, 2816, (16, 2, 1408), (16, 64, 128), (16, 4, 64)),
+    "w2048": (2048, 6, (16, 128), 16, (16, 128, 64, 128, 512), 1024, 5632, (32, 4, 1408), (16, 128, 128), (32, 8, 64)),
+}
+
+
+def zutazen_pair(name):
+    """(Zutazen config and tensors, Zozonex config and tensors) of one size; bf16 weights."""
+    from lumi_b200 import zozonex as zz, zutazen as zt
+    width, n, (rh, rd), blocks, (lh, ld, lr, lv, rank), window, ff, experts, (dh, dk, dv), (ah, ag, ad) = ZUTAZEN_SIZES[name]
+    tl, zl = [], []
+    for i in range(n):
+        dense = zt.dense(ff)
+        tl.append([zt.retention(rh, rd, rd, mlp=dense), zt.rglru(width, blocks, mlp=zt.moe(*experts)), zt.retention(rh, rd, rd, mlp=dense),
+                   zt.rglru(width, blocks, mlp=dense), zt.retention(rh, rd, rd, mlp=dense),
+                   zt.latent_attention(lh, ld, lr, lv, rank, window, mlp=dense)][i % 6])
+        zl.append(zz.delta(dh, dk, dv, ff=3 * ff // 2) if (i + 1) % 6 else zz.attention(ah, ad, window, kv_heads=ag, ff=3 * ff // 2))
+    tcfg = zt.config(width, ZOZONEX_VOCAB, tl, max_seq_len=8192)
+    zcfg = zz.config(width, ZOZONEX_VOCAB, zl, max_seq_len=8192)
+    return (tcfg, zt.iter_tensors(tcfg, seed=0)), (zcfg, zz.iter_tensors(zcfg, seed=0))
+
+
+def run_designs(args, rank, local_rank, kinds, sizes, pair):
+    """Prefill and decode throughput of one design beside another of equal size: CUDA events inside the library, random weights, greedy
+    decode; device times by kernel family from one profiled step."""
     if rank != 0:
         return
     import lumi_b200
@@ -318,13 +344,15 @@ def run_zozonex(args, rank, local_rank, world):
     out = []
     sampler = ClockSampler(local_rank)
     sampler.start()
-    for name in (args.zozonex_sizes.split(",") if args.zozonex_sizes else ZOZONEX_SIZES):
+    for name in (args.sizes.split(",") if args.sizes else sizes):
         entry = {"size": name}
-        for kind, (cfg, tens) in zip(("zozonex", "hybrid"), zozonex_pair(name)):
+        for kind, (cfg, tens) in zip(kinds, pair(name)):
+            if args.only_design and kind != args.only_design:
+                continue
             model = lumi_b200.NmModel.from_tensors(cfg, tens, device=local_rank)
             runs = {"weight_bytes": model.info()["weight_bytes"]}
             for batch, T in ((1, 2048), (16, 2048), (64, 512), (512, 128)):
-                if args.zozonex_batch and batch != args.zozonex_batch:
+                if args.batch and batch != args.batch:
                     continue
                 sess = model.init_states(batch, T + 256)
                 prompts = synth.random_prompts(batch, T, cfg.vocab_size, seed=1)
@@ -350,10 +378,11 @@ def run_zozonex(args, rank, local_rank, world):
             entry[kind] = runs
         out.append(entry)
     clocks = sampler.stop()
-    big = out[-1]["zozonex"][list(out[-1]["zozonex"])[-1]]
+    last = out[-1][list(out[-1])[1]]
+    big = last[list(last)[-1]]
     print(json.dumps({"metric": METRIC, "value": big["decode_tok_s"], "unit": UNIT, "n_gpus": 1, "steps": args.steps, "warmup": 3,
                       "ms_per_step": big["decode_ms_per_step"], "higher_is_better": True, "scaling": "strong", "vs_baseline": None, "dtype": "bf16",
-                      "data": "synthetic", "config": {"workload": "zozonex: decode and prefill beside the hybrid of equal size", "peak_gbs": peak_gbs,
+                      "data": "synthetic", "config": {"workload": "%s: decode and prefill beside the %s of equal size" % tuple(kinds), "peak_gbs": peak_gbs,
                                                       "peak_source": peak_src}, "sizes": out, "clocks": clocks}), flush=True)
 
 
@@ -561,9 +590,10 @@ def main():
     ap.add_argument("--no-batch1", action="store_true")
     ap.add_argument("--only-batch1", action="store_true", help="run just the batch-1 figure (profiling)")
     ap.add_argument("--b1-layers", type=int, default=48)
-    ap.add_argument("--workload", default="sweep", choices=["sweep", "scan", "zozonex"] + sorted(CONFIGS))
-    ap.add_argument("--zozonex-sizes", default="", help="--workload zozonex: only these sizes (commas between them)")
-    ap.add_argument("--zozonex-batch", type=int, default=0, help="--workload zozonex: only this batch")
+    ap.add_argument("--workload", default="sweep", choices=["sweep", "scan", "zozonex", "zutazen"] + sorted(CONFIGS))
+    ap.add_argument("--sizes", "--zozonex-sizes", default="", help="--workload zozonex, zutazen: only these sizes (commas between them)")
+    ap.add_argument("--batch", "--zozonex-batch", type=int, default=0, help="--workload zozonex, zutazen: only this batch")
+    ap.add_argument("--only-design", default="", help="--workload zozonex, zutazen: only this one of the two designs")
     ap.add_argument("--scan-seqs", type=int, default=64, help="--workload scan: sequences")
     ap.add_argument("--scan-tokens", type=int, default=2048, help="--workload scan: tokens per sequence")
     ap.add_argument("--steps-override", type=int, default=0, help="decode tokens for --workload configN (0 = the configuration's own)")
@@ -577,7 +607,9 @@ def main():
             torch.cuda.set_device(local_rank)
             print(json.dumps({"prefill_scan": scan_compare(args.scan_seqs, args.scan_tokens)}), flush=True)
     elif args.workload == "zozonex":
-        run_zozonex(args, rank, local_rank, world)
+        run_designs(args, rank, local_rank, ("zozonex", "hybrid"), ZOZONEX_SIZES, zozonex_pair)
+    elif args.workload == "zutazen":
+        run_designs(args, rank, local_rank, ("zutazen", "zozonex"), ZUTAZEN_SIZES, zutazen_pair)
     elif args.workload != "sweep":
         run_named_config(args, rank, local_rank, world)
     elif args.only_batch1:

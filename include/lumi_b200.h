@@ -87,15 +87,15 @@ const char* lumi_last_error(void);
  * attn_rope_base) and binds the model to a device. */
 int32_t lumi_model_create(const char* config_json, int32_t device_id, lumi_model** out);
 
-/* Designs with an "architecture" key in their config.json (Zozonex: gated delta-rule and windowed attention layers listed one
- * by one) bring their own reader and tensor names; a config without it is the Mamba-3 / attention hybrid above.
+/* Designs with an "architecture" key in their config.json (layers listed one by one. Zozonex: gated delta rule and windowed
+ * attention; Zutazen: retention, gated linear recurrence, latent attention, experts) bring their own reader and tensor names; a config without it is the Mamba-3 / attention hybrid above.
  *
  * Model options, set before the first tensor: "widen_weights" = 1 keeps every bf16 tensor as fp32 on the device, which makes
  * the whole model run in fp32 (products, cache, states). */
 int32_t lumi_model_set_option(lumi_model* m, const char* name, int64_t value);
 
 /* One call per safetensors entry, name including the `item.` prefix (designs with a reader of their own: their own names).  dtype F32 or BF16; rank-2
- * tensors keep their stored width on the device, rank-1 tensors become fp32.  `ssm.h_init` may be
+ * (and rank-3) tensors keep their stored width on the device, rank-1 tensors become fp32.  `ssm.h_init` may be
  * rank 2 [n_heads, d_state] or rank 1 [n_heads * d_state]. */
 int32_t lumi_model_load_tensor(lumi_model* m, const char* name, int32_t dtype, const int64_t* shape,
                                int32_t rank, const void* host_data, uint64_t nbytes);
