@@ -1527,6 +1527,7 @@ int32_t retention_mixer(StepPlan& p, RowPass& r, const Layer& L, int li) {
     a.nseq = r.nseq; a.ts = r.ts; a.b0 = r.b0;
     a.y32 = p.tc ? nullptr : b.y32; a.yhi = p.tc ? b.ah : nullptr; a.ylo = p.tc && s->opt_split ? b.al : nullptr; a.ldy = (int)L.s.out.cols;
     a.o32 = b.mix;
+    a.status = &s->ctl->status;
     p.fam = FAM_SSM;
     mark(p);
     int n = 0;

@@ -681,6 +681,7 @@ struct RetentionArgs {
     int nseq, ts, b0;
     float* y32; __nv_bfloat16 *yhi, *ylo; int ldy;
     float* o32;                                      // chunked form: read-out before its norm, [rows][H][dvp]
+    int32_t* status;                                 // receives STATUS_TIMEOUT if a bounded wait gives up; may be null
 };
 cudaError_t launch_retention_step(const RetentionArgs& a, cudaStream_t st, int* launches);
 bool retention_chunk_supported(int dk, int dv);

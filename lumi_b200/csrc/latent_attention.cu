@@ -20,7 +20,7 @@ constexpr float kNoScore = -1.0e30f;
 constexpr float kLog2e = 1.4426950408889634f;
 constexpr int kPad = 8;                                   // extra bf16 per staged row: no ldmatrix conflicts
 constexpr int kSlices = 16;
-constexpr int kSliceMin = 256;                            // tokens from which a slice of the context is worth a CTA
+constexpr int kSliceMin = 128;                            // tokens from which a slice of the context is worth a CTA
 
 template <typename T> __device__ __forceinline__ T cache_elem(float v);
 template <> __device__ __forceinline__ float cache_elem<float>(float v) { return v; }
@@ -165,6 +165,7 @@ __global__ void __launch_bounds__(128) latent_mma_kernel(LatentArgs a) {
         asm volatile("cp.async.commit_group;" ::: "memory");
         const __nv_bfloat16* s = stage + ((pg - pb) & 1) * stage_elems;
         float sc[2][4] = {}, sl2[2][4] = {};              // products with the query's two halves
+#pragma unroll 4
         for (int k = 0; k < nks; ++k) {
             uint32_t fh[4], fl[4], kb[4];
             const int qo = (lane & 15) * RS + k * 16 + (lane >> 4) * 8;
@@ -292,18 +293,40 @@ __global__ void __launch_bounds__(128) latent_mma_kernel(LatentArgs a) {
     __syncthreads();
     if (!is_last) return;
     __threadfence();
+    // weights of the slices per head (an empty slice has maximum kNoScore and weighs nothing), then the contexts, all loads of an
+    // element's slices in flight together
     const float* all = a.part + unit * nsplit * pw;
-    for (int i = tid; i < nh * ls.lp; i += 128) {
-        const int m = i / ls.lp;
-        float top = kNoScore;
-        for (int sp = 0; sp < nsplit; ++sp) top = fmaxf(top, __ldcg(all + sp * pw + m));
-        float den = 0.f, num = 0.f;
-        for (int sp = 0; sp < nsplit; ++sp) {             // an empty slice has maximum kNoScore and weighs nothing
-            const float f = exp2f(__ldcg(all + sp * pw + m) - top);
-            den = fmaf(f, __ldcg(all + sp * pw + 16 + m), den);
-            num = fmaf(f, __ldcg(all + sp * pw + 32 + i), num);
+    float* wt = reinterpret_cast<float*>(smem_raw);       // [nsplit][16]
+    if (tid < 16) {
+        float top = kNoScore, mv[kSlices], sv[kSlices];
+#pragma unroll
+        for (int sp = 0; sp < kSlices; ++sp) {
+            mv[sp] = sp < nsplit ? __ldcg(all + sp * pw + tid) : kNoScore;
+            sv[sp] = sp < nsplit ? __ldcg(all + sp * pw + 16 + tid) : 0.f;
         }
-        put(m, i % ls.lp, __fdiv_rn(num, den));
+#pragma unroll
+        for (int sp = 0; sp < kSlices; ++sp) top = fmaxf(top, mv[sp]);
+        float den = 0.f;
+#pragma unroll
+        for (int sp = 0; sp < kSlices; ++sp) { mv[sp] = exp2f(mv[sp] - top); den = fmaf(mv[sp], sv[sp], den); }
+        const float inv = __frcp_rn(den);
+#pragma unroll
+        for (int sp = 0; sp < kSlices; ++sp) if (sp < nsplit) wt[sp * 16 + tid] = mv[sp] * inv;
+    }
+    __syncthreads();
+    for (int i = 4 * tid; i < nh * ls.lp; i += 4 * 128) {
+        const int m = i / ls.lp;
+        float4 v[kSlices];
+#pragma unroll
+        for (int sp = 0; sp < kSlices; ++sp) v[sp] = sp < nsplit ? __ldcg(reinterpret_cast<const float4*>(all + sp * pw + 32 + i)) : make_float4(0.f, 0.f, 0.f, 0.f);
+        float4 n = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll
+        for (int sp = 0; sp < kSlices; ++sp) {
+            const float f = sp < nsplit ? wt[sp * 16 + m] : 0.f;
+            n.x = fmaf(f, v[sp].x, n.x); n.y = fmaf(f, v[sp].y, n.y); n.z = fmaf(f, v[sp].z, n.z); n.w = fmaf(f, v[sp].w, n.w);
+        }
+        const int d = i % ls.lp;
+        put(m, d, n.x); put(m, d + 1, n.y); put(m, d + 2, n.z); put(m, d + 3, n.w);
     }
 }
 

@@ -4,7 +4,8 @@
 //
 // o over its root mean square, head by head, times silu of the gate rows.  Two forms of the recurrence:
 //
-//   retention_step_kernel    token after token, the head's state in registers: decode steps (rotation, state, read-out, norm and
+//   retention_step_kernel    token after token, the head's state in registers (few heads), or in shared memory in parts that are
+//                            loaded, worked on and stored one behind the other: decode steps (rotation, state, read-out, norm and
 //                            gate in one launch), prompts of fp32 models, short slices.
 //   retention_chunk_kernel   prompt slices in chunks of 64 tokens on the tensor cores.  With S_0 the state ahead of the chunk,
 //                            o_t = d^(t+1) S_0^T q_t + sum_{s <= t} d^(t-s) (q_t.k_s) v_s, and the state becomes
@@ -27,11 +28,33 @@ __device__ __forceinline__ float rotated(const float* x, int c, const RotSpec& r
     return second ? fmaf(a, cs.x, b * cs.y) : fmaf(a, cs.x, -b * cs.y);
 }
 
+__device__ __forceinline__ uint32_t smem_of(const void* p) { return (uint32_t)__cvta_generic_to_shared(p); }
+constexpr uint64_t kStateWaitNs = 500000000ull;           // limit of the wait for a part of a head's state
+// false if the phase did not complete within the limit
+__device__ __forceinline__ bool state_wait(uint64_t* bar) {
+    uint32_t done = 0, polls = 0;
+    uint64_t t0 = 0;
+    while (true) {
+        asm volatile("{\n.reg .pred p;\nmbarrier.try_wait.parity.shared::cta.b64 p, [%1], 0;\nselp.u32 %0, 1, 0, p;\n}" : "=r"(done) : "r"(smem_of(bar)) : "memory");
+        if (done) return true;
+        if ((++polls & 255u) == 0u) {
+            uint64_t now;
+            asm volatile("mov.u64 %0, %%globaltimer;" : "=l"(now));
+            if (t0 == 0) t0 = now;
+            else if (now - t0 > kStateWaitNs) return false;
+        }
+    }
+}
+
 // CTA = (head, sequence).  Thread (rg, cg) holds rows rg, rg + RG, ... (VPT of them at most) of four neighbouring columns.
-// VPT = 0: the state stays in global memory (heads beyond the registers).
+// VPT = 0: the state stays in global memory (heads beyond shared memory).  VPT = -1: the state lies in shared memory, in kParts parts of
+// `pr` rows (a multiple of RG) that bulk copies bring and take back: while one part is worked on, the others are on their way.
+constexpr int kParts = 4;
 template <int NT, int VPT>
-__global__ void __launch_bounds__(NT) retention_step_kernel(RetentionArgs a, int cwl) {
-    extern __shared__ float sm[];
+__global__ void __launch_bounds__(NT) retention_step_kernel(RetentionArgs a, int cwl, int part_rows) {
+    extern __shared__ __align__(128) float dyn[];
+    __shared__ __align__(8) uint64_t bars[kParts];
+    float* sm = dyn + (VPT < 0 ? (size_t)a.dk * a.dvp : 0);
     const int h = blockIdx.x, sl = blockIdx.y, slot = a.b0 + sl, tid = threadIdx.x, lane = tid & 31;
     const int dk = a.dk, dv = a.dv, dvp = a.dvp, c4n = dvp >> 2;
     const int CW = 1 << cwl, cg = tid & (CW - 1), rg = tid >> cwl, RG = NT >> cwl;
@@ -45,8 +68,23 @@ __global__ void __launch_bounds__(NT) retention_step_kernel(RetentionArgs a, int
     float* part = os + dvp;                               // [slots][dvp]
     float4* S = reinterpret_cast<float4*>(a.S + ((size_t)slot * a.H + h) * dk * dvp);
     const float d = a.decay_pow[(size_t)h * kDecayPowers + 1];
+    auto part_of = [&](int p, int& r0, int& n) { r0 = p * part_rows; n = max(0, min(part_rows, dk - r0)); };
+    auto request = [&]() {                                // thread 0
+        for (int p = 0; p < kParts; ++p) asm volatile("mbarrier.init.shared::cta.b64 [%0], 1;" ::"r"(smem_of(&bars[p])));
+        asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
+        for (int p = 0; p < kParts; ++p) {
+            int r0, n;
+            part_of(p, r0, n);
+            if (n == 0) break;
+            const uint32_t bytes = (uint32_t)n * dvp * 4u;
+            asm volatile("mbarrier.arrive.expect_tx.shared::cta.b64 _, [%0], %1;" ::"r"(smem_of(&bars[p])), "r"(bytes) : "memory");
+            asm volatile("cp.async.bulk.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1], %2, [%3];"
+                         ::"r"(smem_of(dyn + (size_t)r0 * dvp)), "l"(S + (size_t)r0 * c4n), "r"(bytes), "r"(smem_of(&bars[p])) : "memory");
+        }
+    };
     pdl_release();
     // the state belongs to the step before this one, which has ended: read ahead of the predecessor's results
+    if (VPT < 0 && a.row_len == nullptr && tid == 0) request();
     float4 s[VPT > 0 ? VPT : 1];
     if constexpr (VPT > 0) {
 #pragma unroll
@@ -58,7 +96,8 @@ __global__ void __launch_bounds__(NT) retention_step_kernel(RetentionArgs a, int
     const int pos0 = a.pos[slot];
     pdl_sync();
     const int n = pass_tokens(a.row_len, a.ctl, slot, a.ts, a.t_abs0);
-    if (n == 0 && a.ts == 1) return;
+    if (n == 0 && a.ts == 1) return;                      // (with VPT < 0 nothing has been requested then)
+    if (VPT < 0 && a.row_len != nullptr && n > 0 && tid == 0) request();
     for (int t = 0; t < n; ++t) {
         const int row = sl * a.ts + t;
         const float* pr = a.proj + (size_t)row * a.ldp;
@@ -69,7 +108,44 @@ __global__ void __launch_bounds__(NT) retention_step_kernel(RetentionArgs a, int
         for (int c = tid; c < dvp; c += NT) vs[c] = c < dv ? pr[a.off_v + h * dv + c] : 0.f;
         __syncthreads();
         float4 o = make_float4(0.f, 0.f, 0.f, 0.f);
-        if (act) {
+        if constexpr (VPT < 0) {
+            const float4 v = act ? make_float4(vs[4 * cg], vs[4 * cg + 1], vs[4 * cg + 2], vs[4 * cg + 3]) : make_float4(0.f, 0.f, 0.f, 0.f);
+            float4* St = reinterpret_cast<float4*>(dyn);
+            for (int p = 0; p < kParts; ++p) {
+                int r0, cnt;
+                part_of(p, r0, cnt);
+                if (cnt == 0) break;
+                if (t == 0 && __syncthreads_or(!state_wait(&bars[p]))) {
+                    // report, and let what is still on its way land (again with a limit) before the memory goes away
+                    if (tid == 0) {
+                        if (a.status != nullptr) atomicOr(a.status, STATUS_TIMEOUT);
+                        for (int q = p; q < kParts; ++q) { part_of(q, r0, cnt); if (cnt > 0) state_wait(&bars[q]); }
+                        asm volatile("cp.async.bulk.wait_group.read 0;" ::: "memory");
+                    }
+                    __syncthreads();
+                    return;
+                }
+                if (act) {
+#pragma unroll 4
+                    for (int r = r0 + rg; r < r0 + cnt; r += RG) {
+                        float4 x = St[(size_t)r * c4n + cg];
+                        const float k = ks[r], q = qs[r];
+                        x = make_float4(fmaf(k, v.x, d * x.x), fmaf(k, v.y, d * x.y), fmaf(k, v.z, d * x.z), fmaf(k, v.w, d * x.w));
+                        o.x = fmaf(q, x.x, o.x); o.y = fmaf(q, x.y, o.y); o.z = fmaf(q, x.z, o.z); o.w = fmaf(q, x.w, o.w);
+                        St[(size_t)r * c4n + cg] = x;
+                    }
+                }
+                if (t + 1 == n) {                         // the part goes back
+                    asm volatile("fence.proxy.async.shared::cta;" ::: "memory");
+                    __syncthreads();
+                    if (tid == 0) {
+                        asm volatile("cp.async.bulk.global.shared::cta.bulk_group [%0], [%1], %2;"
+                                     ::"l"(S + (size_t)r0 * c4n), "r"(smem_of(dyn + (size_t)r0 * dvp)), "r"((uint32_t)cnt * dvp * 4u) : "memory");
+                        asm volatile("cp.async.bulk.commit_group;" ::: "memory");
+                    }
+                }
+            }
+        } else if (act) {
             const float4 v = make_float4(vs[4 * cg], vs[4 * cg + 1], vs[4 * cg + 2], vs[4 * cg + 3]);
             auto walk = [&](int r, float4& x) {
                 const float k = ks[r], q = qs[r];
@@ -117,6 +193,8 @@ __global__ void __launch_bounds__(NT) retention_step_kernel(RetentionArgs a, int
             }
         }
     }
+    // the memory of the CTA has been read; the writes themselves end with the kernel
+    if (VPT < 0 && tid == 0) asm volatile("cp.async.bulk.wait_group.read 0;" ::: "memory");
 }
 
 // ---- chunks of 64 tokens -----------------------------------------------------------------------------------
@@ -308,14 +386,15 @@ constexpr size_t kSmemMax = 227 * 1024 - 1024;
 template <int NT, int VPT>
 cudaError_t step_launch(const RetentionArgs& a, int cwl, cudaStream_t st) {
     const int share = (1 << cwl) < 32 ? 32 : (1 << cwl);
-    const size_t smem = sizeof(float) * (2 * (size_t)((a.dk + 3) & ~3) + (2 + (size_t)(NT / share)) * a.dvp);
+    const size_t smem = sizeof(float) * (2 * (size_t)((a.dk + 3) & ~3) + (2 + (size_t)(NT / share)) * a.dvp + (VPT < 0 ? (size_t)a.dk * a.dvp : 0));
     if (smem > kSmemMax) return cudaErrorInvalidValue;
     auto kern = retention_step_kernel<NT, VPT>;
     if (smem > 48 * 1024) {
         const cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
         if (e != cudaSuccess) return e;
     }
-    return launch_rows(kern, dim3(a.H, a.nseq), NT, smem, st, a, cwl);
+    const int RG = NT >> cwl, part_rows = ((a.dk + kParts - 1) / kParts + RG - 1) / RG * RG;
+    return launch_rows(kern, dim3(a.H, a.nseq), NT, smem, st, a, cwl, part_rows);
 }
 
 // columns per CTA (nw warp pairs of 8 ntw each): as many as the value dimension has and shared memory takes, fewer where the heads
@@ -343,6 +422,11 @@ cudaError_t launch_retention_step(const RetentionArgs& a, cudaStream_t st, int* 
     while ((4 << cwl) < a.dvp) ++cwl;
     const int CW = 1 << cwl;
     if (CW > 256) return cudaErrorInvalidValue;
+    // many heads: through shared memory, several CTAs per SM; few: straight into registers
+    if ((long)a.nseq * a.H > 296 && CW <= 64 && (size_t)a.dk * a.dvp * 4 <= 100 * 1024) {
+        if ((size_t)a.dk * a.dvp <= 4096 && CW <= 32) return step_launch<128, -1>(a, cwl, st);
+        return step_launch<256, -1>(a, cwl, st);
+    }
     auto per_thread = [&](int nt) { return nt >= CW ? (a.dk + nt / CW - 1) / (nt / CW) : 1 << 30; };
     if (per_thread(128) <= 4) return step_launch<128, 4>(a, cwl, st);
     if (per_thread(128) <= 8) return step_launch<128, 8>(a, cwl, st);

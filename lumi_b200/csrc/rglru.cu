@@ -17,14 +17,21 @@
 namespace lumi {
 namespace {
 
+// sigma(x) with the hardware exponential (relative error of a few 1e-7)
+__device__ __forceinline__ float sigmoid_q(float x) { return __fdividef(1.0f, 1.0f + __expf(-x)); }
+// z / 2 (1 + tanh(w)) = z sigma(2 w); far out the exponential overflows to an exact 0
 __device__ __forceinline__ float gelu_tanh_f(float z) {
-    return 0.5f * z * (1.0f + tanhf(0.7978845608028654f * (z + 0.044715f * z * z * z)));
+    const float w2 = 1.5957691216057308f * (z + 0.044715f * z * z * z);
+    return w2 < -80.f ? 0.f : z * sigmoid_q(w2);
 }
 // decay a and the factor sqrt(1 - a^2) of the input, from the decay gate's logit
 __device__ __forceinline__ void decay_of(float r_logit, float sp_rate, float& a, float& b) {
-    const float la = -sp_rate * sigmoid_f(r_logit);       // sp_rate = rate * softplus(lam)
+    const float la = -sp_rate * sigmoid_q(fmaxf(r_logit, -80.f));       // sp_rate = rate * softplus(lam)
     a = expf(la);
-    b = sqrtf(-expm1f(2.0f * la));
+    // 1 - e^x, x = 2 log a: where x is small by its series (no cancellation), else from a
+    const float x = 2.0f * la;
+    const float series = -x * fmaf(x, fmaf(x, fmaf(x, fmaf(x, fmaf(x, 1.f / 720.f, 1.f / 120.f), 1.f / 24.f), 1.f / 6.f), 0.5f), 1.0f);
+    b = __fsqrt_rn(x > -0.25f ? series : fmaf(-a, a, 1.0f));
 }
 
 // Convolution input of channel c, d tokens before token t of the pass (d > t: from the ring; none before position 0).
@@ -106,7 +113,7 @@ __global__ void __launch_bounds__(1024) rglru_scan_kernel(RglruArgs a) {
                 const float* gt = a.gates + (row0 + k) * grow + gr;
                 float f;
                 decay_of(gt[0], sp, da[k], f);
-                in[k] = f * sigmoid_f(gt[16]) * a.u32[(row0 + k) * a.channels + c];
+                in[k] = f * sigmoid_q(fmaxf(gt[16], -80.f)) * a.u32[(row0 + k) * a.channels + c];
             }
         }
         float p = 1.f, e = 0.f;
@@ -228,7 +235,7 @@ __global__ void __launch_bounds__(256) rglru_step_kernel(RglruArgs a, int per, i
         float d, f;
         decay_of(gt[0], a.rate * softplus_f(a.lam[c]), d, f);
         float* Sp = a.S + (size_t)slot * a.channels + c;
-        const float s = fmaf(d, *Sp, f * sigmoid_f(gt[16]) * us[r * a.bp + i]);
+        const float s = fmaf(d, *Sp, f * sigmoid_q(fmaxf(gt[16], -80.f)) * us[r * a.bp + i]);
         *Sp = s;
         // this token's convolution input for later ones (no CTA reads the slot of its own position)
         a.conv[((size_t)slot * a.taps + a.pos[slot] % a.taps) * a.channels + c] = a.proj[(size_t)sl * a.ldp + a.off_x + c];

@@ -613,6 +613,7 @@ cudaError_t launch_window_attention(const WinAttnArgs& a, cudaStream_t st, int* 
     const int nt = a.dv_pad / 8, nk = a.dk_pad / 16;
     if (nt == 4 && nk == 2) return launch_mma<4, 2>(a, st);
     if (nt == 8 && nk == 4) return launch_mma<8, 4>(a, st);
+    if (nt == 8 && nk == 6) return launch_mma<8, 6>(a, st);
     if (nt == 12 && nk == 6) return launch_mma<12, 6>(a, st);
     if (nt == 16 && nk == 8) return launch_mma<16, 8>(a, st);
     if (nt == 16 && nk == 12) return launch_mma<16, 12>(a, st);

@@ -420,6 +420,29 @@ def test_a_row_does_not_depend_on_the_batch():
     model.close()
 
 
+@pytest.mark.parametrize("fp32", [True, False])
+def test_many_sequences_in_short_slices(fp32):
+    """More heads than the GPU holds at a time, several tokens per slice without the chunked form, equal and unequal lengths."""
+    cfg, tens, W, _, _ = setup("recurrent")
+    batch = 200
+    model = lumi_b200.NmModel.from_tensors(cfg, tens, widen_weights=fp32)
+    sess = model.init_states(batch, 64)
+    g = np.random.default_rng(5)
+    prompts = g.integers(0, cfg.vocab_size, (batch, 14)).astype(np.uint32)
+    lens = g.integers(1, 10, batch).astype(np.int32)
+    lens[:2] = 9, 1
+    for ragged in (False, True):
+        sess.reset()
+        n = lens if ragged else np.full(batch, 9, np.int32)
+        outs = [sess.prefill_ragged(prompts[:, :9], n) if ragged else sess.prefill(prompts[:, :9])]
+        for i in range(4):
+            outs.append(sess.forward_step(prompts[np.arange(batch), n + i])[0])
+        for b in (0, 1, 77, 199):
+            ref = oz.forward(cfg.raw, W, prompts[b, :n[b] + 4])[0][n[b] - 1:]
+            assert rel(np.stack([o[b] for o in outs]), ref) < (1e-4 if fp32 else 2e-3), (ragged, b)
+    sess.close(); model.close()
+
+
 def test_cache_capacity_is_reported():
     """A cache smaller than the window refuses positions it cannot hold."""
     cfg = zt.config(64, 50, [zt.latent_attention(2, 16, 8, 16, 32, 100)])
