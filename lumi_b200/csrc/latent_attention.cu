@@ -100,12 +100,15 @@ __device__ __forceinline__ void halves2(float v0, float v1, uint32_t& hi, uint32
 
 constexpr int PS = kPageTokens + kPad;                    // row of the staged weights
 
-// Grid: (row, block of 16 heads, context slice).  Four warps: each takes 16 tokens of a staged page for the scores, and a quarter of
-// the latent's columns for the contexts.  NTW: 8-column tiles of a warp's quarter, at least.
+// Grid: (row, block of 16 heads, context slice).  Eight warps: for the scores a pair of them takes 16 tokens of a staged page, each half
+// of the key row; for the contexts each takes an eighth of the latent's columns.  NTW: 8-column tiles of a warp's eighth (an even
+// number of them where it is more than one), at least.
+constexpr int kThreads = 256;
 template <int NTW>
-__global__ void __launch_bounds__(128) latent_mma_kernel(LatentArgs a) {
+__global__ void __launch_bounds__(kThreads) latent_mma_kernel(LatentArgs a) {
     extern __shared__ __align__(16) unsigned char smem_raw[];
     __shared__ float wmax[4][16], wsum[4][16];
+    __shared__ float4 half_s[4][2][32];                   // scores over the second half of the key row
     __shared__ int is_last;
     const LatentShape ls(a.m);
     const int H = a.m.heads, RS = ls.row + kPad, stage_elems = kPageTokens * RS;
@@ -123,7 +126,7 @@ __global__ void __launch_bounds__(128) latent_mma_kernel(LatentArgs a) {
     const bool live = t < pass_tokens(a.row_len, a.ctl, slot, a.ts, a.t_abs0);
     auto put = [&](int m, int d, float v) { put_row(a.ctx, a.ch, a.cl, ((size_t)row * H + h0 + m) * ls.lp + d, v); };
     if (!live || (a.limit > 0 && pos >= a.limit)) {
-        if (split == 0 && (a.ts > 1 || live)) for (int i = tid; i < nh * ls.lp; i += 128) put(i / ls.lp, i % ls.lp, 0.f);
+        if (split == 0 && (a.ts > 1 || live)) for (int i = tid; i < nh * ls.lp; i += kThreads) put(i / ls.lp, i % ls.lp, 0.f);
         return;
     }
     const int32_t* pt = a.page_table + (size_t)slot * a.pages_per_seq;
@@ -135,7 +138,7 @@ __global__ void __launch_bounds__(128) latent_mma_kernel(LatentArgs a) {
     auto issue = [&](int pg) {
         __nv_bfloat16* s = stage + ((pg - pb) & 1) * stage_elems;
         const __nv_bfloat16* src = pool + (size_t)pt[pg % a.pages_per_seq] * kPageTokens * ls.row;
-        for (int i = tid; i < kPageTokens * rc; i += 128) {
+        for (int i = tid; i < kPageTokens * rc; i += kThreads) {
             const int r = i / rc, c = i - r * rc, p = pg * kPageTokens + r;
             const int bytes = p >= lo && p <= pos ? 16 : 0;           // 0: filled with zeros
             asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"((uint32_t)__cvta_generic_to_shared(s + r * RS + c * 8)), "l"(src + (size_t)i * 8), "r"(bytes) : "memory");
@@ -143,7 +146,7 @@ __global__ void __launch_bounds__(128) latent_mma_kernel(LatentArgs a) {
     };
     if (pb < pe) issue(pb);
     asm volatile("cp.async.commit_group;" ::: "memory");
-    for (int i = tid; i < 16 * (ls.row / 2); i += 128) {
+    for (int i = tid; i < 16 * (ls.row / 2); i += kThreads) {
         const int m = i / (ls.row / 2), c = 2 * (i % (ls.row / 2));
         float2 v = make_float2(0.f, 0.f);
         if (m < nh) v = *reinterpret_cast<const float2*>(a.qlat + ((size_t)row * H + h0 + m) * ls.row + c);
@@ -157,7 +160,7 @@ __global__ void __launch_bounds__(128) latent_mma_kernel(LatentArgs a) {
     float o[NTW][4];
 #pragma unroll
     for (int i = 0; i < NTW; ++i) { o[i][0] = 0.f; o[i][1] = 0.f; o[i][2] = 0.f; o[i][3] = 0.f; }
-    const int nks = ls.row / 16, ntw = ls.lp / 32, col0 = warp * (ls.lp / 4);
+    const int nks = ls.row / 16, ntw = ls.lp / 64, col0 = warp * (ls.lp / 8), tg = warp & 3, kh = warp >> 2;
     for (int pg = pb; pg < pe; ++pg) {
         asm volatile("cp.async.wait_group 0;" ::: "memory");
         __syncthreads();                                  // the page is here, and every warp has finished with the other stage
@@ -166,31 +169,43 @@ __global__ void __launch_bounds__(128) latent_mma_kernel(LatentArgs a) {
         const __nv_bfloat16* s = stage + ((pg - pb) & 1) * stage_elems;
         float sc[2][4] = {}, sl2[2][4] = {};              // products with the query's two halves
 #pragma unroll 4
-        for (int k = 0; k < nks; ++k) {
+        for (int k = kh * (nks / 2); k < (kh + 1) * (nks / 2); ++k) {      // (nks is a multiple of 4)
             uint32_t fh[4], fl[4], kb[4];
             const int qo = (lane & 15) * RS + k * 16 + (lane >> 4) * 8;
             ldm4(fh, qh + qo);
             ldm4(fl, ql + qo);
-            ldm4(kb, s + (warp * 16 + ((lane >> 4) << 3) + (lane & 7)) * RS + k * 16 + ((lane >> 3) & 1) * 8);
+            ldm4(kb, s + (tg * 16 + ((lane >> 4) << 3) + (lane & 7)) * RS + k * 16 + ((lane >> 3) & 1) * 8);
             mma_bf16(sc[0], fh, kb[0], kb[1]);
             mma_bf16(sc[1], fh, kb[2], kb[3]);
             mma_bf16(sl2[0], fl, kb[0], kb[1]);
             mma_bf16(sl2[1], fl, kb[2], kb[3]);
         }
-        float tm[2] = {kNoScore, kNoScore};
 #pragma unroll
-        for (int e = 0; e < 2; ++e)
+        for (int e = 0; e < 2; ++e) {
 #pragma unroll
-            for (int i = 0; i < 4; ++i) {
-                const int p = pg * kPageTokens + warp * 16 + e * 8 + 2 * tq + (i & 1);
-                sc[e][i] = p >= lo && p <= pos ? (sc[e][i] + sl2[e][i]) * sc2 : kNoScore;
-                tm[i >> 1] = fmaxf(tm[i >> 1], sc[e][i]);
+            for (int i = 0; i < 4; ++i) sc[e][i] += sl2[e][i];
+            if (kh == 1) half_s[tg][e][lane] = make_float4(sc[e][0], sc[e][1], sc[e][2], sc[e][3]);
+        }
+        __syncthreads();
+        if (kh == 0) {
+            float tm[2] = {kNoScore, kNoScore};
+#pragma unroll
+            for (int e = 0; e < 2; ++e) {
+                const float4 h = half_s[tg][e][lane];
+                const float hv[4] = {h.x, h.y, h.z, h.w};
+#pragma unroll
+                for (int i = 0; i < 4; ++i) {
+                    const int p = pg * kPageTokens + tg * 16 + e * 8 + 2 * tq + (i & 1);
+                    sc[e][i] = p >= lo && p <= pos ? (sc[e][i] + hv[i]) * sc2 : kNoScore;
+                    tm[i >> 1] = fmaxf(tm[i >> 1], sc[e][i]);
+                }
             }
 #pragma unroll
-        for (int c = 0; c < 2; ++c) {
-            tm[c] = fmaxf(tm[c], __shfl_xor_sync(0xffffffffu, tm[c], 1));
-            tm[c] = fmaxf(tm[c], __shfl_xor_sync(0xffffffffu, tm[c], 2));
-            if (tq == 0) wmax[warp][g + 8 * c] = tm[c];
+            for (int c = 0; c < 2; ++c) {
+                tm[c] = fmaxf(tm[c], __shfl_xor_sync(0xffffffffu, tm[c], 1));
+                tm[c] = fmaxf(tm[c], __shfl_xor_sync(0xffffffffu, tm[c], 2));
+                if (tq == 0) wmax[tg][g + 8 * c] = tm[c];
+            }
         }
         __syncthreads();
         float f[2];
@@ -202,6 +217,7 @@ __global__ void __launch_bounds__(128) latent_mma_kernel(LatentArgs a) {
             mx[c] = mn;
             lsum[c] *= f[c];
         }
+        if (kh == 0) {
 #pragma unroll
         for (int e = 0; e < 2; ++e) {
             float p[4];
@@ -211,10 +227,11 @@ __global__ void __launch_bounds__(128) latent_mma_kernel(LatentArgs a) {
             for (int c = 0; c < 2; ++c) {
                 uint32_t hi, low;
                 halves2(p[2 * c], p[2 * c + 1], hi, low);
-                const int at = (g + 8 * c) * PS + warp * 16 + e * 8 + 2 * tq;
+                const int at = (g + 8 * c) * PS + tg * 16 + e * 8 + 2 * tq;
                 *reinterpret_cast<uint32_t*>(ph + at) = hi;
                 *reinterpret_cast<uint32_t*>(pl + at) = low;
             }
+        }
         }
 #pragma unroll
         for (int i = 0; i < NTW; ++i) { o[i][0] *= f[0]; o[i][1] *= f[0]; o[i][2] *= f[1]; o[i][3] *= f[1]; }
@@ -227,8 +244,14 @@ __global__ void __launch_bounds__(128) latent_mma_kernel(LatentArgs a) {
             ldm4(fl, pl + po);
             const __nv_bfloat16* v = s + (k * 16 + (((lane >> 3) & 1) << 3) + (lane & 7)) * RS + col0 + (lane >> 4) * 8;
 #pragma unroll
-            for (int dn = 0; dn < NTW / 2; ++dn) {
-                if (2 * dn < ntw) {
+            for (int dn = 0; dn < (NTW + 1) / 2; ++dn) {
+                if constexpr (NTW == 1) {                 // eight columns
+                    uint32_t v0, v1;
+                    asm volatile("ldmatrix.sync.aligned.m8n8.x2.trans.shared.b16 {%0, %1}, [%2];"
+                                 : "=r"(v0), "=r"(v1) : "r"((uint32_t)__cvta_generic_to_shared(s + (k * 16 + (lane & 15)) * RS + col0)) : "memory");
+                    mma_bf16(o[0], fh, v0, v1);
+                    mma_bf16(o[0], fl, v0, v1);
+                } else if (2 * dn < ntw) {
                     uint32_t vb[4];
                     ldm4t(vb, v + dn * 16);
                     mma_bf16(o[2 * dn], fh, vb[0], vb[1]);
@@ -244,7 +267,7 @@ __global__ void __launch_bounds__(128) latent_mma_kernel(LatentArgs a) {
     for (int c = 0; c < 2; ++c) {
         lsum[c] += __shfl_xor_sync(0xffffffffu, lsum[c], 1);
         lsum[c] += __shfl_xor_sync(0xffffffffu, lsum[c], 2);
-        if (tq == 0) wsum[warp][g + 8 * c] = lsum[c];
+        if (kh == 0 && tq == 0) wsum[tg][g + 8 * c] = lsum[c];
     }
     __syncthreads();
     float l[2];
@@ -314,7 +337,7 @@ __global__ void __launch_bounds__(128) latent_mma_kernel(LatentArgs a) {
         for (int sp = 0; sp < kSlices; ++sp) if (sp < nsplit) wt[sp * 16 + tid] = mv[sp] * inv;
     }
     __syncthreads();
-    for (int i = 4 * tid; i < nh * ls.lp; i += 4 * 128) {
+    for (int i = 4 * tid; i < nh * ls.lp; i += 4 * kThreads) {
         const int m = i / ls.lp;
         float4 v[kSlices];
 #pragma unroll
@@ -347,7 +370,7 @@ cudaError_t run_mma(const LatentArgs& a, cudaStream_t st) {
     auto kern = latent_mma_kernel<NTW>;
     const cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     if (e != cudaSuccess) return e;
-    return launch_rows(kern, dim3((unsigned)(a.nseq * a.ts), hb, nsplit), 128, smem, st, a);
+    return launch_rows(kern, dim3((unsigned)(a.nseq * a.ts), hb, nsplit), kThreads, smem, st, a);
 }
 
 }  // namespace
@@ -380,12 +403,14 @@ cudaError_t launch_latent_attention(const LatentArgs& a, cudaStream_t st) {
         int n = 0;
         return launch_window_attention(w, st, &n);
     }
-    const int ntw = ls.lp / 32;
-    if (ntw <= 2) return run_mma<2>(a, st);
-    if (ntw <= 4) return run_mma<4>(a, st);
-    if (ntw <= 8) return run_mma<8>(a, st);
-    if (ntw <= 16) return run_mma<16>(a, st);
-    return run_mma<20>(a, st);
+    switch (ls.lp / 64) {                                 // 8-column tiles per warp
+        case 1: return run_mma<1>(a, st);
+        case 2: return run_mma<2>(a, st);
+        case 3: case 4: return run_mma<4>(a, st);
+        case 5: case 6: return run_mma<6>(a, st);
+        case 7: case 8: return run_mma<8>(a, st);
+        default: return run_mma<10>(a, st);
+    }
 }
 
 }  // namespace lumi

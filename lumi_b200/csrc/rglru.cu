@@ -88,8 +88,10 @@ constexpr int kRun = 16;                                  // tokens per warp and
 
 // CTA = (32 channels, sequence); lane = channel, warp w of nw takes tokens [w kRun, (w + 1) kRun) of every round of nw kRun tokens.
 // A run's decays and inputs stay in registers between the two walks over it.
-__global__ void __launch_bounds__(1024) rglru_scan_kernel(RglruArgs a) {
-    __shared__ float prod[32][33], endv[32][33];
+// (NT: most threads; where there are CTAs enough, small ones overlap each other's phases better)
+template <int NT>
+__global__ void __launch_bounds__(NT, 1024 / NT) rglru_scan_kernel(RglruArgs a) {
+    __shared__ float prod[NT / 32][33], endv[NT / 32][33];
     const int nw = blockDim.x >> 5, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const int c = blockIdx.x * 32 + lane, sl = blockIdx.y, slot = a.b0 + sl;
     pdl_release();
@@ -104,16 +106,17 @@ __global__ void __launch_bounds__(1024) rglru_scan_kernel(RglruArgs a) {
     for (int r0 = 0; r0 < n; r0 += nw * kRun) {
         const int t0 = r0 + warp * kRun, cnt = max(0, min(kRun, n - t0));
         const size_t row0 = (size_t)sl * a.ts + t0;
+        const float *gp = a.gates + row0 * grow + gr, *up = a.u32 + row0 * a.channels + c, *yp = a.proj + row0 * a.ldp + a.off_y + c;
         float da[kRun], in[kRun];
 #pragma unroll
         for (int k = 0; k < kRun; ++k) {
             da[k] = 1.f;
             in[k] = 0.f;
             if (ok && k < cnt) {
-                const float* gt = a.gates + (row0 + k) * grow + gr;
+                const float* gt = gp + (size_t)k * grow;
                 float f;
                 decay_of(gt[0], sp, da[k], f);
-                in[k] = f * sigmoid_q(fmaxf(gt[16], -80.f)) * a.u32[(row0 + k) * a.channels + c];
+                in[k] = f * sigmoid_q(fmaxf(gt[16], -80.f)) * up[(size_t)k * a.channels];
             }
         }
         float p = 1.f, e = 0.f;
@@ -131,7 +134,7 @@ __global__ void __launch_bounds__(1024) rglru_scan_kernel(RglruArgs a) {
         for (int k = 0; k < kRun; ++k) {
             if (k < cnt) {
                 s = fmaf(da[k], s, in[k]);
-                if (ok) put_row(a.y32, a.yhi, a.ylo, (row0 + k) * a.ldy + c, s * gelu_tanh_f(a.proj[(row0 + k) * a.ldp + a.off_y + c]));
+                if (ok) put_row(a.y32, a.yhi, a.ylo, (row0 + k) * a.ldy + c, s * gelu_tanh_f(yp[(size_t)k * a.ldp]));
             }
         }
         __syncthreads();
@@ -258,7 +261,9 @@ cudaError_t launch_rglru_conv(const RglruArgs& a, cudaStream_t st) {
 
 cudaError_t launch_rglru_scan(const RglruArgs& a, cudaStream_t st) {
     const int nw = std::min(32, (a.ts + kRun - 1) / kRun);
-    return launch_rows(rglru_scan_kernel, dim3((a.channels + 31) / 32, a.nseq), 32 * nw, 0, st, a);
+    const dim3 grid((a.channels + 31) / 32, a.nseq);
+    if (nw <= 16 || (long)grid.x * grid.y >= 296) return launch_rows(rglru_scan_kernel<512>, grid, 32 * std::min(nw, 16), 0, st, a);
+    return launch_rows(rglru_scan_kernel<1024>, grid, 32 * nw, 0, st, a);
 }
 
 cudaError_t launch_rglru_tail(const RglruArgs& a, cudaStream_t st) {
