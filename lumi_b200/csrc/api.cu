@@ -1580,6 +1580,10 @@ int32_t rglru_mixer(StepPlan& p, RowPass& r, const Layer& L, int li) {
 // Slices of at least this many tokens expand keys and values per head (bf16 caches).
 constexpr int kLatentExpandMin = 16;
 constexpr size_t kLatentExpandBytes = (size_t)2 << 30;    // of expanded keys and values at a time
+bool latent_expands(const lumi_session* s, const MixerSpec& m, int ts) {
+    const LatentShape ls(m);
+    return ts >= kLatentExpandMin && s->m->wdtype == LUMI_DTYPE_BF16 && ls.dk_pad <= 256 && ls.dv_pad <= 256;
+}
 // Sequences whose rings are expanded together.
 int latent_expand_seqs(const lumi_session* s, const MixerSpec& m, int nseq) {
     const LatentShape ls(m);
@@ -1593,7 +1597,7 @@ int32_t latent_mixer(StepPlan& p, RowPass& r, const Layer& L, int li) {
     const LatentShape ls(m);
     RowBufs& b = *r.b;
     const int rows = r.rows(), ldp = (int)L.s.in.rows;
-    const bool expand = r.ts >= kLatentExpandMin && p.tc && L.s.ukv.p != nullptr && ls.dk_pad <= 256 && ls.dv_pad <= 256;
+    const bool expand = p.tc && latent_expands(s, m, r.ts);
     LatentArgs a{};
     a.proj = b.proj; a.ldp = ldp; a.off_q = L.s.off_q; a.off_c = L.s.off_c;
     a.kv = s->lstate[li].kv; a.kv_is_f32 = s->m->wdtype == LUMI_DTYPE_BF16 ? 0 : 1;
@@ -2069,12 +2073,13 @@ int32_t prefill_listed(lumi_session* s, int batch, int T, bool with_head, float*
         LUMI_TRY(alloc_rows(s, s->pre, rows_max, true));
     }
     RowBufs& b = s->pre;
-    // latent attention: slices that do not expand keys and values need queries in the latent space; the others the expanded rows
-    const bool half = s->m->wdtype == LUMI_DTYPE_BF16;
+    // latent attention: rows of the expanded keys and values, or of queries in the latent space, whichever the slices take
     const int last_ts = T % TS == 0 ? TS : T % TS;
-    LUMI_TRY(ensure_latent_rows(s, b, !half ? rows_max : std::min(TS, last_ts) < kLatentExpandMin || s->opt_gemm == 1 ? (size_t)nb_max * std::min(TS, kLatentExpandMin) : 0));
+    size_t lat_rows = 0;
     for (const LayerSpec& L : c.specs) {
-        if (L.mixer.kind != MIXER_LATENT || !half || TS < kLatentExpandMin) continue;
+        if (L.mixer.kind != MIXER_LATENT) continue;
+        for (int ts : {TS, last_ts}) if (!latent_expands(s, L.mixer, ts)) lat_rows = std::max(lat_rows, (size_t)nb_max * ts);
+        if (!latent_expands(s, L.mixer, TS)) continue;
         const LatentShape ls(L.mixer);
         const size_t need = (size_t)latent_expand_seqs(s, L.mixer, nb_max) * s->pages_per_seq * kPageTokens * L.mixer.heads * (ls.dk_pad + ls.dv_pad);
         if (need > s->lat_kv_cap) {
@@ -2082,6 +2087,7 @@ int32_t prefill_listed(lumi_session* s, int batch, int T, bool with_head, float*
             LUMI_TRY(grow(s->lat_kv, s->lat_kv_cap, need));
         }
     }
+    LUMI_TRY(ensure_latent_rows(s, b, lat_rows));
     if (want != nullptr && want->size() > s->want_cap) LUMI_TRY(grow(s->want_idx, s->want_cap, want->size()));
     size_t wanted = 0;
     std::vector<int32_t> local;                           // outlives the copies below (synchronised before it changes)

@@ -20,7 +20,7 @@ constexpr float kNoScore = -1.0e30f;
 constexpr float kLog2e = 1.4426950408889634f;
 constexpr int kPad = 8;                                   // extra bf16 per staged row: no ldmatrix conflicts
 constexpr int kSlices = 16;
-constexpr int kSliceMin = 128;                            // tokens from which a slice of the context is worth a CTA
+constexpr int kSliceMin = 64;                            // tokens from which a slice of the context is worth a CTA
 
 template <typename T> __device__ __forceinline__ T cache_elem(float v);
 template <> __device__ __forceinline__ float cache_elem<float>(float v) { return v; }

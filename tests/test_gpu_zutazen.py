@@ -66,6 +66,7 @@ ALONE = {
     "latent_many_heads": [zt.latent_attention(19, 8, 4, 6, 72, 64)],
     "latent_large": [zt.latent_attention(5, 96, 64, 128, 512, 130)],
     "latent_larger": [zt.latent_attention(2, 40, 30, 24, 700, 65)],
+    "latent_wide_heads": [zt.latent_attention(2, 250, 16, 264, 48, 50)],
     "latent_unrotated": [zt.latent_attention(2, 48, 0, 40, 64, 1)],
     "latent_all": [zt.latent_attention(4, 32, 16, 32, 96, 0, scale=0.3)],
 }
