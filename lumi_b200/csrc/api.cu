@@ -846,6 +846,7 @@ extern "C" void lumi_session_free(lumi_session* s) {
     if (s->pos_freq) cudaFree(s->pos_freq);
     if (s->want_idx) cudaFree(s->want_idx);
     if (s->lat_kv) cudaFree(s->lat_kv);
+    if (s->ret_seg) cudaFree(s->ret_seg);
     if (s->ctl_host) cudaFreeHost(s->ctl_host);
     if (s->pin_tokens) cudaFreeHost(s->pin_tokens);
     if (s->ev0) cudaEventDestroy(s->ev0);
@@ -1533,6 +1534,7 @@ int32_t retention_mixer(StepPlan& p, RowPass& r, const Layer& L, int li) {
     int n = 0;
     // short slices and fp32 models go token by token (the chunked form's products are tf32 terms)
     const bool chunked = r.ts >= 16 && s->m->wdtype == LUMI_DTYPE_BF16 && retention_chunk_supported(m.dim, m.vdim);
+    if (chunked && retention_segment_floats(m, r.nseq, r.ts) <= s->ret_seg_cap) a.seg = s->ret_seg;
     const cudaError_t e = chunked ? launch_retention_chunk(a, p.st_lo, &n) : launch_retention_step(a, p.st_lo, &n);
     if (e == cudaErrorInvalidValue) return fail(LUMI_E_UNSUPPORTED, "retention heads of %d x %d are not built", m.dim, m.vdim);
     LUMI_CUDA(e);
@@ -2077,6 +2079,14 @@ int32_t prefill_listed(lumi_session* s, int batch, int T, bool with_head, float*
     const int last_ts = T % TS == 0 ? TS : T % TS;
     size_t lat_rows = 0;
     for (const LayerSpec& L : c.specs) {
+        if (L.mixer.kind == MIXER_RETENTION && s->m->wdtype == LUMI_DTYPE_BF16) {
+            size_t need = 0;
+            for (int nb : {nb_max, batch % nb_max}) for (int ts : {TS, last_ts}) need = std::max(need, retention_segment_floats(L.mixer, nb, ts));
+            if (need > s->ret_seg_cap) {
+                LUMI_CUDA(cudaStreamSynchronize(s->stream));
+                LUMI_TRY(grow(s->ret_seg, s->ret_seg_cap, need));
+            }
+        }
         if (L.mixer.kind != MIXER_LATENT) continue;
         for (int ts : {TS, last_ts}) if (!latent_expands(s, L.mixer, ts)) lat_rows = std::max(lat_rows, (size_t)nb_max * ts);
         if (!latent_expands(s, L.mixer, TS)) continue;

@@ -328,6 +328,8 @@ struct lumi_session {
     std::vector<lumi::LayerState> lstate;
     __nv_bfloat16* lat_kv = nullptr;   // latent attention, prompt slices: keys and values per head of a few sequences' rings
     size_t lat_kv_cap = 0;
+    float* ret_seg = nullptr;          // retention, prompt slices: states of segments
+    size_t ret_seg_cap = 0;
     lumi::RowBufs dec, pre;
     int kv_limit = 0;                  // positions at or past it are refused (0 = the ring takes any)
     int slice_max = 0;                 // most tokens of a sequence per pass (what the ring leaves beside the widest window)
@@ -682,7 +684,10 @@ struct RetentionArgs {
     float* y32; __nv_bfloat16 *yhi, *ylo; int ldy;
     float* o32;                                      // chunked form: read-out before its norm, [rows][H][dvp]
     int32_t* status;                                 // receives STATUS_TIMEOUT if a bounded wait gives up; may be null
+    float* seg;                                      // chunked form: retention_segment_floats elements, or null (in one piece)
 };
+// chunked form: room for the states of segments that run side by side (0: the slice goes in one piece)
+size_t retention_segment_floats(const MixerSpec& m, int nseq, int ts);
 cudaError_t launch_retention_step(const RetentionArgs& a, cudaStream_t st, int* launches);
 bool retention_chunk_supported(int dk, int dv);
 cudaError_t launch_retention_chunk(const RetentionArgs& a, cudaStream_t st, int* launches);

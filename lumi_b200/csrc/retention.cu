@@ -10,6 +10,8 @@
 //   retention_chunk_kernel   prompt slices in chunks of 64 tokens on the tensor cores.  With S_0 the state ahead of the chunk,
 //                            o_t = d^(t+1) S_0^T q_t + sum_{s <= t} d^(t-s) (q_t.k_s) v_s, and the state becomes
 //                            d^C S_0 + sum_s d^(C-1-s) k_s v_s^T.  Products take fp32 operands as two tf32 terms each.
+//                            Few heads: a sequence's slice is cut into segments that run side by side; first every segment's own
+//                            contribution to the state, then (retention_join_kernel) the state ahead of each, then the outputs.
 #include "rows.cuh"
 #include "tf32.cuh"
 
@@ -224,10 +226,12 @@ __device__ __forceinline__ void stage_rows(float* dst, int ldd, const float* src
     }
 }
 
-// CTA = (head, block of value columns, sequence).  A pair of warps owns 8 NTW columns of the state and of O from start to end, each
-// of the two half of the rows.
-template <int NTW>
-__global__ void __launch_bounds__(512) retention_chunk_kernel(RetentionArgs a, int dk16) {
+enum ChunkMode { CHUNK_ALL = 0, CHUNK_STATE, CHUNK_OUT };
+// CTA = (head, block of value columns, sequence and segment of seg_tokens).  A pair of warps owns 8 NTW columns of the state and of O
+// from start to end, each of the two half of the rows.  CHUNK_STATE: the segment's contribution to the state alone, into a.seg;
+// CHUNK_OUT: outputs, from the state in a.seg.
+template <int NTW, int MODE>
+__global__ void __launch_bounds__(512) retention_chunk_kernel(RetentionArgs a, int dk16, int seg_tokens, int segs) {
     extern __shared__ __align__(16) float sm[];
     const int nthr = blockDim.x, nw = nthr >> 5, dvb = nw * 4 * NTW;
     const int SK = chunk_sk(dk16), SS = chunk_ss(dvb);
@@ -237,27 +241,29 @@ __global__ void __launch_bounds__(512) retention_chunk_kernel(RetentionArgs a, i
     float* Vs = Ss + dk16 * SS;                           // [CH][SS]
     float* Ps = Vs + CH * SS;                             // [CH][SA]
     float* pw = Ps + CH * SA;                             // powers of the decay
-    const int h = blockIdx.x, sl = blockIdx.z, slot = a.b0 + sl, v0 = blockIdx.y * dvb;
+    const int h = blockIdx.x, sl = MODE == CHUNK_ALL ? blockIdx.z : blockIdx.z / segs, seg = MODE == CHUNK_ALL ? 0 : blockIdx.z % segs;
+    const int slot = a.b0 + sl, v0 = blockIdx.y * dvb;
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, tq = lane & 3;
     for (int i = tid; i < kDecayPowers; i += nthr) pw[i] = a.decay_pow[(size_t)h * kDecayPowers + i];
     pdl_release();
     pdl_sync();
-    const int n = pass_tokens(a.row_len, a.ctl, slot, a.ts, a.t_abs0);
-    if (n == 0) return;
+    const int n = min(pass_tokens(a.row_len, a.ctl, slot, a.ts, a.t_abs0), MODE == CHUNK_ALL ? a.ts : (seg + 1) * seg_tokens);
+    const int t_first = seg * seg_tokens;
+    if (n <= t_first && MODE != CHUNK_STATE) return;
     const int pos0 = a.pos[slot];
-    float* Sg = a.S + ((size_t)slot * a.H + h) * a.dk * a.dvp;
+    float* Sg = (MODE == CHUNK_ALL ? a.S + ((size_t)slot * a.H + h) * a.dk * a.dvp : a.seg + ((size_t)blockIdx.z * a.H + h) * a.dk * a.dvp);
     for (int i = tid; i < dk16 * dvb; i += nthr) {
         const int r = i / dvb, c = i % dvb;
-        Ss[r * SS + c] = r < a.dk && v0 + c < a.dvp ? Sg[(size_t)r * a.dvp + v0 + c] : 0.f;
+        Ss[r * SS + c] = MODE != CHUNK_STATE && r < a.dk && v0 + c < a.dvp ? Sg[(size_t)r * a.dvp + v0 + c] : 0.f;
     }
     const int n0 = (warp >> 1) * 8 * NTW, half = warp & 1;      // this warp's columns of the block, and its half of the rows
     const bool kvec = ((a.dk | a.ldp | a.off_q | a.off_k) & 3) == 0, vvec = ((a.dv | a.ldp | a.off_v) & 3) == 0;
     const int hd = a.rot.dims / 2;
-    for (int t0 = 0; t0 < n; t0 += CH) {
+    for (int t0 = t_first; t0 < n; t0 += CH) {
         const int nt = min(CH, n - t0);
         const float* base = a.proj + (size_t)(sl * a.ts + t0) * a.ldp;
         __syncthreads();                                  // everything of the chunk before has been read
-        stage_rows(Qs, SK, base + a.off_q + h * a.dk, a.ldp, nt, a.dk, dk16, kvec, tid, nthr);
+        if (MODE != CHUNK_STATE) stage_rows(Qs, SK, base + a.off_q + h * a.dk, a.ldp, nt, a.dk, dk16, kvec, tid, nthr);
         stage_rows(Ks, SK, base + a.off_k + h * a.dk, a.ldp, nt, a.dk, dk16, kvec, tid, nthr);
         stage_rows(Vs, SS, base + a.off_v + h * a.dv + v0, a.ldp, nt, a.dv - v0, dvb, vvec, tid, nthr);
         asm volatile("cp.async.commit_group;" ::: "memory");
@@ -268,13 +274,17 @@ __global__ void __launch_bounds__(512) retention_chunk_kernel(RetentionArgs a, i
             const float2 cs = rot_cos_sin(pos0 + t0 + r, a.freq[p]);
             float* q = Qs + r * SK;
             float* k = Ks + r * SK;
-            const float q0 = q[c0], q1 = q[c1], k0 = k[c0] * a.k_scale, k1 = k[c1] * a.k_scale;
-            q[c0] = fmaf(q0, cs.x, -q1 * cs.y); q[c1] = fmaf(q1, cs.x, q0 * cs.y);
+            const float k0 = k[c0] * a.k_scale, k1 = k[c1] * a.k_scale;
+            if (MODE != CHUNK_STATE) {
+                const float q0 = q[c0], q1 = q[c1];
+                q[c0] = fmaf(q0, cs.x, -q1 * cs.y); q[c1] = fmaf(q1, cs.x, q0 * cs.y);
+            }
             k[c0] = fmaf(k0, cs.x, -k1 * cs.y); k[c1] = fmaf(k1, cs.x, k0 * cs.y);
         }
         const int rest = a.dk - a.rot.dims;
         for (int i = tid; i < CH * rest; i += nthr) Ks[i / rest * SK + a.rot.dims + i % rest] *= a.k_scale;
         __syncthreads();
+        if constexpr (MODE != CHUNK_STATE) {
         // P by 16 x 16 blocks on and below the diagonal
         for (int u = warp; u < 10; u += nw) {
             const int rt = u < 1 ? 0 : (u < 3 ? 1 : (u < 6 ? 2 : 3)), ct = u - rt * (rt + 1) / 2;
@@ -334,6 +344,8 @@ __global__ void __launch_bounds__(512) retention_chunk_kernel(RetentionArgs a, i
                         *reinterpret_cast<float2*>(a.o32 + ((size_t)(sl * a.ts + t0 + t) * a.H + h) * a.dvp + c) = make_float2(ro[r2][e][i], ro[r2][e][i + 1]);
                 }
         }
+        }
+        if (MODE == CHUNK_OUT && t0 + CH >= n) break;     // nothing reads the state any more
         // state, 64 rows at a time
         const float dec = pw[nt];
         for (int mb = 0; mb < dk16; mb += 64) {
@@ -374,11 +386,36 @@ __global__ void __launch_bounds__(512) retention_chunk_kernel(RetentionArgs a, i
             }
         }
     }
+    if (MODE == CHUNK_OUT) return;
     __syncthreads();
     for (int i = tid; i < dk16 * dvb; i += nthr) {
         const int r = i / dvb, c = i % dvb;
         if (r < a.dk && v0 + c < a.dvp) Sg[(size_t)r * a.dvp + v0 + c] = Ss[r * SS + c];
     }
+}
+
+// a.seg: contributions of the segments -> the states ahead of them; the state itself moves to the end of the slice.  One thread per
+// four neighbouring elements of a head's state.
+__global__ void __launch_bounds__(256) retention_join_kernel(RetentionArgs a, int seg_tokens, int segs) {
+    const int h = blockIdx.y, sl = blockIdx.z, slot = a.b0 + sl, i = blockIdx.x * 256 + threadIdx.x, n4 = a.dk * (a.dvp >> 2);
+    const float* pw = a.decay_pow + (size_t)h * kDecayPowers;
+    pdl_release();
+    pdl_sync();
+    const int n = pass_tokens(a.row_len, a.ctl, slot, a.ts, a.t_abs0);
+    if (i >= n4 || n == 0) return;
+    float4* S = reinterpret_cast<float4*>(a.S + ((size_t)slot * a.H + h) * a.dk * a.dvp) + i;
+    float4 s = *S;
+    for (int g = 0; g < segs; ++g) {
+        const int len = max(0, min(seg_tokens, n - g * seg_tokens));
+        if (len == 0) break;
+        float4* L = reinterpret_cast<float4*>(a.seg + ((size_t)(sl * segs + g) * a.H + h) * a.dk * a.dvp) + i;
+        const float4 l = *L;
+        float f = pw[len % CH];                           // decay over the segment
+        for (int c = len / CH; c > 0; --c) f *= pw[CH];
+        *L = s;
+        s = make_float4(fmaf(f, s.x, l.x), fmaf(f, s.y, l.y), fmaf(f, s.z, l.z), fmaf(f, s.w, l.w));
+    }
+    *S = s;
 }
 
 constexpr size_t kSmemMax = 227 * 1024 - 1024;
@@ -441,17 +478,50 @@ bool retention_chunk_supported(int dk, int dv) {
     return chunk_shape(dk, dv, 1 << 20, &nw, &ntw) || chunk_shape(dk, dv, 1, &nw, &ntw);
 }
 
-cudaError_t launch_retention_chunk(const RetentionArgs& a, cudaStream_t st, int* launches) {
-    int nw = 0, ntw = 0;
-    if (!chunk_shape(a.dk, a.dv, (long)a.nseq * a.H, &nw, &ntw)) return cudaErrorInvalidValue;
+// Segments of a slice: as many as fill the SMs with CTAs of the widest column blocks; 1 where the heads alone do.
+static int segments_of(int H, int dk, int dv, int nseq, int ts, int* nw, int* ntw, int* seg_tokens) {
+    const int chunks = (ts + CH - 1) / CH;
+    *seg_tokens = chunks * CH;
+    if (!chunk_shape(dk, dv, 1 << 20, nw, ntw)) return 1;
+    const int dvb = *nw * *ntw * 8, units = nseq * H * ((dv + dvb - 1) / dvb), want = units > 0 ? 148 / units : 1;
+    if (want < 2 || chunks < 2) return 1;
+    const int per = (chunks + want - 1) / want;
+    *seg_tokens = per * CH;
+    return (chunks + per - 1) / per;
+}
+
+size_t retention_segment_floats(const MixerSpec& m, int nseq, int ts) {
+    int nw, ntw, st;
+    const int segs = segments_of(m.heads, m.dim, m.vdim, nseq, ts, &nw, &ntw, &st);
+    return segs > 1 ? (size_t)nseq * segs * m.heads * m.dim * ((m.vdim + 3) / 4 * 4) : 0;
+}
+
+template <int MODE>
+static cudaError_t chunk_launch(const RetentionArgs& a, int nw, int ntw, int seg_tokens, int segs, cudaStream_t st) {
     const int dk16 = (a.dk + 15) / 16 * 16, dvb = nw * ntw * 8;
     const size_t smem = chunk_smem(dk16, dvb);
-    const dim3 grid(a.H, (a.dv + dvb - 1) / dvb, a.nseq);
-    auto kern = ntw == 2 ? retention_chunk_kernel<2> : retention_chunk_kernel<1>;
-    cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    const dim3 grid(a.H, (a.dv + dvb - 1) / dvb, (unsigned)(a.nseq * segs));
+    auto kern = ntw == 2 ? retention_chunk_kernel<2, MODE> : retention_chunk_kernel<1, MODE>;
+    const cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     if (e != cudaSuccess) return e;
-    if ((e = launch_rows(kern, grid, nw * 64, smem, st, a, dk16)) != cudaSuccess) return e;
+    return launch_rows(kern, grid, nw * 64, smem, st, a, dk16, seg_tokens, segs);
+}
+
+cudaError_t launch_retention_chunk(const RetentionArgs& a, cudaStream_t st, int* launches) {
+    int nw = 0, ntw = 0, seg_tokens = 0;
+    const int segs = a.seg != nullptr ? segments_of(a.H, a.dk, a.dv, a.nseq, a.ts, &nw, &ntw, &seg_tokens) : 1;
+    cudaError_t e;
     *launches = 2;
+    if (segs > 1) {
+        if ((e = chunk_launch<CHUNK_STATE>(a, nw, ntw, seg_tokens, segs, st)) != cudaSuccess) return e;
+        e = launch_rows(retention_join_kernel, dim3((a.dk * (a.dvp / 4) + 255) / 256, a.H, a.nseq), 256, 0, st, a, seg_tokens, segs);
+        if (e != cudaSuccess) return e;
+        if ((e = chunk_launch<CHUNK_OUT>(a, nw, ntw, seg_tokens, segs, st)) != cudaSuccess) return e;
+        *launches = 4;
+    } else {
+        if (!chunk_shape(a.dk, a.dv, (long)a.nseq * a.H, &nw, &ntw)) return cudaErrorInvalidValue;
+        if ((e = chunk_launch<CHUNK_ALL>(a, nw, ntw, 0, 1, st)) != cudaSuccess) return e;
+    }
     const HeadGateArgs hg{a.o32, a.H, a.dv, a.dvp, a.proj + a.off_g, a.ldp, nullptr, a.eps, a.row_len, a.t_abs0, a.ctl, a.nseq, a.ts, a.b0, a.y32, a.yhi, a.ylo, a.ldy};
     return launch_head_gate(hg, st);
 }
