@@ -1571,11 +1571,9 @@ int32_t rglru_mixer(StepPlan& p, RowPass& r, const Layer& L, int li) {
                            nullptr, nullptr, 0};
     LUMI_TRY(grouped_product(p, r.rows(), q));
     mark(p);
-    LUMI_CUDA(launch_rglru_scan(a, p.st_lo));
-    if (m.taps > 1) {
-        mark(p);
-        LUMI_CUDA(launch_rglru_tail(a, p.st_lo));
-    }
+    int n = 0;
+    LUMI_CUDA(launch_rglru_scan(a, p.st_lo, &n));
+    p.n += n - 1;                                         // mark() counted one
     return LUMI_OK;
 }
 

@@ -710,8 +710,7 @@ struct RglruArgs {
     float* y32; __nv_bfloat16 *yhi, *ylo; int ldy;
 };
 cudaError_t launch_rglru_conv(const RglruArgs& a, cudaStream_t st);
-cudaError_t launch_rglru_scan(const RglruArgs& a, cudaStream_t st);
-cudaError_t launch_rglru_tail(const RglruArgs& a, cudaStream_t st);
+cudaError_t launch_rglru_scan(const RglruArgs& a, cudaStream_t st, int* launches);      // and the ring's new contents
 constexpr int kRglruStepRows = 32;                    // rows up to which a decode token takes the one-launch form
 bool rglru_step_supported(const RglruArgs& a);
 cudaError_t launch_rglru_step(const RglruArgs& a, cudaStream_t st);      // a decode token, everything in one launch

@@ -4,6 +4,7 @@
 //   log a = -rate r softplus(lam),   S_t = a S_{t-1} + sqrt(1 - a^2) i u,   output S * gelu(y)
 //
 //   rglru_step_kernel   a decode token, everything in one launch: a CTA takes one block of channels of a few sequences
+//   rglru_conv_one_kernel, rglru_point_kernel   the same for many sequences, around a product of all rows with the gates' blocks
 //   rglru_conv_kernel   rows of a pass: convolutions, with the halves the block products take
 //   rglru_scan_kernel   gates, recurrence and output of a pass: warps take consecutive runs of tokens, the runs are joined through
 //                       their decay products and end values
@@ -155,7 +156,114 @@ __global__ void __launch_bounds__(256) rglru_tail_kernel(RglruArgs a) {
         a.conv[((size_t)slot * a.taps + (pos0 + n - d) % a.taps) * a.channels + c] = a.proj[(size_t)(sl * a.ts + n - d) * a.ldp + a.off_x + c];
 }
 
-// ---- a decode token -----------------------------------------------------------------------------------------------
+// ---- a decode token, many sequences: one thread per V neighbouring channels of a sequence ---------------------------
+template <int V> struct Vec;
+template <> struct Vec<1> {
+    static __device__ __forceinline__ void load(const float* p, float (&v)[1]) { v[0] = *p; }
+    static __device__ __forceinline__ void store(float* p, const float (&v)[1]) { *p = v[0]; }
+};
+template <> struct Vec<4> {
+    static __device__ __forceinline__ void load(const float* p, float (&v)[4]) {
+        const float4 t = *reinterpret_cast<const float4*>(p);
+        v[0] = t.x; v[1] = t.y; v[2] = t.z; v[3] = t.w;
+    }
+    static __device__ __forceinline__ void store(float* p, const float (&v)[4]) { *reinterpret_cast<float4*>(p) = make_float4(v[0], v[1], v[2], v[3]); }
+};
+// (rows of halves start on multiples of four elements wherever V is 4)
+template <int V>
+__device__ __forceinline__ void put_halves(__nv_bfloat16* hi, __nv_bfloat16* lo, size_t o, const float (&v)[V]) {
+    __nv_bfloat16 h[V], l[V];
+#pragma unroll
+    for (int e = 0; e < V; ++e) bf16_halves(v[e], h[e], l[e]);
+    if constexpr (V == 4) {
+        *reinterpret_cast<__nv_bfloat162*>(hi + o) = __halves2bfloat162(h[0], h[1]);
+        *reinterpret_cast<__nv_bfloat162*>(hi + o + 2) = __halves2bfloat162(h[2], h[3]);
+        if (lo != nullptr) {
+            *reinterpret_cast<__nv_bfloat162*>(lo + o) = __halves2bfloat162(l[0], l[1]);
+            *reinterpret_cast<__nv_bfloat162*>(lo + o + 2) = __halves2bfloat162(l[2], l[3]);
+        }
+    } else {
+        hi[o] = h[0];
+        if (lo != nullptr) lo[o] = l[0];
+    }
+}
+
+template <int V>
+__global__ void __launch_bounds__(128) rglru_conv_one_kernel(RglruArgs a) {
+    const int c = (blockIdx.x * 128 + threadIdx.x) * V, sl = blockIdx.y, slot = a.b0 + sl;
+    pdl_release();
+    float v[V];
+    float4 w4[V];                                         // filters of four taps: a channel's in one load
+    if (c < a.channels) {
+        Vec<V>::load(a.conv_b + c, v);
+        if (a.taps == 4)
+#pragma unroll
+            for (int e = 0; e < V; ++e) w4[e] = __ldg(reinterpret_cast<const float4*>(a.conv_w) + c + e);
+    }
+    const int pos = a.pos[slot];
+    pdl_sync();
+    if (c >= a.channels) return;
+    const bool live = pass_tokens(a.row_len, a.ctl, slot, 1, a.t_abs0) > 0;
+    const float* ring = a.conv + (size_t)slot * a.taps * a.channels + c;
+    if (a.taps == 4) {
+        float x[4][V] = {};
+#pragma unroll
+        for (int d = 1; d < 4; ++d) if (pos >= d) Vec<V>::load(ring + (size_t)((pos - d) & 3) * a.channels, x[3 - d]);
+        Vec<V>::load(a.proj + (size_t)sl * a.ldp + a.off_x + c, x[3]);
+#pragma unroll
+        for (int e = 0; e < V; ++e) v[e] = fmaf(w4[e].w, x[3][e], fmaf(w4[e].z, x[2][e], fmaf(w4[e].y, x[1][e], fmaf(w4[e].x, x[0][e], v[e]))));
+    } else for (int j = 0; j < a.taps; ++j) {
+        const int d = a.taps - 1 - j;
+        float x[V] = {};
+        if (d == 0) Vec<V>::load(a.proj + (size_t)sl * a.ldp + a.off_x + c, x);
+        else if (pos >= d) Vec<V>::load(ring + (size_t)((pos - d) % a.taps) * a.channels, x);
+#pragma unroll
+        for (int e = 0; e < V; ++e) v[e] = fmaf(a.conv_w[(size_t)(c + e) * a.taps + j], x[e], v[e]);
+    }
+#pragma unroll
+    for (int e = 0; e < V; ++e) if (!live) v[e] = 0.f;
+    Vec<V>::store(a.u32 + (size_t)sl * a.channels + c, v);
+    const int bs = a.channels / a.blocks;
+    if (a.uh != nullptr) put_halves<V>(a.uh, a.ul, (size_t)sl * a.blocks * a.bp + c / bs * a.bp + c % bs, v);
+}
+
+template <int V>
+__global__ void __launch_bounds__(128) rglru_point_kernel(RglruArgs a) {
+    const int c = (blockIdx.x * 128 + threadIdx.x) * V, sl = blockIdx.y, slot = a.b0 + sl;
+    pdl_release();
+    float lam[V], S[V], r[V], in[V], u[V], y[V], x[V];
+    float* Sp = a.S + (size_t)slot * a.channels + c;
+    const int pos = a.pos[slot];
+    if (c < a.channels) {                                 // the state belongs to the step before this one, which has ended
+        Vec<V>::load(a.lam + c, lam);
+        Vec<V>::load(Sp, S);
+    }
+    pdl_sync();
+    if (c >= a.channels || pass_tokens(a.row_len, a.ctl, slot, 1, a.t_abs0) == 0) return;
+    const int bs = a.channels / a.blocks, i = c % bs;
+    const float* gt = a.gates + (size_t)sl * a.blocks * 2 * a.bp + c / bs * 2 * a.bp + (i >> 4) * 32 + (i & 15);
+    const float* pr = a.proj + (size_t)sl * a.ldp;
+    Vec<V>::load(gt, r);
+    Vec<V>::load(gt + 16, in);
+    Vec<V>::load(a.u32 + (size_t)sl * a.channels + c, u);
+    Vec<V>::load(pr + a.off_y + c, y);
+    Vec<V>::load(pr + a.off_x + c, x);
+#pragma unroll
+    for (int e = 0; e < V; ++e) {
+        float d, f;
+        decay_of(r[e], a.rate * softplus_f(lam[e]), d, f);
+        S[e] = fmaf(d, S[e], f * sigmoid_q(fmaxf(in[e], -80.f)) * u[e]);
+        y[e] = S[e] * gelu_tanh_f(y[e]);
+    }
+    Vec<V>::store(Sp, S);
+    Vec<V>::store(a.conv + ((size_t)slot * a.taps + pos % a.taps) * a.channels + c, x);      // for later tokens
+    if (a.y32 != nullptr) Vec<V>::store(a.y32 + (size_t)sl * a.ldy + c, y);
+    if (a.yhi != nullptr) put_halves<V>(a.yhi, a.ylo, (size_t)sl * a.ldy + c, y);
+}
+// four channels per thread where blocks and rows allow it
+bool by_four(const RglruArgs& a) { return ((a.channels | a.channels / a.blocks | a.ldp | a.ldy | a.off_x | a.off_y) & 3) == 0; }
+
+// ---- a decode token, few sequences ---------------------------------------------------------------------------------
 constexpr int kStepRows = 4;                              // sequences per CTA
 
 __device__ __forceinline__ void widen16(const uint4& v, const float*, float (&w)[4]) {
@@ -251,6 +359,10 @@ size_t step_smem(const RglruArgs& a, int per) { return sizeof(float) * kStepRows
 }  // namespace
 
 cudaError_t launch_rglru_conv(const RglruArgs& a, cudaStream_t st) {
+    if (a.ts == 1 && a.nseq <= 65535) {
+        if (by_four(a)) return launch_rows(rglru_conv_one_kernel<4>, dim3((a.channels + 511) / 512, a.nseq), 128, 0, st, a);
+        return launch_rows(rglru_conv_one_kernel<1>, dim3((a.channels + 127) / 128, a.nseq), 128, 0, st, a);
+    }
     const int runs = (a.ts + kConvRows - 1) / kConvRows;
     const dim3 grid((unsigned)((long)a.nseq * runs), (a.channels + 127) / 128);
     if (a.taps == 2) return launch_rows(rglru_conv_kernel<2>, grid, 128, 0, st, a, runs);
@@ -259,14 +371,19 @@ cudaError_t launch_rglru_conv(const RglruArgs& a, cudaStream_t st) {
     return launch_rows(rglru_conv_kernel<0>, grid, 128, 0, st, a, runs);
 }
 
-cudaError_t launch_rglru_scan(const RglruArgs& a, cudaStream_t st) {
+cudaError_t launch_rglru_scan(const RglruArgs& a, cudaStream_t st, int* launches) {
+    *launches = 1;
+    if (a.ts == 1 && a.nseq <= 65535) {
+        if (by_four(a)) return launch_rows(rglru_point_kernel<4>, dim3((a.channels + 511) / 512, a.nseq), 128, 0, st, a);
+        return launch_rows(rglru_point_kernel<1>, dim3((a.channels + 127) / 128, a.nseq), 128, 0, st, a);
+    }
+    cudaError_t e;
     const int nw = std::min(32, (a.ts + kRun - 1) / kRun);
     const dim3 grid((a.channels + 31) / 32, a.nseq);
-    if (nw <= 16 || (long)grid.x * grid.y >= 296) return launch_rows(rglru_scan_kernel<512>, grid, 32 * std::min(nw, 16), 0, st, a);
-    return launch_rows(rglru_scan_kernel<1024>, grid, 32 * nw, 0, st, a);
-}
-
-cudaError_t launch_rglru_tail(const RglruArgs& a, cudaStream_t st) {
+    if (nw <= 16 || (long)grid.x * grid.y >= 296) e = launch_rows(rglru_scan_kernel<512>, grid, 32 * std::min(nw, 16), 0, st, a);
+    else e = launch_rows(rglru_scan_kernel<1024>, grid, 32 * nw, 0, st, a);
+    if (e != cudaSuccess || a.taps == 1) return e;
+    *launches = 2;
     return launch_rows(rglru_tail_kernel, dim3((a.channels + 255) / 256, a.nseq), 256, 0, st, a);
 }
 
